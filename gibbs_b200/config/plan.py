@@ -87,6 +87,8 @@ class ModelPlan:
     # for random weights: (fnmatch pattern of checkpoint names, value) pairs for vectors that are neither noise nor
     # gains around one (a norm weight stored around zero, a scale per channel); the first match wins
     random_values: tuple[tuple[str, float], ...] = ()
+    # residual vectors a token has (more than one: arrangements that mix several streams)
+    streams: int = 1
 
     def validate(self) -> None:
         for i, e in enumerate(self.order):

@@ -29,7 +29,8 @@ template <typename T>
 __global__ void embed_scaled_kernel(const T* __restrict__ table, const int* ids, float* out, int dim, int vocab,
                                     float scale, const T* __restrict__ pairs, int buckets, long long mul_prev,
                                     long long mul_cur, const int* tok_req, const int* tok_pos, const int* q_start,
-                                    const int* q_len, int* last, long long slot_stride, const int* slot_ids) {
+                                    const int* q_len, int* last, long long slot_stride, const int* slot_ids, int copies,
+                                    const float* __restrict__ freq) {
   __shared__ int before;
   pdl_trigger();
   const int row = blockIdx.x;
@@ -41,14 +42,23 @@ __global__ void embed_scaled_kernel(const T* __restrict__ table, const int* ids,
     count = q_len[r];
     pos = tok_pos[row];
     mine = last + (size_t)slot_ids[r] * slot_stride;
+  } else if (freq) {
+    pos = tok_pos[row];
   }
   pdl_wait();
   int id = __ldcg(ids + row);                       // (the kernel in front may have rewritten it)
   if (id < 0 || id >= vocab) id = 0;                // ids are checked on the host; a bad one reads row 0
   const T* src = table + (size_t)id * dim;
-  float* dst = out + (size_t)row * dim;
+  float* dst = out + (size_t)row * copies * dim;
   if (!pairs) {
-    for (int d = threadIdx.x; d < dim; d += blockDim.x) dst[d] = to_f32(src[d]) * scale;
+    for (int d = threadIdx.x; d < dim; d += blockDim.x) {
+      float v = to_f32(src[d]) * scale;
+      if (freq) {
+        const float ang = (float)pos * freq[d >> 1];
+        v += (d & 1) ? cosf(ang) : sinf(ang);
+      }
+      for (int c = 0; c < copies; ++c) dst[(size_t)c * dim + d] = v;
+    }
     return;
   }
   if (threadIdx.x == 0) {
@@ -61,7 +71,10 @@ __global__ void embed_scaled_kernel(const T* __restrict__ table, const int* ids,
   long long pr = buckets;
   if (before >= 0) pr = ((long long)before * mul_prev + (long long)id * mul_cur) % buckets;
   const T* add = pairs + (size_t)pr * dim;
-  for (int d = threadIdx.x; d < dim; d += blockDim.x) dst[d] = fmaf(to_f32(src[d]), scale, to_f32(add[d]));
+  for (int d = threadIdx.x; d < dim; d += blockDim.x) {
+    const float v = fmaf(to_f32(src[d]), scale, to_f32(add[d]));
+    for (int c = 0; c < copies; ++c) dst[(size_t)c * dim + d] = v;
+  }
 }
 
 // How q and k are normed and turned (qk_prep's flags).
@@ -97,7 +110,8 @@ __global__ void qk_prep_kernel(const float* fused, long long ld, int k_col, int 
                                const float* __restrict__ k_gain, const float* __restrict__ inv_freq, int rot_dims,
                                const int* tok_req, const int* tok_pos, const int* block_table, int bt_stride,
                                int page_size, TC* k_pages, TC* v_pages, int n_pages, int H, int G, int dim, int vdim,
-                               int maps, int mode, float eps, TQ* q_out, long long ldq, int* status) {
+                               int maps, int mode, float eps, float temp_coef, float temp_every, TQ* q_out, long long ldq,
+                               int* status) {
   __shared__ float scratch[32];
   pdl_trigger();
   const int t = blockIdx.x;
@@ -107,6 +121,8 @@ __global__ void qk_prep_kernel(const float* fused, long long ld, int k_col, int 
   const bool whole = mode & PREP_NORM_WHOLE, per_head = mode & PREP_NORM_HEAD, halves = mode & PREP_ROT_HALVES;
   // PREP_NORM_AFTER: every head is turned first and then divided by the root mean square of the TURNED head (no gain)
   const bool after = mode & PREP_NORM_AFTER;
+  // a query grows with its position: 1 + coef * ln(floor((pos + 1) / every) + 1)
+  const float temp = temp_every > 0.f ? fmaf(temp_coef, logf(floorf((float)(pos + 1) / temp_every) + 1.f), 1.f) : 1.f;
   int page = -1;
   if (writes) page = block_table[(size_t)tok_req[t] * bt_stride + pos / page_size];
   pdl_wait();
@@ -131,14 +147,14 @@ __global__ void qk_prep_kernel(const float* fused, long long ld, int k_col, int 
       for (int d = lane; d < dim; d += 32) ss += row[h * dim + d] * row[h * dim + d];
       rstd = 1.0f / sqrtf(warp_sum(ss) / (float)dim + eps);
     }
-    float post = 1.f;
+    float post = temp;
     if (after) {
       float ss = 0.f;
       for (int d = lane; d < dim; d += 32) {
         const float v = prep_element(row, nullptr, true, 1.f, h * dim, d, rot_dims, halves, inv_freq, pos);
         ss += v * v;
       }
-      post = 1.0f / sqrtf(warp_sum(ss) / (float)dim + eps);
+      post = temp / sqrtf(warp_sum(ss) / (float)dim + eps);
     }
     for (int d = lane; d < dim; d += 32)
       q_out[(size_t)t * ldq + h * dim + d] = from_f32<TQ>(post * prep_element(row, normed ? q_gain : nullptr, per_head, rstd,
@@ -194,13 +210,16 @@ __device__ __forceinline__ float sa_sink_score(const float* __restrict__ scores,
 __device__ __forceinline__ float sa_top(float m, int sink, float z) { return sink ? fmaxf(m, z) : m; }
 __device__ __forceinline__ float sa_sink_weight(float M, int sink, float z) { return sink ? expf(z - M) : 0.f; }
 
-template <typename TC, typename TQ, typename TO, int VR>
+// With SIG there is no softmax: a visible key's weight is sigmoid(score + bias[head]) and nothing is normalised over
+// keys; a chunk's partial result is a plain sum (its first two numbers in the workspace are not used).
+template <typename TC, typename TQ, typename TO, int VR, bool SIG>
 __global__ void __launch_bounds__(32 * SA_WARPS)
 sink_attention_kernel(const TQ* q, long long ldq, const TC* k_pages, const TC* v_pages, const int* block_table,
                       int bt_stride, int page_size, int n_pages, const int* tok_req, const int* tok_pos,
                       const float* gate, long long ld_gate, TO* out, long long ldo, int H, int G, int dim, int vdim,
                       float scale, float softcap, int window, int sink, int splits, int chunk, float* ws, int maps,
-                      int blocked, const float* __restrict__ sink_scores, int keep_first, int* status) {
+                      int blocked, const float* __restrict__ sink_scores, int keep_first, int* status,
+                      const float* __restrict__ score_bias, float factor) {
   // (H counts heads of `dim` entries: `maps` of them make one query head, and a key row holds `maps` keys side
   // by side, of which head h scores against number h % maps)
   extern __shared__ __align__(16) float sm[];
@@ -240,6 +259,7 @@ sink_attention_kernel(const TQ* q, long long ldq, const TC* k_pages, const TC* v
 #pragma unroll
   for (int i = 0; i < VR; ++i) acc[i] = 0.f;
   float m = -INFINITY, l = 0.f;
+  const float bias = SIG && score_bias && live ? score_bias[h / maps] : 0.f;
   for (int k0 = k_begin; k0 <= k_end; k0 += SA_KT) {
     __syncthreads();                                          // the last tile has been used (and qs is written)
     if (threadIdx.x < SA_KT) {
@@ -276,14 +296,19 @@ sink_attention_kernel(const TQ* q, long long ldq, const TC* k_pages, const TC* v
     float s = (s0 + s1) * scale;
     if (softcap > 0.f) s = softcap * tanhf(s / softcap);
     if (k0 + lane > k_end) s = -INFINITY;
-    const float m_new = fmaxf(m, warp_max(s));
-    if (m_new == -INFINITY) continue;                         // (cannot happen: a tile holds a visible key)
-    const float corr = expf(m - m_new);                 // 0 while m = -inf
-    const float p = expf(s - m_new);                    // 0 for a key that is not seen
-    l = l * corr + warp_sum(p);
-    m = m_new;
+    float p;
+    if constexpr (SIG) {
+      p = hy_sigmoid(s + bias);                               // (0 for a key that is not seen)
+    } else {
+      const float m_new = fmaxf(m, warp_max(s));
+      if (m_new == -INFINITY) continue;                       // (cannot happen: a tile holds a visible key)
+      const float corr = expf(m - m_new);                     // 0 while m = -inf
+      p = expf(s - m_new);                                    // 0 for a key that is not seen
+      l = l * corr + warp_sum(p);
+      m = m_new;
 #pragma unroll
-    for (int i = 0; i < VR; ++i) acc[i] *= corr;
+      for (int i = 0; i < VR; ++i) acc[i] *= corr;
+    }
     const int n_keys = min(SA_KT, k_end - k0 + 1);
     for (int j = 0; j < n_keys; ++j) {
       const float pj = __shfl_sync(0xffffffffu, p, j);
@@ -307,8 +332,8 @@ sink_attention_kernel(const TQ* q, long long ldq, const TC* k_pages, const TC* v
   }
   const float z = sa_sink_score(sink_scores, h / maps);
   const float M = sa_top(m, sink, z);
-  const float e = expf(m - M);
-  const float inv = 1.0f / fmaf(e, l, sa_sink_weight(M, sink, z));
+  const float e = SIG ? 1.f : expf(m - M);
+  const float inv = SIG ? factor : 1.0f / fmaf(e, l, sa_sink_weight(M, sink, z));
 #pragma unroll
   for (int i = 0; i < VR; ++i) {
     const int dv = lane + 32 * i;
@@ -353,6 +378,25 @@ __global__ void sink_attention_merge_kernel(const float* ws, int splits, const f
   }
 }
 
+// One warp per (token, head): the chunks' plain sums, added in chunk order.
+template <typename TO>
+__global__ void sigmoid_attention_sum_kernel(const float* ws, int splits, const float* gate, long long ld_gate, TO* out,
+                                             long long ldo, int n, int H, int vdim, float factor) {
+  pdl_trigger();
+  pdl_wait();
+  const int lane = threadIdx.x & 31;
+  const long long idx = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (idx >= (long long)n * H) return;
+  const int t = (int)(idx / H), h = (int)(idx - (long long)t * H);
+  const float* w = ws + (size_t)idx * splits * (vdim + 2);
+  for (int dv = lane; dv < vdim; dv += 32) {
+    float a = 0.f;
+    for (int s = 0; s < splits; ++s) a += w[(size_t)s * (vdim + 2) + 2 + dv];
+    const float gt = gate ? hy_sigmoid(gate[(size_t)t * ld_gate + (size_t)h * vdim + dv]) : 1.f;
+    out[(size_t)t * ldo + (size_t)h * vdim + dv] = from_f32<TO>(a * factor * gt);
+  }
+}
+
 constexpr int SA_WS_ROWS = 1 << 16;
 
 }  // namespace
@@ -372,6 +416,20 @@ int gb_sink_attention_merge(const float* ws, int splits, const float* gate, long
     gb_launch(sink_attention_merge_kernel<float>, mgrid, dim3(128), 0, stream, ws, splits, gate, ld_gate, (float*)out, ldo,
               n, H, vdim, sink, sink_scores, maps);
   GB_CHECK_LAUNCH("sink_attention_merge");
+  return 1;
+}
+
+// The same for weights that are not normalised: the chunks' sums added up.
+int gb_sigmoid_attention_sum(const float* ws, int splits, const float* gate, long long ld_gate, void* out, int out_bf16,
+                             long long ldo, int n, int H, int vdim, float factor, cudaStream_t stream) {
+  const dim3 grid(gb_div_up((long long)n * H, 4));
+  if (out_bf16)
+    gb_launch(sigmoid_attention_sum_kernel<bf16>, grid, dim3(128), 0, stream, ws, splits, gate, ld_gate, (bf16*)out, ldo, n, H,
+              vdim, factor);
+  else
+    gb_launch(sigmoid_attention_sum_kernel<float>, grid, dim3(128), 0, stream, ws, splits, gate, ld_gate, (float*)out, ldo, n,
+              H, vdim, factor);
+  GB_CHECK_LAUNCH("sigmoid_attention (sum of chunks)");
   return 1;
 }
 
@@ -401,17 +459,21 @@ GB_API int gb_sink_attention_chunks(int n, int H, int G, int window, int max_ctx
 // a0 table, a1 its dtype, a2 token ids, a3 out (f32 [tokens, dim]), a4 tokens, a5 dim, a6 vocabulary; with a pair
 // table: a7 the table [buckets + 1, dim] (same dtype) or 0, a8 buckets, a9 factor of the id before, a10 factor of the
 // id, a11 token -> request, a12 token -> position, a13 first row per request, a14 rows per request, a15 the id
-// before (int32, one per slot) of slot 0, a16 elements between slots, a17 slot ids; f0 scale
+// before (int32, one per slot) of slot 0, a16 elements between slots, a17 slot ids; a18 copies of a row side by side in
+// out (0 means 1: out is [tokens, copies * dim]); a19 frequencies [(dim + 1) / 2] (f32) or 0: entry 2i also gets
+// sin(position * freq[i]), entry 2i + 1 the cosine (angles in 32-bit; not together with a pair table); f0 scale
 GB_OP(gb_op_embed_scaled) {
   const int n = (int)a[4], dim = (int)a[5];
   if (n <= 0) return 0;
   if (a[7] && a[8] <= 0) GB_FAIL(GB_ERR_ARG, "embed_scaled: a pair table of %lld buckets", a[8]);
+  if (a[7] && a[19]) GB_FAIL(GB_ERR_ARG, "embed_scaled: a pair table and position vectors");
+  const int copies = a[18] > 0 ? (int)a[18] : 1;
   const dim3 block(dim >= 1024 ? 256 : 128);
 #define EMBED(T)                                                                                                        \
   gb_launch(embed_scaled_kernel<T>, dim3(n), block, 0, ctx->stream, op_ptr<const T>(a[0]), op_ptr<const int>(a[2]),      \
             op_ptr<float>(a[3]), dim, (int)a[6], (float)f[0], op_ptr<const T>(a[7]), (int)a[8], a[9], a[10],              \
             op_ptr<const int>(a[11]), op_ptr<const int>(a[12]), op_ptr<const int>(a[13]), op_ptr<const int>(a[14]),      \
-            op_ptr<int>(a[15]), a[16], op_ptr<const int>(a[17]))
+            op_ptr<int>(a[15]), a[16], op_ptr<const int>(a[17]), copies, op_ptr<const float>(a[19]))
   if (a[1] == GB_BF16) EMBED(bf16); else EMBED(float);
 #undef EMBED
   GB_CHECK_LAUNCH("embed_scaled");
@@ -427,7 +489,8 @@ GB_OP(gb_op_embed_scaled) {
 // projection (gains as long as the projection), bit 1: q out is bfloat16 (else 32-bit), bit 2: the pages are bfloat16,
 // bit 3: norm over every head of `dim` entries (gains of `dim` entries, shared), bit 4: the rotation pairs entry i
 // with entry i + rot_dims / 2 (else adjacent entries), bit 5: every head of `dim` entries is divided by its root mean
-// square AFTER the rotation, without a gain; f0 eps
+// square AFTER the rotation, without a gain; f0 eps; f2 > 0: the query at position p is multiplied by
+// 1 + f1 * ln(floor((p + 1) / f2) + 1)
 GB_OP(gb_op_qk_prep) {
   const int n = (int)a[16], H = (int)a[17], G = (int)a[18], dim = (int)a[19], vdim = (int)a[20];
   const int maps = a[22] > 0 ? (int)a[22] : 1;
@@ -443,8 +506,8 @@ GB_OP(gb_op_qk_prep) {
   gb_launch(qk_prep_kernel<TC, TQ>, dim3(n), dim3(threads), 0, ctx->stream, op_ptr<const float>(a[0]), a[1], (int)a[2],    \
             (int)a[3], op_ptr<const float>(a[4]), op_ptr<const float>(a[5]), op_ptr<const float>(a[6]), (int)a[7],        \
             op_ptr<const int>(a[8]), op_ptr<const int>(a[9]), op_ptr<const int>(a[10]), (int)a[11], (int)a[12],           \
-            op_ptr<TC>(a[13]), op_ptr<TC>(a[14]), (int)a[15], H, G, dim, vdim, maps, mode, (float)f[0], op_ptr<TQ>(a[21]), \
-            ldq, ctx->status)
+            op_ptr<TC>(a[13]), op_ptr<TC>(a[14]), (int)a[15], H, G, dim, vdim, maps, mode, (float)f[0], (float)f[1], \
+            (float)f[2], op_ptr<TQ>(a[21]), ldq, ctx->status)
   if (flags & PREP_PAGES_BF16) { if (flags & PREP_Q_BF16) PREP(bf16, bf16); else PREP(bf16, float); }
   else { if (flags & PREP_Q_BF16) GB_FAIL(GB_ERR_ARG, "qk_prep: bfloat16 queries with 32-bit pages"); PREP(float, float); }
 #undef PREP
@@ -452,18 +515,12 @@ GB_OP(gb_op_qk_prep) {
   return 1;
 }
 
-// a0 q [tokens, heads * maps * dim], a1 key pages, a2 value pages, a3 block table, a4 its entries per request, a5 page
-// size, a6 number of pages, a7 token -> request, a8 token -> position, a9 gate logits (f32, [t, heads * vdim] at a row
-// stride) or 0, a10 that stride, a11 out [tokens, heads * maps * vdim], a12 its row stride, a13 tokens, a14 heads, a15 kv
-// heads, a16 dim, a17 vdim, a18 window (0: every earlier position), a19 longest context of the step (an upper bound
-// will do), a20 workspace for partial results (gb_sink_attention_workspace_rows() rows of vdim + 2 floats) or 0, a21
-// maps (0 means 1): a query head is `maps` heads of `dim` entries, a key row [maps * dim] holds one key for each, all
-// share the value; every map is a softmax of its own and has an output of its own;
-// flags bit 0: the softmax has a sink, bit 1: q is bfloat16 (else 32-bit), bit 2: the pages are, bit 3: out is,
-// bit 4: position p sees the positions of its own block of `window` positions, counted from 0, up to p (else
-// the last `window`); a22 a learned score of the sink per head (f32 [heads]) or 0: the sink's score is 0;
-// f0 scale, f1 soft cap (0: none), f2 keep_first: a windowed position also sees the positions below this number
-GB_OP(gb_op_sink_attention) {
+namespace {
+
+// (operands as of gb_op_sink_attention; SIG: weights sigmoid(score + score_bias[head]), the output times `factor`)
+template <bool SIG>
+int run_sink_attention(const GbPlanCtx* ctx, const long long* a, const double* f, int flags, const float* score_bias,
+                       float factor) {
   const int n = (int)a[13], G = (int)a[15], dim = (int)a[16], vdim = (int)a[17];
   const int maps = a[21] > 0 ? (int)a[21] : 1;
   const int H = (int)a[14] * maps;
@@ -490,15 +547,15 @@ GB_OP(gb_op_sink_attention) {
   do {                                                                                                                  \
     static size_t allowed = 48 * 1024;     /* raised once per size, before any stream capture replays the launch */    \
     if (smem > allowed) {                                                                                               \
-      GB_CUDA(cudaFuncSetAttribute(sink_attention_kernel<TC, TQ, TO, VR>, cudaFuncAttributeMaxDynamicSharedMemorySize,  \
+      GB_CUDA(cudaFuncSetAttribute(sink_attention_kernel<TC, TQ, TO, VR, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize,  \
                                    (int)smem));                                                                         \
       allowed = smem;                                                                                                   \
     }                                                                                                                   \
-    gb_launch(sink_attention_kernel<TC, TQ, TO, VR>, grid, block, smem, ctx->stream, op_ptr<const TQ>(a[0]),             \
+    gb_launch(sink_attention_kernel<TC, TQ, TO, VR, SIG>, grid, block, smem, ctx->stream, op_ptr<const TQ>(a[0]),             \
               (long long)H * dim, op_ptr<const TC>(a[1]), op_ptr<const TC>(a[2]), op_ptr<const int>(a[3]), (int)a[4],    \
               (int)a[5], (int)a[6], op_ptr<const int>(a[7]), op_ptr<const int>(a[8]), op_ptr<const float>(a[9]), a[10],  \
               op_ptr<TO>(a[11]), a[12], H, G, dim, vdim, (float)f[0], (float)f[1], (int)a[18], sink, splits, chunk, ws,  \
-              maps, blocked, sink_scores, keep_first, ctx->status);                                                    \
+              maps, blocked, sink_scores, keep_first, ctx->status, score_bias, factor);                                                  \
   } while (0)
 #define SA_VR(TC, TQ, TO)                                                                                               \
   do {                                                                                                                  \
@@ -515,7 +572,39 @@ GB_OP(gb_op_sink_attention) {
 #undef SA
   GB_CHECK_LAUNCH("sink_attention");
   if (splits == 1) return 1;
+  if (SIG) {
+    const int rs = gb_sigmoid_attention_sum(ws, splits, op_ptr<const float>(a[9]), a[10], op_ptr<void>(a[11]), ob ? 1 : 0, a[12],
+                                            n, H, vdim, factor, ctx->stream);
+    return rs < 0 ? rs : 2;
+  }
   const int rc = gb_sink_attention_merge(ws, splits, op_ptr<const float>(a[9]), a[10], op_ptr<void>(a[11]), ob ? 1 : 0, a[12],
                                          n, H, vdim, sink, sink_scores, maps, ctx->stream);
   return rc < 0 ? rc : 2;
+}
+
+}  // namespace
+
+// a0 q [tokens, heads * maps * dim], a1 key pages, a2 value pages, a3 block table, a4 its entries per request, a5 page
+// size, a6 number of pages, a7 token -> request, a8 token -> position, a9 gate logits (f32, [t, heads * vdim] at a row
+// stride) or 0, a10 that stride, a11 out [tokens, heads * maps * vdim], a12 its row stride, a13 tokens, a14 heads, a15 kv
+// heads, a16 dim, a17 vdim, a18 window (0: every earlier position), a19 longest context of the step (an upper bound
+// will do), a20 workspace for partial results (gb_sink_attention_workspace_rows() rows of vdim + 2 floats) or 0, a21
+// maps (0 means 1): a query head is `maps` heads of `dim` entries, a key row [maps * dim] holds one key for each, all
+// share the value; every map is a softmax of its own and has an output of its own;
+// flags bit 0: the softmax has a sink, bit 1: q is bfloat16 (else 32-bit), bit 2: the pages are, bit 3: out is,
+// bit 4: position p sees the positions of its own block of `window` positions, counted from 0, up to p (else
+// the last `window`); a22 a learned score of the sink per head (f32 [heads]) or 0: the sink's score is 0;
+// f0 scale, f1 soft cap (0: none), f2 keep_first: a windowed position also sees the positions below this number
+GB_OP(gb_op_sink_attention) { return run_sink_attention<false>(ctx, a, f, flags, nullptr, 1.f); }
+
+// Attention without a softmax: the weight of a visible key is sigmoid(score + bias[head]), the weights are not
+// normalised over keys, and the output is multiplied by a factor.  Operands as above, with a22 the bias per head (f32
+// [heads]) or 0, no sink and no kept first positions; f0 scale, f1 soft cap (0: none), f2 the factor
+GB_OP(gb_op_sigmoid_attention) {
+  if (flags & 1) GB_FAIL(GB_ERR_ARG, "sigmoid_attention: weights that are not normalised have no sink");
+  long long b[24];
+  for (int i = 0; i < 24; ++i) b[i] = a[i];
+  b[22] = 0;
+  const double g[3] = {f[0], f[1], 0.0};
+  return run_sink_attention<true>(ctx, b, g, flags, op_ptr<const float>(a[22]), (float)f[2]);
 }

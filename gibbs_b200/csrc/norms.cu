@@ -6,11 +6,12 @@
 //  gb_op_clamped_glu     out = g' * sigmoid(alpha g') * (u' + up_add) for rows [g | u] with clamps
 //  gb_op_gelu_mul_rows   g = gelu_tanh(g) * table[id, offset : offset + dim] (a per-token input)
 //  gb_op_gated_group_norm  out = rmsnorm_in_groups(y * silu(z)) * gain
-//  gb_op_act_rows        out = act(x), act one of gelu (erf), gelu (tanh), silu, relu: the unit of a feed-forward
+//  gb_op_act_rows        out = act(x), act one of gelu (erf), gelu (tanh), silu, relu, relu squared: the unit of a feed-forward
 //                        without a gate; or out = act(g) * u for rows [g | u]: a gated unit
 //  gb_op_scaled_sum      x += mult * (s1 * y1 + s2 * y2): two sublayers' outputs, scaled per channel, into the stream
 //  gb_op_head_norm       per head: out = rmsnorm(x - lambda * x2) * gain * sigmoid(gate) * factor, each of x2,
-//                        gain and gate optional: the norm behind a recurrence or behind two attention maps
+//                        gain and gate optional: the norm behind a recurrence or behind two attention maps; or of
+//                        x / (max(|den|, floor) + add) with two numbers per head: a read-out divided by its normaliser
 #include "hybrid.cuh"
 
 namespace {
@@ -417,14 +418,16 @@ __global__ void gated_group_norm_kernel(const float* y, long long ldy, const flo
     o[d] = from_f32<TO>(yr[d] * hy_silu(zr[d]) * rstd * gain[c0 + d]);
 }
 
-enum { ACT_GELU_ERF = 0, ACT_GELU_TANH = 1, ACT_SILU = 2, ACT_RELU = 3 };
+enum { ACT_GELU_ERF = 0, ACT_GELU_TANH = 1, ACT_SILU = 2, ACT_RELU = 3, ACT_RELU2 = 4, ACT_NONE = 5 };
 
 __device__ __forceinline__ float act_value(float z, int kind) {
   switch (kind) {
     case ACT_GELU_ERF: return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f));
     case ACT_GELU_TANH: return hy_gelu_tanh(z);
     case ACT_SILU: return hy_silu(z);
-    default: return fmaxf(z, 0.f);
+    case ACT_RELU: return fmaxf(z, 0.f);
+    case ACT_RELU2: z = fmaxf(z, 0.f); return z * z;
+    default: return z;
   }
 }
 
@@ -475,7 +478,9 @@ constexpr int HN_VR = 8;
 template <typename TO>
 __global__ void head_norm_kernel(const float* x, long long ldx, long long xh, const float* x2,
                                  const float* __restrict__ gain, const float* gate, long long ld_gate, TO* out,
-                                 long long ldo, int n, int H, int vdim, float eps, float lambda, float factor) {
+                                 long long ldo, int n, int H, int vdim, float eps, float lambda, float factor,
+                                 const float* den, const float* floor_, int gain_whole) {
+  // (with `den`, lambda is what is added to the divisor)
   pdl_trigger();
   pdl_wait();
   const int lane = threadIdx.x & 31;
@@ -485,11 +490,12 @@ __global__ void head_norm_kernel(const float* x, long long ldx, long long xh, co
   const size_t at = (size_t)t * ldx + (size_t)h * xh;
   float v[HN_VR];
   float ss = 0.f;
+  const float div = den ? fmaxf(fabsf(den[idx]), floor_[idx]) + lambda : 1.f;
 #pragma unroll
   for (int i = 0; i < HN_VR; ++i) {
     const int d = lane + 32 * i;
     v[i] = 0.f;
-    if (d < vdim) v[i] = x2 ? x[at + d] - lambda * x2[at + d] : x[at + d];
+    if (d < vdim) v[i] = x2 ? x[at + d] - lambda * x2[at + d] : den ? x[at + d] / div : x[at + d];
     ss += v[i] * v[i];
   }
   const float rstd = factor / sqrtf(warp_sum(ss) / (float)vdim + eps);
@@ -498,7 +504,7 @@ __global__ void head_norm_kernel(const float* x, long long ldx, long long xh, co
     const int d = lane + 32 * i;
     if (d >= vdim) continue;
     float o = v[i] * rstd;
-    if (gain) o *= gain[d];
+    if (gain) o *= gain[gain_whole ? h * vdim + d : d];
     if (gate) o *= hy_sigmoid(gate[(size_t)t * ld_gate + (size_t)h * vdim + d]);
     out[(size_t)t * ldo + (size_t)h * vdim + d] = from_f32<TO>(o);
   }
@@ -682,13 +688,13 @@ GB_OP(gb_op_scaled_sum) {
 }
 
 // a0 x (f32), a1 its row stride, a2 out [rows, inner], a3 out dtype, a4 its row stride, a5 rows, a6 inner, a7 which
-// function: 0 gelu (erf), 1 gelu (tanh), 2 silu, 3 relu, a8 gated (0/1): the rows are [g | u] of `inner` entries each
+// function: 0 gelu (erf), 1 gelu (tanh), 2 silu, 3 relu, 4 the square of relu, 5 none (a cast), a8 gated (0/1): the rows are [g | u] of `inner` entries each
 // and out = act(g) * u
 GB_OP(gb_op_act_rows) {
   const int n = (int)a[5], inner = (int)a[6];
   const int up = a[8] ? inner : 0;
   if (n <= 0) return 0;
-  if (a[7] > ACT_RELU) GB_FAIL(GB_ERR_ARG, "act_rows: function %lld", a[7]);
+  if (a[7] > ACT_NONE) GB_FAIL(GB_ERR_ARG, "act_rows: function %lld", a[7]);
   const size_t out_bytes = a[3] == GB_BF16 ? 2 : 4;
   if (inner % 4 == 0 && a[1] % 4 == 0 && a[4] % 4 == 0 && (a[0] & 15) == 0 && (a[2] & (4 * out_bytes - 1)) == 0) {
     const dim3 grid4(gb_div_up((long long)n * (inner / 4), 256)), block4(256);
@@ -714,21 +720,23 @@ GB_OP(gb_op_act_rows) {
 
 // a0 x (f32; head h of row t starts at t * a1 + h * a2), a1 row stride, a2 elements between heads, a3 x2 (f32, laid
 // out as x) or 0, a4 gain [vdim] (shared by the heads) or 0, a5 gate logits (f32, [t, h * vdim + d] at a row stride)
-// or 0, a6 that stride, a7 out [rows, heads * vdim], a8 out dtype, a9 its row stride, a10 rows, a11 heads, a12 vdim;
-// f0 eps, f1 lambda, f2 factor
+// or 0, a6 that stride, a7 out [rows, heads * vdim], a8 out dtype, a9 its row stride, a10 rows, a11 heads, a12 vdim,
+// a13 den [rows, heads] (f32) or 0: x is first divided by max(|den|, floor) + f1 (then no x2), a14 floor [rows, heads];
+// flags bit 0: the gain is [heads * vdim], not shared; f0 eps, f1 lambda, f2 factor
 GB_OP(gb_op_head_norm) {
   const int n = (int)a[10], H = (int)a[11], vdim = (int)a[12];
   if (n <= 0) return 0;
   if (vdim > 32 * HN_VR) GB_FAIL(GB_ERR_ARG, "head_norm: heads of %d values (at most %d)", vdim, 32 * HN_VR);
+  if (a[13] && (a[3] || !a[14])) GB_FAIL(GB_ERR_ARG, "head_norm: a divisor comes with a floor and without a second operand");
   const dim3 grid(gb_div_up((long long)n * H, 4)), block(128);
   if (a[8] == GB_BF16)
     gb_launch(head_norm_kernel<bf16>, grid, block, 0, ctx->stream, op_ptr<const float>(a[0]), a[1], a[2],
               op_ptr<const float>(a[3]), op_ptr<const float>(a[4]), op_ptr<const float>(a[5]), a[6], op_ptr<bf16>(a[7]), a[9],
-              n, H, vdim, (float)f[0], (float)f[1], (float)f[2]);
+              n, H, vdim, (float)f[0], (float)f[1], (float)f[2], op_ptr<const float>(a[13]), op_ptr<const float>(a[14]), flags & 1);
   else
     gb_launch(head_norm_kernel<float>, grid, block, 0, ctx->stream, op_ptr<const float>(a[0]), a[1], a[2],
               op_ptr<const float>(a[3]), op_ptr<const float>(a[4]), op_ptr<const float>(a[5]), a[6], op_ptr<float>(a[7]), a[9],
-              n, H, vdim, (float)f[0], (float)f[1], (float)f[2]);
+              n, H, vdim, (float)f[0], (float)f[1], (float)f[2], op_ptr<const float>(a[13]), op_ptr<const float>(a[14]), flags & 1);
   GB_CHECK_LAUNCH("head_norm");
   return 1;
 }

@@ -20,7 +20,7 @@ namespace {
 __global__ void causal_conv_silu_kernel(const float* in, long long ld, const float* __restrict__ taps,
                                         const float* __restrict__ bias, const float* state, long long slot_stride,
                                         const int* slot_ids, const int* tok_req, const int* q_start, float* out,
-                                        long long ldo, int n, int C, int K) {
+                                        long long ldo, int n, int C, int K, bf16* copy, long long ldcopy) {
   pdl_trigger();
   pdl_wait();
   const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -36,7 +36,37 @@ __global__ void causal_conv_silu_kernel(const float* in, long long ld, const flo
     const float v = s >= 0 ? in[(size_t)(first + s) * ld + c] : st[(size_t)(K - 1 + s) * C + c];
     acc = fmaf(taps[(size_t)c * K + j], v, acc);
   }
-  out[(size_t)t * ldo + c] = hy_silu(acc);
+  const float y = hy_silu(acc);
+  out[(size_t)t * ldo + c] = y;
+  if (copy) copy[(size_t)t * ldcopy + c] = __float2bfloat16_rn(y);
+}
+
+// A step in which every request brings one token: convolution and state in one kernel, a thread per (request, channel)
+// (the same arithmetic as in the two kernels around it).
+__global__ void causal_conv_silu_decode_kernel(const float* in, long long ld, const float* __restrict__ taps,
+                                               const float* __restrict__ bias, float* state, long long slot_stride,
+                                               const int* slot_ids, const int* q_start, float* out, long long ldo, int R,
+                                               int C, int K, bf16* copy, long long ldcopy) {
+  pdl_trigger();
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= R * C) return;
+  const int r = i / C, c = i - r * C;
+  const int t = q_start[r];
+  float* st = state + (size_t)slot_ids[r] * slot_stride + c;
+  float acc = bias ? bias[c] : 0.f;
+  const float* w = taps + (size_t)c * K;
+  pdl_wait();
+  const float now = in[(size_t)t * ld + c];
+  for (int j = 0; j < K - 1; ++j) {
+    const float v = st[(size_t)j * C];
+    acc = fmaf(w[j], v, acc);
+    if (j > 0) st[(size_t)(j - 1) * C] = v;
+  }
+  acc = fmaf(w[K - 1], now, acc);
+  if (K > 1) st[(size_t)(K - 2) * C] = now;
+  const float y = hy_silu(acc);
+  out[(size_t)t * ldo + c] = y;
+  if (copy) copy[(size_t)t * ldcopy + c] = __float2bfloat16_rn(y);
 }
 
 // one thread per (request, channel): the slot's K-1 rows become the last K-1 inputs seen
@@ -285,15 +315,24 @@ __global__ void ssm_scan_cols_kernel(const float* xbc, long long ld, const float
 
 // a0 in (f32; the convolved columns of a wider row), a1 its row stride, a2 taps [C, K], a3 bias [C] or 0, a4 conv
 // state of slot 0, a5 elements between slots, a6 slot ids, a7 token -> request, a8 first row per request, a9 rows per
-// request, a10 out (f32), a11 its row stride, a12 tokens, a13 channels, a14 taps per channel, a15 requests
+// request, a10 out (f32), a11 its row stride, a12 tokens, a13 channels, a14 taps per channel, a15 requests, a16 a
+// bfloat16 copy of out for a product that reads it, or 0, a17 its row stride
 GB_OP(gb_op_causal_conv_silu) {
   const int n = (int)a[12], C = (int)a[13], K = (int)a[14], R = (int)a[15];
   if (n <= 0) return 0;
   if (K < 1) GB_FAIL(GB_ERR_ARG, "causal_conv_silu: %d taps", K);
+  if (n == R && (long long)R * C < (1ll << 30)) {
+    gb_launch(causal_conv_silu_decode_kernel, dim3(gb_div_up((long long)R * C, 128)), dim3(128), 0, ctx->stream,
+              op_ptr<const float>(a[0]), a[1], op_ptr<const float>(a[2]), op_ptr<const float>(a[3]), op_ptr<float>(a[4]), a[5],
+              op_ptr<const int>(a[6]), op_ptr<const int>(a[8]), op_ptr<float>(a[10]), a[11], R, C, K, op_ptr<bf16>(a[16]),
+              a[17]);
+    GB_CHECK_LAUNCH("causal_conv_silu (one token each)");
+    return 1;
+  }
   gb_launch(causal_conv_silu_kernel, dim3(gb_div_up((long long)n * C, 256)), dim3(256), 0, ctx->stream,
             op_ptr<const float>(a[0]), a[1], op_ptr<const float>(a[2]), op_ptr<const float>(a[3]), op_ptr<const float>(a[4]),
             a[5], op_ptr<const int>(a[6]), op_ptr<const int>(a[7]), op_ptr<const int>(a[8]), op_ptr<float>(a[10]), a[11], n,
-            C, K);
+            C, K, op_ptr<bf16>(a[16]), a[17]);
   GB_CHECK_LAUNCH("causal_conv_silu");
   if (K == 1) return 1;
   gb_launch(conv_state_update_kernel, dim3(gb_div_up((long long)R * C, 256)), dim3(256), 0, ctx->stream,

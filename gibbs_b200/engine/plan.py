@@ -93,10 +93,12 @@ class _Run(ctypes.Structure):
 class PlanBuilder:
     """Collects operations and owns the buffers they work on.  ``cap`` is the
     largest number of tokens a step may bring.  The residual stream is
-    ``self.residual`` (float32 [cap, hidden]); a product that adds into it may
+    ``self.residual`` (float32 [cap, hidden], or wider when a token has several streams); a product that adds into it may
     leave partial sums for the next norm (the walker keeps track)."""
 
-    def __init__(self, rt, hidden: int, cap: int, max_requests: int, with_tensorcore: bool):
+    def __init__(self, rt, hidden: int, cap: int, max_requests: int, with_tensorcore: bool,
+                 residual: Optional[int] = None):
+        """``residual``: entries of a token's row of the residual stream (default: ``hidden``)."""
         self.rt, self.device, self.hidden, self.cap = rt, rt.device, int(hidden), int(cap)
         self.max_requests = int(max_requests)
         self.tc = with_tensorcore
@@ -110,7 +112,7 @@ class PlanBuilder:
         self.labels: list = []      # names under which the operations' times are added up in timing mode
         self.bt_stride = 0
         self.LOGITS, self.WANTED = sym(S_LOGITS), S_W          # what a head writes to, and how many rows
-        self.residual = self.buffer("residual", hidden, torch.float32)
+        self.residual = self.buffer("residual", residual or hidden, torch.float32)
 
     def buffer(self, name: str, width: int, dtype=None, rows: Optional[int] = None) -> torch.Tensor:
         """A [cap, width] buffer; the same name, width and dtype give the same buffer."""
@@ -375,7 +377,7 @@ def build_step_plan(model, cache, cap: int, max_requests: int) -> StepPlan:
     if len(cache.groups) > S_TABLE_STRIDE - S_BLOCK_TABLE0:
         raise NotPlannable(f"{len(cache.groups)} cache groups")
     with_tc = "tensorcore" in model.kernel_libraries()
-    b = PlanBuilder(model.rt, model.hidden_size, cap, max_requests, with_tc)
+    b = PlanBuilder(model.rt, model.hidden_size, cap, max_requests, with_tc, residual=model.residual_size)
     b.bt_stride = sym(S_TABLE_STRIDE)          # a step packs only as many table columns as its longest context needs
     views = cache.views([TableRef(g) for g in range(len(cache.groups))], SlotRef(), [])
     model.plan_ops(b, views)

@@ -210,3 +210,58 @@ class ParallelResidual(Block):
 
 
 register_part("block", "parallel_residual", ParallelResidual)
+
+
+class HyperResidual(Block):
+    """Pre-norm sublayers over several residual streams (``parts.streams``): a sublayer reads a weighted sum of the
+    streams through its norm, and its ``branch_sum`` part (a ``hyper_connection``) mixes the streams and spreads the
+    output over them.  The feed-forward is optional.
+
+    What the next sublayer reads, in this layer or in the one that runs next (``hands_over``), is taken in the kernel
+    that mixes the streams."""
+    ROLES = (("mixer_norm", "norm"), ("mixer", "mixer"), ("mixer_streams", "branch_sum"), ("ffn_norm", "norm"),
+             ("ffn", "feed_forward"), ("ffn_streams", "branch_sum"))
+    OPTIONAL_ROLES = ("ffn_norm", "ffn", "ffn_streams")
+
+    def __init__(self, parts, rt, params=None):
+        super().__init__(parts, rt, params)
+        have = set(self.parts)
+        if len(have & set(self.OPTIONAL_ROLES)) not in (0, 3):
+            raise ValueError("a feed-forward comes with a norm and a mixing of the streams of its own")
+        for role in ("mixer", "ffn"):
+            if role in have and not getattr(self.parts[role], "writes_branch", False):
+                raise ValueError(f"the {role} of this arrangement must be able to write its output; "
+                                 f"{type(self.parts[role]).__name__} only adds into the stream")
+        self._next = None          # the block that runs next, when what it reads is taken here
+        self._handed = None        # the normed rows the block in front left for this one
+
+    def hands_over(self, following) -> bool:
+        if (FUSE_NEXT_NORM and isinstance(following, HyperResidual)
+                and following.mixer_streams.streams == self.mixer_streams.streams):
+            self._next = following
+            return True
+        return False
+
+    def _run(self, rn, x, caches):
+        h, self._handed = self._handed, None
+        if h is None:
+            h = self.mixer_streams.read(rn, x, self.mixer_norm)
+        y = rn.buffer("branch", self.mixer_streams.dim, torch.float32)
+        behind = None if self._next is None else (self._next.mixer_streams, self._next.mixer_norm)
+        has_ffn = "ffn" in self.parts
+        self.mixer.run(rn, h, y, self.caches_of("mixer", caches))
+        h = self.mixer_streams.add(rn, x, y, then=(self.ffn_streams, self.ffn_norm) if has_ffn else behind)
+        if has_ffn:
+            self.ffn.run(rn, h, y, None)
+            h = self.ffn_streams.add(rn, x, y, then=behind)
+        if self._next is not None:
+            self._next._handed = h
+
+    def forward(self, x, step, caches):
+        self._run(Eager(self.rt, step), stream_tensor(x), caches)
+
+    def plan_ops(self, plan, caches):
+        self._run(Planned(plan), plan.residual, caches)
+
+
+register_part("block", "hyper_residual", HyperResidual)

@@ -1,6 +1,7 @@
 """Token embedding and the output head."""
 from __future__ import annotations
 
+import numpy as np
 import torch
 
 from .. import ops
@@ -47,6 +48,38 @@ class TokenEmbedding(Part):
         else:
             rn = Planned(plan)
             self._scaled(rn, rn.token_ids, plan.residual)
+
+
+class PositionedEmbedding(TokenEmbedding):
+    """x[t, :] = table[id_t, :] * scale + a sinusoidal vector of the token's position p: entry 2i is
+    sin(p * base^(-2i / dim)), entry 2i + 1 the cosine of the same angle (32-bit; frequencies rounded once from
+    64-bit).  ``copies``: the row stands that many times side by side (several residual streams that start equal)."""
+    needs_step = True
+
+    def __init__(self, params, tensors, rt):
+        super().__init__(params, tensors, rt)
+        self.copies = int(params.get("copies", 1))
+        i = np.arange((self.dim + 1) // 2, dtype=np.float64)
+        freq = np.power(float(params.get("base", 10000.0)), -2.0 * i / self.dim)
+        self.freq = torch.from_numpy(freq.astype(np.float32)).to(rt.device)
+
+    def kernel_libraries(self):
+        return ("core", hybrid.LIBRARY)
+
+    def _run(self, rn, out: torch.Tensor) -> None:
+        rn.op("embed_scaled", [keep(rn, self.table), ops.dtype_code(self.table.dtype), rn.token_ids, out.data_ptr(), rn.N,
+                               self.dim, self.vocab, 0, 0, 0, 0, 0, rn.tok_pos, 0, 0, 0, 0, 0, self.copies,
+                               keep(rn, self.freq)], [self.scale], label="embed_positions")
+
+    def forward(self, ids: torch.Tensor, step=None) -> torch.Tensor:
+        if step is None:
+            raise ValueError("an embedding that adds position vectors needs the step")
+        out = self.rt.empty(ids.numel(), self.copies * self.dim, dtype=torch.float32)
+        self._run(Eager(self.rt, step), out)
+        return out
+
+    def plan_ops(self, plan):
+        self._run(Planned(plan), plan.residual)
 
 
 class PairEmbedding(TokenEmbedding):
@@ -131,5 +164,6 @@ class LMHead(Part):
 
 
 register_part("embedding", "token_embedding", TokenEmbedding)
+register_part("embedding", "positioned_embedding", PositionedEmbedding)
 register_part("embedding", "pair_embedding", PairEmbedding)
 register_part("head", "lm_head", LMHead)

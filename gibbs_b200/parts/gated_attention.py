@@ -20,7 +20,12 @@ rot_dims / 2) instead of "adjacent"; ``rot_factor`` (every frequency is divided
 by it: positions stretched linearly); ``qk_norm`` "head_after_rot": q and k are
 turned first and every head is then divided by its root mean square over
 ``dim`` (no gain); ``keep_first`` n with a window: position i also sees every
-j < n (at their true positions), and the pages of those positions stay.  With ``shares_kv`` the layer has no key/value projections and reads the
+j < n (at their true positions), and the pages of those positions stay;
+``qk_norm`` "head": every head of q and k is normed over ``dim`` with a gain
+shared by the heads (before the rotation); ``q_temp`` {coef, every}: the query
+at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1);
+``weights`` "sigmoid": no softmax, p_j = sigmoid(s_j + pb_h) with a number per
+head (tensor ``pb``), not normalised over keys.  With ``shares_kv`` the layer has no key/value projections and reads the
 pages another entry of the model's order writes (keys as that entry stored
 them: normed and rotated); its window is its own.  ``retain`` is what the pages
 keep for the layers that read them (their widest window; None: everything).
@@ -65,21 +70,24 @@ class GatedAttention(Mixer):
         d, H, G = params["hidden"], params["heads"], params["kv_heads"]
         dim, vdim = params["dim"], params["vdim"]
         shares, whole = params.get("shares_kv", False), params.get("qk_norm") == "whole"
+        per_head = params.get("qk_norm") == "head"
         t = {"q": TensorDecl.of(H * dim, d), "o": TensorDecl.of(d, H * vdim)}
-        if whole:
-            t["q.norm"] = TensorDecl.of(H * dim, role=VECTOR)
+        if whole or per_head:
+            t["q.norm"] = TensorDecl.of(H * dim if whole else dim, role=VECTOR)
         if params.get("gate", True):
             t["g"] = TensorDecl.of(H * vdim, d)
         if not shares:
             t["k"], t["v"] = TensorDecl.of(G * dim, d), TensorDecl.of(G * vdim, d)
-            if whole:
-                t["k.norm"] = TensorDecl.of(G * dim, role=VECTOR)
+            if whole or per_head:
+                t["k.norm"] = TensorDecl.of(G * dim if whole else dim, role=VECTOR)
         if params.get("bias", False):
             t["q.b"] = TensorDecl.of(H * dim, role=VECTOR)
             if not shares:
                 t["k.b"], t["v.b"] = TensorDecl.of(G * dim, role=VECTOR), TensorDecl.of(G * vdim, role=VECTOR)
         if params.get("sink") == "learned":
             t["sink"] = TensorDecl.of(H, role=VECTOR)
+        if params.get("weights") == "sigmoid":
+            t["pb"] = TensorDecl.of(H, role=VECTOR)
         return t
 
     def __init__(self, params, tensors, rt):
@@ -98,11 +106,20 @@ class GatedAttention(Mixer):
         self.keep_first = int(p.get("keep_first") or 0) if self.window else 0
         if self.keep_first < 0:
             raise ValueError(f"{self.keep_first} kept first positions")
-        self.whole_norm = p.get("qk_norm") == "whole"
+        self.whole_norm, self.head_norm = p.get("qk_norm") == "whole", p.get("qk_norm") == "head"
         self.norm_after_rot = p.get("qk_norm") == "head_after_rot"
-        if p.get("qk_norm") not in (None, "whole", "head_after_rot"):
-            raise ValueError(f"qk_norm '{p.get('qk_norm')}': this mixer norms the whole projection, every head behind "
-                             "the rotation, or nothing")
+        if p.get("qk_norm") not in (None, "whole", "head", "head_after_rot"):
+            raise ValueError(f"qk_norm '{p.get('qk_norm')}': this mixer norms the whole projection, every head before or "
+                             "behind the rotation, or nothing")
+        if p.get("weights", "softmax") not in ("softmax", "sigmoid"):
+            raise ValueError(f"weights '{p['weights']}': a softmax over the visible keys, or a sigmoid of each score")
+        self.sigmoid = p.get("weights") == "sigmoid"
+        self.score_bias = tensors["pb"].to(torch.float32).contiguous() if self.sigmoid else None
+        if self.sigmoid and (self.sink or self.keep_first):
+            raise ValueError("weights that are not normalised over keys come without a sink and without kept first positions")
+        self.takes_factor = self.sigmoid           # (``mix_heads`` can multiply its output by a factor)
+        temp = p.get("q_temp") or {}
+        self.temp_coef, self.temp_every = float(temp.get("coef", 0.0)), float(temp.get("every", 0.0))
         self.rot_halves = {"adjacent": False, "halves": True}[p.get("rot_pairs", "adjacent")]
         self.shares_kv = bool(p.get("shares_kv", False))
         self.rot_dims = int(p.get("rot_dims", 0) or 0)
@@ -122,7 +139,8 @@ class GatedAttention(Mixer):
         self.gate_col = H * dim if self.shares_kv else self.v_col + G * vdim
         f32 = lambda n: tensors[n].to(torch.float32).contiguous() if n in tensors else None
         self.q_gain, self.k_gain = f32("q.norm"), f32("k.norm")
-        self.out_proj = Linear(tensors["o"], None, rt)
+        self.out_weight, self.heads_width = tensors["o"].contiguous(), H * vdim
+        self.out_proj = Linear(self.out_weight, None, rt)
         i = np.arange(self.rot_dims // 2, dtype=np.float64)
         inv = np.power(float(p.get("rot_base", 10000.0)), -2.0 * i / max(self.rot_dims, 1)) / float(p.get("rot_factor") or 1.0)
         self.inv_freq = torch.from_numpy(np.concatenate([inv, [0.0]]).astype(np.float32)).to(rt.device)
@@ -144,7 +162,11 @@ class GatedAttention(Mixer):
                 pairs += full * self.keep_first + (far - full) * (far - full + 1) // 2
         return 2 * self.heads * (self.dim + self.vdim) * pairs
 
-    def _attend(self, rn: Runner, fused: torch.Tensor, kv) -> torch.Tensor:
+    def mix_heads(self, rn: Runner, u: torch.Tensor, caches, out: torch.Tensor, factor: float = 1.0) -> None:
+        """Between the products, for a mixer beside others (``parts.parallel_mixers``)."""
+        self._attend(rn, u, caches[0], out, factor)
+
+    def _attend(self, rn: Runner, fused: torch.Tensor, kv, out: torch.Tensor = None, factor: float = 1.0) -> torch.Tensor:
         """Everything between the two products: fused [rows, q | k | v | gate] (float32) -> heads' outputs."""
         H, G, dim, vdim = self.heads, self.kv_heads, self.dim, self.vdim
         if not self.shares_kv and not kv.writable:
@@ -167,23 +189,29 @@ class GatedAttention(Mixer):
         rn.op("qk_prep", [fused.data_ptr(), fused.stride(0), self.k_col, self.v_col, keep(rn, self.q_gain),
                           keep(rn, self.k_gain), keep(rn, self.inv_freq), self.rot_dims, rn.tok_req, rn.tok_pos, table,
                           bt_stride, kv.page_size, keep(rn, kp) if write else 0, keep(rn, vp) if write else 0,
-                          kp.shape[0], rn.N, H, G, dim, vdim, q.data_ptr()], [self.eps],
-              flags=(1 if self.whole_norm else 0) | (2 if tc else 0) | (4 if pages_bf16 else 0) |
+                          kp.shape[0], rn.N, H, G, dim, vdim, q.data_ptr()],
+              [self.eps, self.temp_coef, self.temp_every],
+              flags=(1 if self.whole_norm else 0) | (8 if self.head_norm else 0) | (2 if tc else 0) | (4 if pages_bf16 else 0) |
                     (16 if self.rot_halves else 0) | (32 if self.norm_after_rot else 0))
-        out = rn.buffer("ga_heads_out", H * vdim)
+        if out is None:
+            out = rn.buffer("ga_heads_out", H * vdim)
+        if factor != 1.0 and not self.sigmoid:
+            raise ValueError("a factor on the heads' outputs is taken by unnormalised weights only")
+        # (unnormalised weights: an operation of their own, whose last constant is the factor on the output)
+        op, per_head, last = ("sigmoid_attention", self.score_bias, factor) if self.sigmoid else \
+            ("sink_attention", self.sink_scores, self.keep_first)
         ws = rn.buffer("ga_partial", vdim + 2, torch.float32, fixed_rows=_workspace_rows())
         gate = fused.data_ptr() + 4 * self.gate_col if self.gated else 0
         if tc:
-            rn.op("sink_attention_tc", [q.data_ptr(), keep(rn, kp), keep(rn, vp), table, bt_stride, kv.page_size,
-                                        kp.shape[0], rn.tok_req, rn.tok_pos, gate, fused.stride(0), out.data_ptr(),
-                                        out.stride(0), rn.N, H, G, dim, vdim, self.window or 0, rn.max_context,
-                                        ws.data_ptr(), rn.R, rn.q_start, keep(rn, self.sink_scores)],
-                  [self.scale, self.softcap, self.keep_first], label="sink_attention", flags=1 if self.sink else 0)
+            rn.op(op + "_tc", [q.data_ptr(), keep(rn, kp), keep(rn, vp), table, bt_stride, kv.page_size, kp.shape[0],
+                               rn.tok_req, rn.tok_pos, gate, fused.stride(0), out.data_ptr(), out.stride(0), rn.N, H, G, dim,
+                               vdim, self.window or 0, rn.max_context, ws.data_ptr(), rn.R, rn.q_start, keep(rn, per_head)],
+                  [self.scale, self.softcap, last], label=op, flags=1 if self.sink else 0)
             return out
-        rn.op("sink_attention", [q.data_ptr(), keep(rn, kp), keep(rn, vp), table, bt_stride, kv.page_size, kp.shape[0],
-                                 rn.tok_req, rn.tok_pos, gate, fused.stride(0), out.data_ptr(), out.stride(0), rn.N, H, G,
-                                 dim, vdim, self.window or 0, rn.max_context, ws.data_ptr(), 1, keep(rn, self.sink_scores)],
-              [self.scale, self.softcap, self.keep_first],
+        rn.op(op, [q.data_ptr(), keep(rn, kp), keep(rn, vp), table, bt_stride, kv.page_size, kp.shape[0], rn.tok_req,
+                   rn.tok_pos, gate, fused.stride(0), out.data_ptr(), out.stride(0), rn.N, H, G, dim, vdim, self.window or 0,
+                   rn.max_context, ws.data_ptr(), 1, keep(rn, per_head)],
+              [self.scale, self.softcap, last],
               flags=(1 if self.sink else 0) | (4 if pages_bf16 else 0) | (8 if out.dtype == torch.bfloat16 else 0))
         return out
 

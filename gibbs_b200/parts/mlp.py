@@ -2,7 +2,7 @@
 (``dense_mlp``), and with one, out = W_down (act(W_gate h) * (W_up h)) (``gated_mlp``).
 
 ``act`` is one of "gelu" (the exact one, with erf), "gelu_tanh", "silu",
-"relu".  The first product writes 32-bit values, the function (and the gate's
+"relu", "relu2" (the square of relu).  The first product writes 32-bit values, the function (and the gate's
 product with the up rows) is taken in 32-bit and rounded to the compute dtype
 for the second product, which adds into the residual stream or writes for an
 arrangement that takes the output as it is.
@@ -17,7 +17,7 @@ from .base import FeedForward, TensorDecl, VECTOR, register_part
 from .linear import can_fuse_swiglu, interleave_gate_up
 from .runner import BranchPart, Runner
 
-ACTIVATIONS = {"gelu": 0, "gelu_tanh": 1, "silu": 2, "relu": 3}
+ACTIVATIONS = {"gelu": 0, "gelu_tanh": 1, "silu": 2, "relu": 3, "relu2": 4, "none": 5}
 # act(g) = g * sigmoid(alpha * (g + cubic * g^3)) for the functions that have this form: (alpha, cubic).  The tanh form
 # of gelu has it because 0.5 (1 + tanh y) = sigmoid(2 y), with y = sqrt(2 / pi) (g + 0.044715 g^3).
 SIGMOID_FORMS = {"silu": (1.0, 0.0), "gelu_tanh": (1.5957691216057308, 0.044715)}

@@ -26,6 +26,8 @@ class CausalLM:
         self.plan, self.rt = plan, rt
         self.embedding, self.blocks, self.final_norm, self.head = embedding, blocks, final_norm, head
         self.vocab_size, self.hidden_size = plan.vocab_size, plan.hidden_size
+        # entries of a token's row of the residual stream: its streams lie side by side
+        self.residual_size = plan.hidden_size * plan.streams
         # neighbours in the order may share a kernel across their border (the norm in front of the next layer taken
         # by the kernel that completes this one's residual sum): a block that can says so with ``hands_over``.  Only
         # for layers that run once, so that "the block behind" is one block.
@@ -59,6 +61,8 @@ class CausalLM:
         32-bit logits of the wanted rows, [n_want, vocab], or None."""
         if getattr(self.embedding, "cache_needs", None) is not None:
             x = Residual(self.embedding.forward(step.token_ids, step, caches[len(self.plan.order)]))
+        elif getattr(self.embedding, "needs_step", False):
+            x = Residual(self.embedding.forward(step.token_ids, step))
         else:
             x = Residual(self.embedding.forward(step.token_ids))
         for e, entry in enumerate(self.plan.order):
