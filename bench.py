@@ -138,6 +138,29 @@ def selivik_shape(size: str) -> dict:
             "embedding": {"scale": 8.0}, "layers": [{"type": k, "mixer": m, "mlp": f} for k, m, f in four * 2]}
 
 
+def guvetar_shape(size: str) -> dict:
+    """Layer sizes that resemble a real model's, for the Guvetar design: four residual streams; selective scans in turn
+    with a matrix memory and with sigmoid attention beside a gated linear recurrence; a dense feed-forward behind each."""
+    if size == "1k":
+        d, vocab = 1024, 32768
+        scan = {"inner": 2048, "state": 16, "dt_rank": 64, "conv": 4}
+        memory = {"heads": 8, "dim": 64, "vdim": 128, "gate_cap": 15.0}
+        left = {"heads": 8, "kv_heads": 2, "dim": 64, "vdim": 64, "scale": 0.125}
+        right = {"heads": 8, "dim": 64, "vdim": 64}
+    else:
+        d, vocab = 2048, 65536
+        scan = {"inner": 4096, "state": 16, "dt_rank": 128, "conv": 4}
+        memory = {"heads": 16, "dim": 128, "vdim": 128, "gate_cap": 15.0}
+        left = {"heads": 16, "kv_heads": 4, "dim": 64, "vdim": 64, "scale": 0.125}
+        right = {"heads": 8, "dim": 128, "vdim": 128}
+    left["q_temp"] = {"coef": 0.5, "every": 1024}
+    both = {"left": left, "right": right, "left_scale": 0.7, "right_scale": 0.8}
+    mlp = {"kind": "dense", "ff": 4 * d}
+    four = [("mamba1", scan), ("parallel", both), ("mamba1", scan), ("mlstm", memory)]
+    return {"architecture": "Guvetar", "vocab": vocab, "width": d, "streams": 4, "norm": {"eps": 1e-6},
+            "layers": [{"type": k, "mixer": m, "mlp": mlp} for k, m in four * 2]}
+
+
 def potivik_workload(a):
     """Prompt and decode throughput of the Potivik design at two sizes (random weights), beside an LFM2
     model of equal width, depth and feed-forward width, with the time per kind of operation of one
@@ -147,7 +170,8 @@ def potivik_workload(a):
     beside an LFM2 model and a Potivik model (state-space and latent-attention layers in turn) of equal width,
     depth and feed-forward width.  'selivik': the Selivik design beside an LFM2 model, a Petelix model (windowed
     attention with a sink and routed experts) and a Potivik model (latent attention with a rotated part) of equal
-    width and depth."""
+    width and depth.  'guvetar': the Guvetar design beside an LFM2 model, a Sisadra model (a delta rule, attention on the
+    same tensor-core kernel, a dense feed-forward: the closest design) and a Potivik model (a state-space scan)."""
     import torch
     from gibbs_b200 import Engine, Lfm2Config, parse_config, random_model
     from gibbs_b200.engine import benchmark as B
@@ -166,8 +190,8 @@ def potivik_workload(a):
             twin = dict(LFM2_1P2B, hidden_size=d, num_hidden_layers=8, num_attention_heads=d // 64, num_key_value_heads=d // 256,
                         head_dim=64, vocab_size=pot["vocab"], intermediate_size=4 * d, block_auto_adjust_ff_dim=False,
                         full_attn_idxs=[1, 3, 5, 7], max_position_embeddings=4096)
-        elif a.workload == "selivik":
-            pot = selivik_shape(size)
+        elif a.workload in ("selivik", "guvetar"):
+            pot = selivik_shape(size) if a.workload == "selivik" else guvetar_shape(size)
             d = pot["width"]
             twin = dict(LFM2_1P2B, hidden_size=d, num_hidden_layers=8, num_attention_heads=d // 64, num_key_value_heads=d // 256,
                         head_dim=64, vocab_size=pot["vocab"], intermediate_size=4 * d, block_auto_adjust_ff_dim=False,
@@ -181,10 +205,13 @@ def potivik_workload(a):
         models = [(pot["architecture"], parse_config(pot)), ("LFM2 of equal size", Lfm2Config.from_dict(twin))]
         if a.workload == "sisadra":
             models.append(("Potivik of equal size", parse_config(potivik_shape(size))))
+        if a.workload == "guvetar":
+            models.append(("Sisadra of equal size", parse_config(sisadra_shape(size))))
+            models.append(("Potivik of equal size", parse_config(potivik_shape(size))))
         if a.workload == "selivik":
             models.append(("Petelix of equal size", parse_config(petelix_shape(size))))
             models.append(("Potivik of equal size", parse_config(potivik_shape(size))))
-        for name, conf in models:
+        for name, conf in models[:1] if a.no_twins else models:
             model = random_model(conf, SEED, dtype="bfloat16", device="cuda:0", stored_dtype=torch.bfloat16)
             eng = Engine(model, n_pages=(batch + 1) * (4096 // 16), page_size=16, max_requests=batch, max_step_tokens=prompt,
                          max_context=4096)
@@ -275,10 +302,11 @@ def main():
                     help="float32: the engine's true 32-bit twin on the same (bfloat16-rounded) weights; "
                          "with --only prefill or --only decode (the benchmark line itself is bfloat16)")
     ap.add_argument("--skip-points", action="store_true", help="skip batch 1 and 64")
-    ap.add_argument("--workload", choices=["serve700m", "long2p6b", "sweep", "potivik", "petelix", "sisadra", "selivik"], default=None,
+    ap.add_argument("--workload", choices=["serve700m", "long2p6b", "sweep", "potivik", "petelix", "sisadra", "selivik", "guvetar"], default=None,
                     help="run one of the other workloads instead (prints its own JSON lines); 'potivik' / 'petelix' / "
-                         "'sisadra' / 'selivik': that design at layer sizes of a real model, beside an LFM2 model of equal size")
-    ap.add_argument("--size", default=None, help="with --workload potivik, petelix, sisadra or selivik: '1k', '2k' or both with a comma (default both)")
+                         "'sisadra' / 'selivik' / 'guvetar': that design at layer sizes of a real model, beside an LFM2 model of equal size")
+    ap.add_argument("--size", default=None, help="with --workload potivik, petelix, sisadra, selivik or guvetar: '1k', '2k' or both with a comma (default both)")
+    ap.add_argument("--no-twins", action="store_true", help="with such a workload: the design alone, without the models beside it")
     ap.add_argument("--prompt-tokens", type=int, default=None,
                     help="with --only prefill / prefill-timeline / products: another prompt length than 2,048")
     ap.add_argument("--only", default=None,
@@ -301,7 +329,7 @@ def main():
     from gibbs_b200 import Generator, Lfm2Config, random_model
     from gibbs_b200.engine import benchmark as B
 
-    if a.workload in ("potivik", "petelix", "sisadra", "selivik"):
+    if a.workload in ("potivik", "petelix", "sisadra", "selivik", "guvetar"):
         return potivik_workload(a)
     if a.workload:
         return other_workload(a)

@@ -67,6 +67,7 @@ class GatedWriteRecurrence(RecurrentHeads):
 
     def __init__(self, params, tensors, rt):
         super().__init__(params, tensors, rt)
+        self.hidden = int(params["hidden"])
         self.H, self.dim, self.vdim = int(params["heads"]), int(params["dim"]), int(params["vdim"])
         self.eps = float(params["eps"])
         self.heads_width = self.H * self.vdim
@@ -105,6 +106,7 @@ class MatrixMemory(RecurrentHeads):
 
     def __init__(self, params, tensors, rt):
         super().__init__(params, tensors, rt)
+        self.hidden = int(params["hidden"])
         self.H, self.dim, self.vdim = int(params["heads"]), int(params["dim"]), int(params["vdim"])
         self.eps, self.cap = float(params["eps"]), float(params["gate_cap"])
         self.div_eps = float(params.get("div_eps", 1e-6))

@@ -32,7 +32,7 @@ class ParallelMixers(BranchPart, Mixer):
 
     def __init__(self, params, tensors, rt):
         super().__init__(params, tensors, rt)
-        self.sides, self.factors = [], []
+        self.hidden, self.sides, self.factors = int(params["hidden"]), [], []
         for side in params["sides"]:
             name = side["name"] + "."
             part = part_class("mixer", side["kind"])(side["params"], {k[len(name):]: v for k, v in tensors.items()

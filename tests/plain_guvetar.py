@@ -7,11 +7,31 @@ a time and whole: position t sees what the design lets it see of positions 0..t.
 """
 from __future__ import annotations
 
+import contextlib
 import math
 
 import torch
 
 F64 = torch.float64
+
+
+_GRID = 0.0
+
+
+@contextlib.contextmanager
+def rounded_rows(grid=1.0):
+    """Inside: what enters a matrix product, and an attention's queries, keys and values, is rounded to bfloat16 (times
+    ``grid``: another grid of the same fineness).  How far the results move tells how much rounding alone moves them."""
+    global _GRID
+    _GRID = grid
+    try:
+        yield
+    finally:
+        _GRID = 0.0
+
+
+def rows(x):
+    return (x * _GRID).to(torch.bfloat16).to(F64) / _GRID if _GRID else x
 
 
 def rms(x, eps):
@@ -26,7 +46,7 @@ def silu(x):
 def sinusoids(T, width):
     """[T, width]: entry 2i is sin(p * 10000^(-2i/width)), entry 2i + 1 the cosine of the same angle."""
     e = torch.arange(width)
-    ang = torch.arange(T, dtype=F64)[:, None] * torch.pow(torch.tensor(10000.0, dtype=F64), -(2.0 * (e // 2)) / width)[None, :]
+    ang = torch.arange(T, dtype=F64)[:, None] * torch.pow(torch.tensor(10000.0, dtype=F64), -(2 * (e // 2)).to(F64) / width)[None, :]
     return torch.where(e % 2 == 0, torch.sin(ang), torch.cos(ang))
 
 
@@ -68,13 +88,14 @@ def selective_scan(x, dt, A, B, C, D):
 
 def mamba1(h, w, m, eps):
     inner, rank, n = m["inner"], m["dt_rank"], m["state"]
+    h = rows(h)
     u = h @ w["in"].T
     x, z = u[:, :inner], u[:, inner:]
     x = silu(causal_conv(x, w["conv"], w["conv.b"]))
-    p = x @ w["x"].T
-    dt = torch.nn.functional.softplus(p[:, :rank] @ w["dt"].T + w["dt.b"])
+    p = rows(x) @ w["x"].T
+    dt = torch.nn.functional.softplus(rows(p[:, :rank]) @ w["dt"].T + w["dt.b"])
     y = selective_scan(x, dt, -torch.exp(w["A_log"]), p[:, rank:rank + n], p[:, rank + n:], w["D"])
-    return (y * silu(z)) @ w["o"].T
+    return rows(y * silu(z)) @ w["o"].T
 
 
 def query_temperature(T, coef, every):
@@ -92,17 +113,19 @@ def sigmoid_weights(scores):
 def sigmoid_attention(h, w, m, eps):
     T = h.shape[0]
     H, G, dim, vdim = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    h = rows(h)
     q = rms((h @ w["q"].T).reshape(T, H, dim), eps) * w["q.norm"]
     k = rms((h @ w["k"].T).reshape(T, G, dim), eps) * w["k.norm"]
     v = (h @ w["v"].T).reshape(T, G, vdim)
     t = m.get("q_temp")
     if t:
         q = q * query_temperature(T, float(t["coef"]), float(t["every"]))[:, None, None]
+    q, k, v = rows(q), rows(k), rows(v)
     out = torch.zeros(T, H, vdim, dtype=F64)
     for hd in range(H):
         g = hd // (H // G)
         out[:, hd] = sigmoid_weights((q[:, hd] @ k[:, g].T) * m["scale"] + w["pb"][hd]) @ v[:, g]
-    return out.reshape(T, H * vdim) @ w["o"].T
+    return rows(out.reshape(T, H * vdim)) @ w["o"].T
 
 
 def gated_write_recurrence(q, f, v):
@@ -118,11 +141,12 @@ def gated_write_recurrence(q, f, v):
 def hgrn2(h, w, m, eps):
     T = h.shape[0]
     H, dim, vdim = m["heads"], m["dim"], m["vdim"]
+    h = rows(h)
     q = silu(h @ w["q"].T).reshape(T, H, dim)
     f = (w["lower"] + (1.0 - w["lower"]) * torch.sigmoid(h @ w["f"].T + w["f.b"])).reshape(T, H, dim)
     v = (h @ w["v"].T).reshape(T, H, vdim)
     out = torch.stack([gated_write_recurrence(q[:, n], f[:, n], v[:, n]) for n in range(H)], 1)
-    return (rms(out, eps) * w["norm"]).reshape(T, H * vdim) @ w["o"].T
+    return rows((rms(out, eps) * w["norm"]).reshape(T, H * vdim)) @ w["o"].T
 
 
 def parallel(h, w, m, eps):
@@ -150,6 +174,7 @@ def matrix_memory(q, k, v, i, f):
 def mlstm(h, w, m, eps):
     T = h.shape[0]
     H, dim, vdim, cap = m["heads"], m["dim"], m["vdim"], float(m["gate_cap"])
+    h = rows(h)
     q = (h @ w["q"].T).reshape(T, H, dim) * dim ** -0.5
     k = (h @ w["k"].T).reshape(T, H, dim)
     v = (h @ w["v"].T).reshape(T, H, vdim)
@@ -157,14 +182,14 @@ def mlstm(h, w, m, eps):
     f = torch.nn.functional.logsigmoid(cap * torch.tanh((h @ w["f"].T + w["f.b"]) / cap))
     out = torch.stack([matrix_memory(q[:, n], k[:, n], v[:, n], i[:, n], f[:, n]) for n in range(H)], 1)
     out = rms(out, eps).reshape(T, H * vdim) * w["norm"]
-    return (out * torch.sigmoid(h @ w["g"].T)) @ w["o"].T
+    return rows(out * torch.sigmoid(h @ w["g"].T)) @ w["o"].T
 
 
 MIXERS = {"mamba1": mamba1, "parallel": parallel, "mlstm": mlstm}
 
 
 def dense_mlp(h, w):
-    return torch.square(torch.relu(h @ w["up"].T)) @ w["down"].T
+    return rows(torch.square(torch.relu(rows(h) @ w["up"].T))) @ w["down"].T
 
 
 def sub(tensors, prefix):
@@ -192,4 +217,4 @@ def forward(cfg, tensors, tokens, want=None, layers_out=None):
     x = rms(streams.sum(0), eps) * tensors["final.norm"].to(F64)
     if want is not None:
         x = x[torch.as_tensor(want, dtype=torch.long)]
-    return x @ table.T
+    return rows(x) @ table.T
