@@ -104,8 +104,9 @@ __global__ void __launch_bounds__(TC_THREADS, (DK + DV <= 128) ? 4 : 2) sink_att
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int group = p.H / p.G, tpt = p.tokens_per_tile;
   const int g = blockIdx.y / p.maps, mp = blockIdx.y - g * p.maps;      // kv head and map
-  // this CTA's request and first token: the tiles of the step's requests, one request after the other
-  int tile = blockIdx.x, t0 = -1, n_tok = 0;
+  // this CTA's request and first token: the tiles of the step's requests, one request after the other, taken from the
+  // last to the first (a prompt's last tiles see the most keys: they start first)
+  int tile = gridDim.x - 1 - blockIdx.x, t0 = -1, n_tok = 0;
   for (int r = 0; r < p.R; ++r) {
     const int qs = p.q_start[r], qe = r + 1 < p.R ? p.q_start[r + 1] : p.N;
     const int tiles = (qe - qs + tpt - 1) / tpt;

@@ -31,9 +31,16 @@ struct GbPlanCtx {
   const float* pend;         // [pend_splits][tokens * residual_ld] sums a product left to be added
   int pend_splits;
   const float* pend_bias;    // [residual_ld] or null
+  // for a record whose flags have GB_OP_TAKES_PARTIALS (null / 0 otherwise, and when the product in front did not split
+  // its sums): the partial tiles [part_splits][rows][columns] of the 32-bit output of the product recorded directly in
+  // front, which was told to leave them; its output was then not written, and is their sum in this order (+ part_bias)
+  const float* part;
+  int part_splits;
+  const float* part_bias;
 };
 
 #define GB_OP_TAKES_PENDING (1 << 30)
+#define GB_OP_TAKES_PARTIALS (1 << 29)
 #define GB_OP_PENDING_MIN_ROWS 64
 
 typedef int (*GbPlanOpFn)(const GbPlanCtx* ctx, const long long* a, const double* f, int flags);

@@ -86,7 +86,18 @@ struct GemmParams {
   // g' * sigmoid(alpha * (g' + cubic * g'^3)) * u'.  SwiGLU is alpha 1, no limit (infinity), add 0, cubic 0; the tanh
   // form of gelu as the gate's function is alpha 2 sqrt(2 / pi), cubic 0.044715 (0.5 (1 + tanh y) = sigmoid(2 y)).
   float glu_alpha, glu_limit, glu_add, glu_cubic;
+  int act;                      // of mode OUT_BF16: applied to the 32-bit sum before it is rounded (Act)
 };
+
+// The function of a feed-forward without a gate, in the epilogue of its first product.
+enum Act : int { ACT_NONE = 0, ACT_RELU2 = 1 };
+__device__ __forceinline__ float apply_act(int act, float v) {
+  if (act == ACT_RELU2) {
+    v = fmaxf(v, 0.f);
+    v *= v;
+  }
+  return v;
+}
 
 __device__ __forceinline__ float glu_exact(float alpha, float limit, float add, float cubic, float g, float u) {
   g = fminf(g, limit);
@@ -106,7 +117,7 @@ __device__ __forceinline__ void epilogue_barrier() { asm volatile("bar.sync 1, 1
 // Applies the epilogue to one finished value D[n][m] (n: weight row) and stores it.
 __device__ __forceinline__ void store_value(const GemmParams& p, int m, int n, float val) {
   if (p.mode == OUT_BF16) {
-    ((bf16*)p.out)[(size_t)m * p.ldo + n] = __float2bfloat16_rn(val);
+    ((bf16*)p.out)[(size_t)m * p.ldo + n] = __float2bfloat16_rn(apply_act(p.act, val));
   } else if (p.mode == OUT_F32) {
     ((float*)p.out)[(size_t)m * p.ldo + n] = val;
   } else {
@@ -363,7 +374,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant
           float v[16];
           tmem_ld_16(tmem_base + ((uint32_t)(32 * q) << 16) + (uint32_t)c0, v);
 #pragma unroll
-          for (int j = 0; j < 16; ++j) ob[(c0 + j) * BM + row] = __float2bfloat16_rn(v[j] + b);
+          for (int j = 0; j < 16; ++j) ob[(c0 + j) * BM + row] = __float2bfloat16_rn(apply_act(p.act, v[j] + b));
         }
         epilogue_barrier();
         bf16* dst = (bf16*)p.out + (size_t)m0 * p.ldo + n0;
@@ -760,7 +771,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
             tmem_ld_32(acc + (uint32_t)(h0 + c0), v);
 #pragma unroll
             for (int j = 0; j < 32; ++j)
-              if (c0 + j < hc) ob[(c0 + j) * BM + row] = __float2bfloat16_rn(v[j] + b);
+              if (c0 + j < hc) ob[(c0 + j) * BM + row] = __float2bfloat16_rn(apply_act(p.act, v[j] + b));
           }
           tc_fence_before();
           epilogue_barrier();
@@ -895,7 +906,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
 // out = epilogue(sum over splits of the partial tiles (+ bias)), in split order.
 __global__ void splitk_reduce_kernel(const float* ws, int splits, const float* __restrict__ bias,
                                      void* __restrict__ out, long long ldo, int mode, int M, int N, float glu_alpha,
-                                     float glu_limit, float glu_add, float glu_cubic) {
+                                     float glu_limit, float glu_add, float glu_cubic, int act) {
   pdl_trigger();
   pdl_wait();
   const long long total = (long long)M * N;
@@ -921,7 +932,7 @@ __global__ void splitk_reduce_kernel(const float* ws, int splits, const float* _
       for (int s = 0; s < splits; ++s) acc += ws[(size_t)s * total + (size_t)m * N + c];
       if (bias) acc += bias[c];
       const size_t o = (size_t)m * ldo + c;
-      if (mode == OUT_BF16) ((bf16*)out)[o] = __float2bfloat16_rn(acc);
+      if (mode == OUT_BF16) ((bf16*)out)[o] = __float2bfloat16_rn(apply_act(act, acc));
       else if (mode == OUT_F32) ((float*)out)[o] = acc;
       else ((float*)out)[o] += acc;
     }
@@ -1156,13 +1167,14 @@ GB_API int gb_linear_tc_supported(const void* X, long long ldx, const void* W, l
 // mode 0: out bf16 [M, N]; 1: out f32; 2: out f32 += ; 3: SwiGLU, W rows alternating in blocks of
 // 64 between gate and up (N = 2 * features, a multiple of 128), out bf16 [M, N / 2].
 // workspace: gb_linear_tc_workspace(M, N, K) floats (may be null when that is 0).
-// defer != 0 (modes 0 and 2): when K is split, leave the partial tiles in the workspace
+// defer != 0 (modes 0, 1 and 2): when K is split, leave the partial tiles in the workspace
 // ([splits][M][N], without bias) for the caller's next kernel to add (mode 0: and to round to
 // bfloat16); nothing is written to out.  defer == 2 (mode 2): the same also when K is not split:
 // the whole product goes to the workspace as one "partial" tile set, so that a large product into
 // the residual stream only stores (the norm that reads the stream next adds it while it reads)
 // instead of reading and rewriting 32-bit rows from its epilogue.
-// flags bit 0: read the weights with an evict-first hint.
+// flags bit 0: read the weights with an evict-first hint; bits 8 to 15 (mode 0, not deferred): a function of the finished
+// sums (1: the square of relu), applied in 32-bit before they are rounded.
 // Returns the number of kernels launched, or a negative error code.
 static int linear_tc_impl(const void* X, long long ldx, const void* W, long long ldw, const float* bias, void* out,
                           int mode, long long ldo, int M, int N, int K, float* workspace, int defer, int flags,
@@ -1200,8 +1212,11 @@ static int linear_tc_impl(const void* X, long long ldx, const void* W, long long
   int bn, splits, kb_per_split;
   plan(M, N, K, &bn, &splits, &kb_per_split);
   if (splits > 1 && workspace == nullptr) GB_FAIL(GB_ERR_ARG, "gb_linear_tc: these sizes need a workspace");
-  if (defer && mode != OUT_F32_ACC && mode != OUT_BF16)
-    GB_FAIL(GB_ERR_ARG, "gb_linear_tc: only a plain bfloat16 or an accumulating product can be deferred");
+  if (defer && mode == OUT_SWIGLU)
+    GB_FAIL(GB_ERR_ARG, "gb_linear_tc: only a plain or an accumulating product can be deferred");
+  const int act = (flags >> 8) & 255;
+  if (act > ACT_RELU2 || (act && (mode != OUT_BF16 || defer)))
+    GB_FAIL(GB_ERR_ARG, "gb_linear_tc: function %d of an output of mode %d (deferred: %d)", act, mode, defer);
 
   CUtensorMap tw, tx;
   {
@@ -1238,6 +1253,7 @@ static int linear_tc_impl(const void* X, long long ldx, const void* W, long long
   p.vec_store = (((uintptr_t)out & 15) == 0 && (ldo * (mode == OUT_BF16 || mode == OUT_SWIGLU ? 2 : 4)) % 16 == 0) ? 1 : 0;
   p.status = status;
   p.glu_alpha = glu_alpha; p.glu_limit = glu_limit; p.glu_add = glu_add; p.glu_cubic = glu_cubic;
+  p.act = act;
   int rc;
   const long long n_tiles = (long long)gb_div_up(N, BM) * gb_div_up(M, bn);
   if (pairs) {
@@ -1256,7 +1272,7 @@ static int linear_tc_impl(const void* X, long long ldx, const void* W, long long
     const long long work = (long long)M * (mode == OUT_SWIGLU ? N / 2 : N);
     const int blocks = (int)((work + 255) / 256 < 148 * 8 ? (work + 255) / 256 : 148 * 8);
     gb_launch(splitk_reduce_kernel, dim3(blocks), dim3(256), 0, stream, workspace, splits, bias, out, ldo, mode, M, N,
-              p.glu_alpha, p.glu_limit, p.glu_add, p.glu_cubic);
+              p.glu_alpha, p.glu_limit, p.glu_add, p.glu_cubic, p.act);
     GB_CHECK_LAUNCH("gb_linear_tc (split-K reduce)");
     return 2;
   }
@@ -1351,6 +1367,7 @@ GB_API int gb_linear_tc_no_alloc(const void* X, long long ldx, const void* W, lo
   p.vec_store = (((uintptr_t)out & 15) == 0 && (ldo * (mode == OUT_BF16 || mode == OUT_SWIGLU ? 2 : 4)) % 16 == 0) ? 1 : 0;
   p.status = status;
   p.glu_alpha = 1.f; p.glu_limit = INFINITY; p.glu_add = 0.f; p.glu_cubic = 0.f;
+  p.act = ACT_NONE;
   int rc;
   switch (bn) {
     case 16: rc = launch<16>(tw, tx, p, stream); break;
@@ -1364,7 +1381,7 @@ GB_API int gb_linear_tc_no_alloc(const void* X, long long ldx, const void* W, lo
     const long long work = (long long)M * (mode == OUT_SWIGLU ? N / 2 : N);
     const int blocks = (int)((work + 255) / 256 < 148 * 8 ? (work + 255) / 256 : 148 * 8);
     gb_launch(splitk_reduce_kernel, dim3(blocks), dim3(256), 0, stream, (const float*)ws, splits, bias, out, ldo, mode,
-              M, N, p.glu_alpha, p.glu_limit, p.glu_add, p.glu_cubic);
+              M, N, p.glu_alpha, p.glu_limit, p.glu_add, p.glu_cubic, p.act);
     GB_CHECK_LAUNCH("gb_linear_tc_no_alloc (split-K reduce)");
     return 2;
   }

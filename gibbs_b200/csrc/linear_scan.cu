@@ -42,19 +42,28 @@ template <int LEFT> __device__ __forceinline__ void ls_wait() {
 }
 
 // A column of S lies in the registers of SPLIT neighbouring lanes, PER of its dim values each (dim <= SPLIT * PER;
-// lane q holds rows 4 (q + SPLIT i) + e).  The inputs of TOK tokens at a time arrive by asynchronous copies into one
-// of two buffers while the tokens of the other are consumed.  GROUP tokens are computed one after the other, each
+// lane q holds rows 4 (q + SPLIT i) + e).  The inputs of TOK tokens at a time arrive by asynchronous copies in a ring of
+// STAGES buffers, of which all but one are on their way while one is consumed; what a thread copies is the same for every
+// token, so its source and place are worked out once.  GROUP tokens are computed one after the other, each
 // leaving this lane's share of its read-out in a register, and the shares of all of them are then added over the lanes
 // together, every exchange halving what a lane still carries: one shuffle a token instead of log2(SPLIT).  A portion's
 // last tokens, fewer than GROUP, are added one by one in the same order of additions, so how a prompt is cut does not
 // change a bit.
+constexpr int LS_STAGES = 4;
+
+template <int SPLIT, int PER, int TOK, bool CHANNEL>
+struct ScanCfg {
+  static constexpr int NR = SPLIT * PER, COLS = LS_THREADS / SPLIT, ROWS = CHANNEL ? 3 : 2;
+  static constexpr int BUF = TOK * (ROWS * NR + COLS + 4);   // q [TOK][NR] | k | (g) | v [TOK][COLS] | (g, w, -, -) [TOK]
+  static constexpr int SMEM = LS_STAGES * BUF * 4;
+};
+
 template <int SPLIT, int PER, int TOK, bool CHANNEL>
 __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(ScanParams p) {
-  constexpr int NR = SPLIT * PER, COLS = LS_THREADS / SPLIT, Q4 = PER / 4;
+  using C = ScanCfg<SPLIT, PER, TOK, CHANNEL>;
+  constexpr int NR = C::NR, COLS = C::COLS, Q4 = PER / 4, ROWS = C::ROWS, BUF = C::BUF;
   constexpr int GROUP = SPLIT < 8 ? SPLIT : 8;
-  constexpr int ROWS = CHANNEL ? 3 : 2;
-  constexpr int BUF = TOK * (ROWS * NR + COLS + 2);      // q [TOK][NR] | k | (g) | v [TOK][COLS] | g [TOK] | w [TOK]
-  extern __shared__ __align__(16) float ls_sm[];         // [2][BUF]
+  extern __shared__ __align__(16) float ls_sm[];         // [LS_STAGES][BUF]
   pdl_trigger();
   const int col = threadIdx.x / SPLIT, q = threadIdx.x % SPLIT;
   const int r = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * COLS, c = c0 + col;
@@ -62,8 +71,38 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(ScanParams p) {
   const bool counts = c == p.vdim;                       // the normaliser's column: its value is always 1
   const int first = p.q_start[r], len = p.q_len[r];
   float* S = p.state + (size_t)p.slot_ids[r] * p.slot_stride + ((size_t)h * p.cols + (active ? c : 0)) * p.dim;
-  if (p.dim < NR || p.vdim - c0 < COLS)                  // what is never copied stays zero
-    for (int i = threadIdx.x; i < 2 * BUF; i += LS_THREADS) ls_sm[i] = 0.f;
+  const int vcols = max(0, min(COLS, p.vdim - c0));
+  if (p.dim < NR || vcols < COLS)                        // what is never copied stays zero
+    for (int i = threadIdx.x; i < LS_STAGES * BUF; i += LS_THREADS) ls_sm[i] = 0.f;
+  // what this thread copies of every token: pieces of 16 bytes (of 4 where rows are not aligned) of [q | k | g | v]
+  constexpr int VEC_ROLES = (ROWS * NR / 4 + COLS / 4 + LS_THREADS) / LS_THREADS;
+  const float* r_src[VEC_ROLES];
+  long long r_ld[VEC_ROLES];
+  int r_dst[VEC_ROLES], r_step[VEC_ROLES];
+  const bool vec = p.vec_rows && p.vec_v;
+  if (vec) {
+    const int pieces = p.dim >> 2;
+#pragma unroll
+    for (int j = 0; j < VEC_ROLES; ++j) {
+      const int i = threadIdx.x + j * LS_THREADS;
+      r_src[j] = nullptr;
+      r_ld[j] = 0;
+      r_dst[j] = r_step[j] = 0;
+      if (i < ROWS * pieces) {
+        const int which = i / pieces, c4 = 4 * (i - which * pieces);
+        r_ld[j] = which == 0 ? p.ldq : which == 1 ? p.ldk : p.ldg;
+        r_src[j] = (which == 0 ? p.q : which == 1 ? p.k : p.g) + (size_t)first * r_ld[j] + (size_t)h * p.dim + c4;
+        r_dst[j] = which * TOK * NR + c4;
+        r_step[j] = NR;
+      } else if (i < ROWS * pieces + (vcols >> 2)) {
+        const int c4 = 4 * (i - ROWS * pieces);
+        r_ld[j] = p.ldv;
+        r_src[j] = p.v + (size_t)first * p.ldv + (size_t)h * p.vdim + c0 + c4;
+        r_dst[j] = ROWS * TOK * NR + c4;
+        r_step[j] = COLS;
+      }
+    }
+  }
   pdl_wait();
   const bool vec_state = (p.dim & 3) == 0 && (p.slot_stride & 3) == 0 && ((uintptr_t)p.state & 15) == 0;
   float s[PER];
@@ -85,78 +124,71 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(ScanParams p) {
   }
   __syncthreads();
 
-  const int vcols = max(0, min(COLS, p.vdim - c0));
-  auto stage = [&](int t0, int b) {
-    const int nt = min(TOK, len - t0);
-    float* Q = ls_sm + b * BUF;
-    float* V = Q + ROWS * TOK * NR;
-    const size_t row0 = (size_t)(first + t0);
-    const float* src[3] = {p.q + row0 * p.ldq + (size_t)h * p.dim, p.k + row0 * p.ldk + (size_t)h * p.dim,
-                           CHANNEL ? p.g + row0 * p.ldg + (size_t)h * p.dim : nullptr};
-    const long long ld[3] = {p.ldq, p.ldk, p.ldg};
-    if (p.vec_rows) {
-      const int pieces = p.dim >> 2;
-      for (int i = threadIdx.x; i < pieces; i += LS_THREADS) {      // (a thread's piece is the same for every token)
+  const int chunks = (len + TOK - 1) / TOK;
+  auto stage = [&](int chunk) {                          // (always one group of copies, possibly an empty one)
+    if (chunk < chunks) {
+      const int t0 = chunk * TOK, nt = min(TOK, len - t0);
+      float* Q = ls_sm + (chunk % LS_STAGES) * BUF;
+      if (vec) {
 #pragma unroll
-        for (int a = 0; a < ROWS; ++a)
-          for (int tt = 0; tt < nt; ++tt)
-            gb_cp_async_16(Q + (a * TOK + tt) * NR + 4 * i, src[a] + (size_t)tt * ld[a] + 4 * i);
-      }
-    } else {
-      for (int i = threadIdx.x; i < p.dim; i += LS_THREADS)
+        for (int j = 0; j < VEC_ROLES; ++j) {
+          if (r_src[j] == nullptr) continue;
+          const float* src = r_src[j] + (size_t)t0 * r_ld[j];
+          float* dst = Q + r_dst[j];
+          if (nt == TOK) {
 #pragma unroll
-        for (int a = 0; a < ROWS; ++a)
-          for (int tt = 0; tt < nt; ++tt) gb_cp_async_4(Q + (a * TOK + tt) * NR + i, src[a] + (size_t)tt * ld[a] + i);
-    }
-    const float* vs = p.v + row0 * p.ldv + (size_t)h * p.vdim + c0;
-    if (p.vec_v) {
-      const int vp = vcols >> 2;
-      for (int i = LS_THREADS - 1 - threadIdx.x; i < nt * vp; i += LS_THREADS) {
-        const int tt = i / vp, c4 = i - tt * vp;
-        gb_cp_async_16(V + tt * COLS + 4 * c4, vs + (size_t)tt * p.ldv + 4 * c4);
+            for (int tt = 0; tt < TOK; ++tt, src += r_ld[j], dst += r_step[j]) gb_cp_async_16(dst, src);
+          } else {
+            for (int tt = 0; tt < nt; ++tt, src += r_ld[j], dst += r_step[j]) gb_cp_async_16(dst, src);
+          }
+        }
+      } else {
+        const size_t row0 = (size_t)(first + t0);
+        for (int tt = 0; tt < nt; ++tt) {
+          for (int i = threadIdx.x; i < p.dim; i += LS_THREADS) {
+            gb_cp_async_4(Q + tt * NR + i, p.q + (row0 + tt) * p.ldq + (size_t)h * p.dim + i);
+            gb_cp_async_4(Q + (TOK + tt) * NR + i, p.k + (row0 + tt) * p.ldk + (size_t)h * p.dim + i);
+            if (CHANNEL) gb_cp_async_4(Q + (2 * TOK + tt) * NR + i, p.g + (row0 + tt) * p.ldg + (size_t)h * p.dim + i);
+          }
+          for (int i = threadIdx.x; i < vcols; i += LS_THREADS)
+            gb_cp_async_4(Q + ROWS * TOK * NR + tt * COLS + i, p.v + (row0 + tt) * p.ldv + (size_t)h * p.vdim + c0 + i);
+        }
       }
-    } else {
-      for (int i = LS_THREADS - 1 - threadIdx.x; i < nt * vcols; i += LS_THREADS) {
-        const int tt = i / vcols, cc = i - tt * vcols;
-        gb_cp_async_4(V + tt * COLS + cc, vs + (size_t)tt * p.ldv + cc);
+      float* G = Q + TOK * (ROWS * NR + COLS);
+      const int tt = LS_THREADS - 1 - threadIdx.x;         // (the last threads: the first ones copy most pieces)
+      if (tt < nt) {
+        const size_t row = (size_t)(first + t0 + tt);
+        if (!CHANNEL) gb_cp_async_4(G + 4 * tt, p.g + row * p.ldg + h);
+        if (p.w) gb_cp_async_4(G + 4 * tt + 1, p.w + row * p.ldw + h);
       }
-    }
-    float* G = V + TOK * COLS;
-    if ((int)threadIdx.x < nt) {
-      if (!CHANNEL) gb_cp_async_4(G + threadIdx.x, p.g + (row0 + threadIdx.x) * p.ldg + h);
-      if (p.w) gb_cp_async_4(G + TOK + threadIdx.x, p.w + (row0 + threadIdx.x) * p.ldw + h);
     }
     ls_commit();
   };
 
-  if (len > 0) stage(0, 0);
-  int b = 0;
-  for (int t0 = 0; t0 < len; t0 += TOK, b ^= 1) {
-    const int nt = min(TOK, len - t0);
-    if (t0 + TOK < len) {
-      stage(t0 + TOK, b ^ 1);
-      ls_wait<1>();                                      // this chunk has landed, the next is on its way
-    } else {
-      ls_wait<0>();
-    }
-    __syncthreads();
-    const float* Q = ls_sm + b * BUF + 4 * q;
+#pragma unroll
+  for (int i = 0; i < LS_STAGES - 1; ++i) stage(i);
+  const bool weighted = p.w != nullptr;
+  for (int chunk = 0; chunk < chunks; ++chunk) {
+    ls_wait<LS_STAGES - 2>();                            // this chunk's copies have landed ...
+    __syncthreads();                                     // ... everybody's, and the chunk before has been used
+    stage(chunk + LS_STAGES - 1);
+    const int t0 = chunk * TOK, nt = min(TOK, len - t0);
+    const float* Q = ls_sm + (chunk % LS_STAGES) * BUF + 4 * q;
     const float* K = Q + TOK * NR;
     const float* G = K + TOK * NR;
-    const float* V = ls_sm + b * BUF + ROWS * TOK * NR;
-    const float* Gh = V + TOK * COLS;
-    const float* Wh = Gh + TOK;
+    const float* V = ls_sm + (chunk % LS_STAGES) * BUF + ROWS * TOK * NR + col;
+    const float* GW = ls_sm + (chunk % LS_STAGES) * BUF + TOK * (ROWS * NR + COLS);
     // one token: the state's step, and this lane's share of the read-out
     auto token = [&](int tt) {
-      float v = counts ? 1.f : V[tt * COLS + col];
-      if (p.w) v *= Wh[tt];
-      const float gh = CHANNEL ? 0.f : Gh[tt];
+      float v = counts ? 1.f : V[tt * COLS];
+      const float2 gw = *reinterpret_cast<const float2*>(GW + 4 * tt);
+      if (weighted) v *= gw.y;
       float d0 = 0.f, d1 = 0.f, d2 = 0.f, d3 = 0.f;      // four chains, added in a fixed order
 #pragma unroll
       for (int i = 0; i < Q4; ++i) {
         const float4 k4 = *reinterpret_cast<const float4*>(K + tt * NR + 4 * SPLIT * i);
         const float4 q4 = *reinterpret_cast<const float4*>(Q + tt * NR + 4 * SPLIT * i);
-        float4 g4 = make_float4(gh, gh, gh, gh);
+        float4 g4 = make_float4(gw.x, gw.x, gw.x, gw.x);
         if (CHANNEL) g4 = *reinterpret_cast<const float4*>(G + tt * NR + 4 * SPLIT * i);
         s[4 * i] = fmaf(g4.x, s[4 * i], k4.x * v);             d0 = fmaf(s[4 * i], q4.x, d0);
         s[4 * i + 1] = fmaf(g4.y, s[4 * i + 1], k4.y * v);     d1 = fmaf(s[4 * i + 1], q4.y, d1);
@@ -170,12 +202,11 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(ScanParams p) {
       if (counts) p.nq[row * p.H + h] = o * p.q_scale;
       else p.out[row * p.ldo + (size_t)h * p.vdim + c] = o * p.q_scale;
     };
-    int tt = 0;
-    for (; tt + GROUP <= nt; tt += GROUP) {
+    // lanes whose bit `w` is set keep the upper half of the tokens they carry, the others the lower half
+    auto group = [&](int tt) {
       float o[GROUP];
 #pragma unroll
       for (int u = 0; u < GROUP; ++u) o[u] = token(tt + u);
-      // lanes whose bit `w` is set keep the upper half of the tokens they carry, the others the lower half
       int mine = 0;
 #pragma unroll
       for (int w = SPLIT / 2, carried = GROUP; w > 0; w >>= 1) {
@@ -197,6 +228,13 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(ScanParams p) {
       }
       // (several lanes carry the same token when there are more lanes than tokens: the first of them stores)
       if (active && (q & (SPLIT / GROUP - 1)) == 0) put(tt + mine, o[0]);
+    };
+    int tt = 0;
+    if (nt == TOK) {
+#pragma unroll
+      for (; tt + GROUP <= TOK; tt += GROUP) group(tt);
+    } else {
+      for (; tt + GROUP <= nt; tt += GROUP) group(tt);
     }
     for (; tt < nt; ++tt) {
       float o = token(tt);
@@ -204,7 +242,6 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(ScanParams p) {
       for (int w = SPLIT / 2; w > 0; w >>= 1) o += __shfl_xor_sync(0xffffffffu, o, w);
       if (active && q == 0) put(tt, o);
     }
-    __syncthreads();                                     // before the copies of the chunk after next land here
   }
   if (!active) return;
 #pragma unroll
@@ -237,41 +274,41 @@ __global__ void forget_write_gates_kernel(float* q, long long ldq, float* f, lon
   k[(size_t)t * ldk + c] = (1.f - l) * hy_sigmoid(-z);   // (1 - f without the cancellation where f is near one)
 }
 
-// One warp per (request, head).  m -> max(m + F, I) is closed under composition ((F1, I1) then (F2, I2) is
-// (F1 + F2, max(I1 + F2, I2))), so 32 tokens are combined by a scan over the lanes.
+// A block per (request, head).  m -> max(m + F, I) is closed under composition ((F1, I1) then (F2, I2) is
+// (F1 + F2, max(I1 + F2, I2))), so a round of tokens, one a thread, is combined by scans over the lanes of each warp and
+// then over the warps.
 __global__ void exp_gates_kernel(const float* zi, long long ldi, const float* zf, long long ldf,
                                  const float* __restrict__ bi, const float* __restrict__ bf_, float* m_state,
                                  long long slot_stride, const int* slot_ids, const int* q_start, const int* q_len, float* g,
                                  float* w, float* floor_, int H, float cap) {
+  __shared__ float wF[32], wI[32], s_m;
   pdl_trigger();
-  const int lane = threadIdx.x & 31;
-  const int h = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
-  if (h >= H) return;                                    // (whole warps; nothing below meets the block)
-  const int r = blockIdx.x;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+  const int r = blockIdx.x, h = blockIdx.y;
   const int first = q_start[r], len = q_len[r];
   float* ms = m_state + (size_t)slot_ids[r] * slot_stride + h;
   const float ib = bi[h], fb = bf_[h];
   pdl_wait();
   float m = *ms;
-  float ni = 0.f, nf = 0.f;                              // the next 32 tokens' logits, requested a round ahead
+  float ni = 0.f, nf = 0.f;                              // the next round's logits, requested a round ahead
   auto fetch = [&](int t0) {
-    const int t = t0 + lane;
+    const int t = t0 + threadIdx.x;
     if (t < len) {
       ni = zi[(size_t)(first + t) * ldi + h];
       nf = zf[(size_t)(first + t) * ldf + h];
     }
   };
   fetch(0);
-  for (int t0 = 0; t0 < len; t0 += 32) {
-    const int t = t0 + lane;
+  for (int t0 = 0; t0 < len; t0 += blockDim.x) {
+    const int t = t0 + threadIdx.x;
     const float ri = ni, rf = nf;
-    fetch(t0 + 32);
+    fetch(t0 + blockDim.x);
     const bool in = t < len;
     const float i = in ? cap * tanhf((ri + ib) / cap) : -INFINITY;
     const float zz = cap * tanhf((rf + fb) / cap);
     // log sigmoid(z) = min(z, 0) - log1p(exp(-|z|))
     const float f = in ? fminf(zz, 0.f) - log1pf(expf(-fabsf(zz))) : 0.f;
-    float F = f, I = i;                                  // composition of tokens t0 .. t
+    float F = f, I = i;                                  // composition of this warp's tokens up to t
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
       const float Fp = __shfl_up_sync(0xffffffffu, F, o), Ip = __shfl_up_sync(0xffffffffu, I, o);
@@ -280,18 +317,30 @@ __global__ void exp_gates_kernel(const float* zi, long long ldi, const float* zf
         F = Fp + F;
       }
     }
-    const float mt = fmaxf(m + F, I);
+    float mw = m;                                        // the maximum in front of this warp's tokens
+    if (warps > 1) {
+      __syncthreads();                                   // (the round before has read these)
+      if (lane == 31) { wF[warp] = F; wI[warp] = I; }
+      __syncthreads();
+      for (int k = 0; k < warp; ++k) mw = fmaxf(mw + wF[k], wI[k]);
+    }
+    const float mt = fmaxf(mw + F, I);
     float before = __shfl_up_sync(0xffffffffu, mt, 1);
-    if (lane == 0) before = m;
+    if (lane == 0) before = mw;
     if (in) {
       const size_t at = (size_t)(first + t) * H + h;
       g[at] = expf(f + before - mt);
       w[at] = expf(i - mt);
       floor_[at] = expf(-mt);
     }
-    m = __shfl_sync(0xffffffffu, mt, 31);
+    m = __shfl_sync(0xffffffffu, mt, 31);                // (the last warp's is the round's)
+    if (warps > 1) {
+      if (threadIdx.x == blockDim.x - 1) s_m = mt;
+      __syncthreads();
+      m = s_m;
+    }
   }
-  if (lane == 0) *ms = m;
+  if (threadIdx.x == 0) *ms = m;
 }
 
 }  // namespace
@@ -319,19 +368,27 @@ GB_OP(gb_op_linear_scan) {
   p.vec_rows = p.dim % 4 == 0 && p.ldq % 4 == 0 && p.ldk % 4 == 0 && (a[0] & 15) == 0 && (a[2] & 15) == 0 &&
                (!channel || (p.ldg % 4 == 0 && (a[6] & 15) == 0));
   p.vec_v = p.vdim % 4 == 0 && p.ldv % 4 == 0 && (a[4] & 15) == 0;
-#define SCAN(SPLIT, PER, TOK)                                                                                           \
+#define SCAN_LAUNCH(SPLIT, PER, TOK, CHANNEL)                                                                          \
   do {                                                                                                                  \
-    const dim3 grid(R, p.H, gb_div_up(p.cols, LS_THREADS / SPLIT));                                                     \
-    const size_t smem = sizeof(float) * 2 * (size_t)TOK * ((channel ? 3 : 2) * SPLIT * PER + LS_THREADS / SPLIT + 2);   \
-    if (channel) gb_launch(linear_scan_kernel<SPLIT, PER, TOK, true>, grid, dim3(LS_THREADS), smem, ctx->stream, p);    \
-    else gb_launch(linear_scan_kernel<SPLIT, PER, TOK, false>, grid, dim3(LS_THREADS), smem, ctx->stream, p);           \
+    constexpr int smem = ScanCfg<SPLIT, PER, TOK, CHANNEL>::SMEM;                                                       \
+    static bool raised = false;            /* once, before any stream capture replays the launch */                    \
+    if (!raised && smem > 48 * 1024) {                                                                                  \
+      GB_CUDA((cudaFuncSetAttribute(linear_scan_kernel<SPLIT, PER, TOK, CHANNEL>,                                       \
+                                    cudaFuncAttributeMaxDynamicSharedMemorySize, smem)));                               \
+      raised = true;                                                                                                    \
+    }                                                                                                                   \
+    gb_launch(linear_scan_kernel<SPLIT, PER, TOK, CHANNEL>, dim3(R, p.H, gb_div_up(p.cols, LS_THREADS / SPLIT)),         \
+              dim3(LS_THREADS), smem, ctx->stream, p);                                                                  \
   } while (0)
+#define SCAN(SPLIT, PER, TOK)                                                                                           \
+  do { if (channel) SCAN_LAUNCH(SPLIT, PER, TOK, true); else SCAN_LAUNCH(SPLIT, PER, TOK, false); } while (0)
   if (p.dim <= 16) SCAN(4, 4, 16);
   else if (p.dim <= 32) SCAN(8, 4, 16);
   else if (p.dim <= 64) SCAN(16, 4, 16);
   else if (p.dim <= 128) SCAN(8, 16, 8);
-  else SCAN(16, 16, 4);                      // (a group of eight tokens never fills: added one by one)
+  else SCAN(16, 16, 8);
 #undef SCAN
+#undef SCAN_LAUNCH
   GB_CHECK_LAUNCH("linear_scan");
   return 1;
 }
@@ -351,13 +408,13 @@ GB_OP(gb_op_forget_write_gates) {
 // a0 input-gate logits (f32 [t, heads] at a row stride), a1 that stride, a2 forget-gate logits, a3 their stride, a4 bias
 // of the former [heads], a5 of the latter, a6 m of slot 0 ([heads], f32), a7 elements between slots, a8 slot ids, a9
 // first row per request, a10 rows per request, a11 decays out (f32 [t, heads]), a12 write weights out, a13 exp(-m) out,
-// a14 requests, a15 heads; f0 cap
+// a14 requests, a15 heads, a16 tokens; f0 cap
 GB_OP(gb_op_exp_gates) {
   const int R = (int)a[14], H = (int)a[15];
   if (R <= 0) return 0;
   if (!(f[0] > 0.0)) GB_FAIL(GB_ERR_ARG, "exp_gates: a cap of %g", f[0]);
-  const int warps = H < 4 ? H : 4;
-  gb_launch(exp_gates_kernel, dim3(R, gb_div_up(H, warps)), dim3(32 * warps), 0, ctx->stream, op_ptr<const float>(a[0]), a[1],
+  const int threads = a[16] > 2 * R ? 256 : 32;          // (a few tokens a request: one warp)
+  gb_launch(exp_gates_kernel, dim3(R, H), dim3(threads), 0, ctx->stream, op_ptr<const float>(a[0]), a[1],
             op_ptr<const float>(a[2]), a[3], op_ptr<const float>(a[4]), op_ptr<const float>(a[5]), op_ptr<float>(a[6]), a[7],
             op_ptr<const int>(a[8]), op_ptr<const int>(a[9]), op_ptr<const int>(a[10]), op_ptr<float>(a[11]),
             op_ptr<float>(a[12]), op_ptr<float>(a[13]), H, (float)f[0]);

@@ -11,7 +11,7 @@
 
 namespace {
 
-constexpr int SEL_THREADS = 128, SEL_TOKENS = 16;
+constexpr int SEL_THREADS = 64, SEL_TOKENS = 16, SEL_STAGES = 4;
 
 struct SelParams {
   const float* x; long long ldx;           // [t, inner], behind the convolution
@@ -23,7 +23,7 @@ struct SelParams {
   const int* slot_ids; const int* q_start; const int* q_len;
   void* out; long long ldo;
   int inner, N;
-  int vec_bc, vec_x;                       // rows of B and C (of x and dt) can be copied in 16-byte pieces
+  int vec;                                 // all rows can be copied in 16-byte pieces
 };
 
 __device__ __forceinline__ void sel_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
@@ -38,20 +38,25 @@ __device__ __forceinline__ float sel_ex2(float x) {
 }
 
 // SPLIT neighbouring lanes share a channel, PER state entries each (state <= SPLIT * PER; lane q holds entries
-// 4 (q + SPLIT i) + e).  B, C, x and the raw step sizes of SEL_TOKENS tokens at a time arrive by asynchronous copies
-// into one of two buffers while the tokens of the other are consumed.  Once they have landed the block turns raw step
-// sizes into (dt, dt x) in place; the read-outs of a chunk's tokens are left in shared memory, and the block finishes
-// them (D x, the gate) with coalesced loads and stores.  The read-outs of GROUP tokens are added over a channel's lanes
-// together, every exchange halving what a lane still carries; single tokens at a portion's end are added in the same
-// order.  FAST: exponentials of decays as the hardware's 2^x (bfloat16 models); else expf.
+// 4 (q + SPLIT i) + e).  B, C, x, the raw step sizes and z of SEL_TOKENS tokens at a time arrive by asynchronous copies in
+// a ring of SEL_STAGES buffers; what a thread copies is the same for every token, so its source and place are worked out
+// once.  Tokens are taken four at a time: each lane of a channel turns ONE token's raw step size into (dt, dt x) and the
+// lanes exchange them, the read-outs of the four are added over the channel's lanes together (every exchange halves what
+// a lane still carries), and the lane that ends up with a token's read-out finishes it (D x, the gate).  Single tokens at
+// a portion's end are computed with the same arithmetic, so how a prompt is cut does not change a bit.
+// FAST: exponentials of decays as the hardware's 2^x (bfloat16 models); else expf.
+template <int SPLIT, int PER> struct SelCfg {
+  static constexpr int NR = SPLIT * PER, CH = SEL_THREADS / SPLIT;
+  static constexpr int BUF = SEL_TOKENS * (2 * NR + 3 * CH);       // B [TOK][NR] | C | x [TOK][CH] | dt | z
+  static constexpr int SMEM = SEL_STAGES * BUF * 4;
+};
+
 template <int SPLIT, int PER, bool FAST, typename TO>
 __global__ void __launch_bounds__(SEL_THREADS) selective_scan_kernel(SelParams p) {
-  constexpr int NR = SPLIT * PER, CH = SEL_THREADS / SPLIT, Q4 = PER / 4, TOK = SEL_TOKENS;
-  constexpr int GROUP = SPLIT < 4 ? SPLIT : 4;
-  constexpr int BUF = TOK * (2 * NR + 2 * CH);           // B [TOK][NR] | C [TOK][NR] | x [TOK][CH] | dt [TOK][CH]
-  extern __shared__ __align__(16) float sel_sm[];        // [2][BUF], then step sizes [TOK][CH], then read-outs [TOK][CH]
-  float* sDt = sel_sm + 2 * BUF;
-  float* sY = sDt + TOK * CH;
+  using Cf = SelCfg<SPLIT, PER>;
+  constexpr int NR = Cf::NR, CH = Cf::CH, Q4 = PER / 4, TOK = SEL_TOKENS, BUF = Cf::BUF;
+  static_assert(SPLIT >= 4, "four lanes share the work around four tokens");
+  extern __shared__ __align__(16) float sel_sm[];        // [SEL_STAGES][BUF]
   pdl_trigger();
   const int ch = threadIdx.x / SPLIT, q = threadIdx.x % SPLIT;
   const int r = blockIdx.x, c0 = blockIdx.y * CH, c = c0 + ch;
@@ -67,9 +72,38 @@ __global__ void __launch_bounds__(SEL_THREADS) selective_scan_kernel(SelParams p
       const int n = 4 * (q + SPLIT * i) + e;
       A[4 * i + e] = (active && n < N) ? -expf(p.a_log[(size_t)c * N + n]) * (FAST ? LOG2E : 1.f) : 0.f;
     }
+  const float bias = active ? p.dt_bias[c] : 0.f, dskip = active ? p.dskip[c] : 0.f;
   float* S = p.state + (size_t)p.slot_ids[r] * p.slot_stride + (size_t)(active ? c : 0) * N;
   if (N < NR || channels < CH)                           // what is never copied stays zero
-    for (int i = threadIdx.x; i < 2 * BUF; i += SEL_THREADS) sel_sm[i] = 0.f;
+    for (int i = threadIdx.x; i < SEL_STAGES * BUF; i += SEL_THREADS) sel_sm[i] = 0.f;
+  // what this thread copies of every token: 16-byte pieces of [B | C | x | dt | z]
+  constexpr int ROLES = (2 * NR / 4 + 3 * CH / 4 + SEL_THREADS - 1) / SEL_THREADS;
+  const float* r_src[ROLES];
+  long long r_ld[ROLES];
+  int r_dst[ROLES], r_step[ROLES];
+  if (p.vec) {
+    const int nb = N >> 2, nx = channels >> 2;
+#pragma unroll
+    for (int j = 0; j < ROLES; ++j) {
+      const int i = threadIdx.x + j * SEL_THREADS;
+      r_src[j] = nullptr;
+      r_ld[j] = 0;
+      r_dst[j] = r_step[j] = 0;
+      if (i < 2 * nb) {
+        const int which = i / nb, c4 = 4 * (i - which * nb);
+        r_ld[j] = p.ldbc;
+        r_src[j] = (which ? p.C : p.B) + (size_t)first * p.ldbc + c4;
+        r_dst[j] = which * TOK * NR + c4;
+        r_step[j] = NR;
+      } else if (i < 2 * nb + 3 * nx) {
+        const int which = (i - 2 * nb) / nx, c4 = 4 * (i - 2 * nb - which * nx);
+        r_ld[j] = which == 0 ? p.ldx : which == 1 ? p.lddt : p.ldz;
+        r_src[j] = (which == 0 ? p.x : which == 1 ? p.dt : p.z) + (size_t)first * r_ld[j] + c0 + c4;
+        r_dst[j] = 2 * TOK * NR + which * TOK * CH + c4;
+        r_step[j] = CH;
+      }
+    }
+  }
   pdl_wait();
   const bool vec_state = (N & 3) == 0 && (p.slot_stride & 3) == 0 && ((uintptr_t)p.state & 15) == 0;
   float s[PER];
@@ -91,60 +125,55 @@ __global__ void __launch_bounds__(SEL_THREADS) selective_scan_kernel(SelParams p
   }
   __syncthreads();
 
-  auto rows = [&](float* dst, int stride, const float* src, long long ld, int nt, int width, bool vec) {
-    if (vec) {
-      const int pieces = width >> 2;
-      for (int i = threadIdx.x; i < nt * pieces; i += SEL_THREADS) {
-        const int tt = i / pieces, c4 = i - tt * pieces;
-        gb_cp_async_16(dst + tt * stride + 4 * c4, src + (size_t)tt * ld + 4 * c4);
-      }
-    } else {
-      for (int i = threadIdx.x; i < nt * width; i += SEL_THREADS) {
-        const int tt = i / width, cc = i - tt * width;
-        gb_cp_async_4(dst + tt * stride + cc, src + (size_t)tt * ld + cc);
+  const int chunks = (len + TOK - 1) / TOK;
+  auto stage = [&](int chunk) {                          // (always one group of copies, possibly an empty one)
+    if (chunk < chunks) {
+      const int t0 = chunk * TOK, nt = min(TOK, len - t0);
+      float* Bs = sel_sm + (chunk % SEL_STAGES) * BUF;
+      if (p.vec) {
+#pragma unroll
+        for (int j = 0; j < ROLES; ++j) {
+          if (r_src[j] == nullptr) continue;
+          const float* src = r_src[j] + (size_t)t0 * r_ld[j];
+          float* dst = Bs + r_dst[j];
+          if (nt == TOK) {
+#pragma unroll
+            for (int tt = 0; tt < TOK; ++tt, src += r_ld[j], dst += r_step[j]) gb_cp_async_16(dst, src);
+          } else {
+            for (int tt = 0; tt < nt; ++tt, src += r_ld[j], dst += r_step[j]) gb_cp_async_16(dst, src);
+          }
+        }
+      } else {
+        for (int tt = 0; tt < nt; ++tt) {
+          const size_t row = (size_t)(first + t0 + tt);
+          for (int i = threadIdx.x; i < N; i += SEL_THREADS) {
+            gb_cp_async_4(Bs + tt * NR + i, p.B + row * p.ldbc + i);
+            gb_cp_async_4(Bs + (TOK + tt) * NR + i, p.C + row * p.ldbc + i);
+          }
+          float* X = Bs + 2 * TOK * NR + tt * CH;
+          for (int i = threadIdx.x; i < channels; i += SEL_THREADS) {
+            gb_cp_async_4(X + i, p.x + row * p.ldx + c0 + i);
+            gb_cp_async_4(X + TOK * CH + i, p.dt + row * p.lddt + c0 + i);
+            gb_cp_async_4(X + 2 * TOK * CH + i, p.z + row * p.ldz + c0 + i);
+          }
+        }
       }
     }
-  };
-  auto stage = [&](int t0, int b) {
-    const int nt = min(TOK, len - t0);
-    float* Bs = sel_sm + b * BUF;
-    const size_t row0 = (size_t)(first + t0);
-    rows(Bs, NR, p.B + row0 * p.ldbc, p.ldbc, nt, N, p.vec_bc);
-    rows(Bs + TOK * NR, NR, p.C + row0 * p.ldbc, p.ldbc, nt, N, p.vec_bc);
-    rows(Bs + 2 * TOK * NR, CH, p.x + row0 * p.ldx + c0, p.ldx, nt, channels, p.vec_x);
-    rows(Bs + 2 * TOK * NR + TOK * CH, CH, p.dt + row0 * p.lddt + c0, p.lddt, nt, channels, p.vec_x);
     sel_commit();
   };
 
-  if (len > 0) stage(0, 0);
-  int b = 0;
-  for (int t0 = 0; t0 < len; t0 += TOK, b ^= 1) {
-    const int nt = min(TOK, len - t0);
-    if (t0 + TOK < len) {
-      stage(t0 + TOK, b ^ 1);
-      sel_wait<1>();                                     // this chunk has landed, the next is on its way
-    } else {
-      sel_wait<0>();
-    }
-    __syncthreads();
-    const float* Bs = sel_sm + b * BUF;
-    const float* X = Bs + 2 * TOK * NR;
-    float* Dx = sel_sm + b * BUF + 2 * TOK * NR + TOK * CH;       // raw step sizes, replaced by dt * x
-    for (int i = threadIdx.x; i < nt * CH; i += SEL_THREADS) {
-      const int cc = i % CH;
-      if (cc < channels) {
-        const float dt = hy_softplus(Dx[i] + p.dt_bias[c0 + cc]);
-        sDt[i] = dt;
-        Dx[i] = dt * X[i];
-      } else {
-        sDt[i] = 0.f;
-      }
-    }
-    __syncthreads();
+#pragma unroll
+  for (int i = 0; i < SEL_STAGES - 1; ++i) stage(i);
+  for (int chunk = 0; chunk < chunks; ++chunk) {
+    sel_wait<SEL_STAGES - 2>();                          // this chunk's copies have landed ...
+    __syncthreads();                                     // ... everybody's, and the chunk before has been used
+    stage(chunk + SEL_STAGES - 1);
+    const int t0 = chunk * TOK, nt = min(TOK, len - t0);
+    const float* Bs = sel_sm + (chunk % SEL_STAGES) * BUF;
+    const float* X = Bs + 2 * TOK * NR + ch;
     const float* Bq = Bs + 4 * q;
     const float* Cq = Bq + TOK * NR;
-    auto token = [&](int tt) {
-      const float dt = sDt[tt * CH + ch], dx = Dx[tt * CH + ch];
+    auto token = [&](int tt, float dt, float dx) {
       float y0 = 0.f, y1 = 0.f, y2 = 0.f, y3 = 0.f;      // four chains, added in a fixed order
 #pragma unroll
       for (int i = 0; i < Q4; ++i) {
@@ -161,19 +190,27 @@ __global__ void __launch_bounds__(SEL_THREADS) selective_scan_kernel(SelParams p
       }
       return (y0 + y1) + (y2 + y3);
     };
-    int tt = 0;
-    for (; tt + GROUP <= nt; tt += GROUP) {
-      float y[GROUP];
+    auto put = [&](int tt, float y) {
+      const float xv = X[tt * CH], z = X[2 * TOK * CH + tt * CH];
+      ((TO*)p.out)[(size_t)(first + t0 + tt) * p.ldo + c] = from_f32<TO>(fmaf(dskip, xv, y) * hy_silu(z));
+    };
+    auto four = [&](int tt) {
+      const int own = tt + (q & 3);
+      const float odt = hy_softplus(X[TOK * CH + own * CH] + bias), odx = odt * X[own * CH];
+      float y[4];
 #pragma unroll
-      for (int u = 0; u < GROUP; ++u) y[u] = token(tt + u);
+      for (int u = 0; u < 4; ++u) {
+        const float dt = __shfl_sync(0xffffffffu, odt, u, SPLIT), dx = __shfl_sync(0xffffffffu, odx, u, SPLIT);
+        y[u] = token(tt + u, dt, dx);
+      }
       int mine = 0;
 #pragma unroll
-      for (int w = SPLIT / 2, carried = GROUP; w > 0; w >>= 1) {
+      for (int w = SPLIT / 2, carried = 4; w > 0; w >>= 1) {
         if (carried > 1) {
           const int half = carried / 2;
           const bool upper = q & w;
 #pragma unroll
-          for (int u = 0; u < GROUP / 2; ++u) {
+          for (int u = 0; u < 2; ++u) {
             if (u < half) {
               const float give = upper ? y[u] : y[u + half], keep = upper ? y[u + half] : y[u];
               y[u] = keep + __shfl_xor_sync(0xffffffffu, give, w);
@@ -185,24 +222,22 @@ __global__ void __launch_bounds__(SEL_THREADS) selective_scan_kernel(SelParams p
           y[0] += __shfl_xor_sync(0xffffffffu, y[0], w);
         }
       }
-      if ((q & (SPLIT / GROUP - 1)) == 0) sY[(tt + mine) * CH + ch] = y[0];
+      if (active && (q & (SPLIT / 4 - 1)) == 0) put(tt + mine, y[0]);
+    };
+    int tt = 0;
+    if (nt == TOK) {
+#pragma unroll 2
+      for (; tt < TOK; tt += 4) four(tt);
+    } else {
+      for (; tt + 4 <= nt; tt += 4) four(tt);
     }
     for (; tt < nt; ++tt) {
-      float y = token(tt);
+      const float dt = hy_softplus(X[TOK * CH + tt * CH] + bias);
+      float y = token(tt, dt, dt * X[tt * CH]);
 #pragma unroll
       for (int w = SPLIT / 2; w > 0; w >>= 1) y += __shfl_xor_sync(0xffffffffu, y, w);
-      if (q == 0) sY[tt * CH + ch] = y;
+      if (active && q == 0) put(tt, y);
     }
-    __syncthreads();
-    // the chunk's outputs, neighbouring threads on neighbouring channels
-    for (int i = threadIdx.x; i < nt * CH; i += SEL_THREADS) {
-      const int t = i / CH, cc = i % CH;
-      if (cc >= channels) continue;
-      const size_t row = (size_t)(first + t0 + t);
-      const float y = fmaf(p.dskip[c0 + cc], X[i], sY[i]);
-      ((TO*)p.out)[row * p.ldo + c0 + cc] = from_f32<TO>(y * hy_silu(p.z[row * p.ldz + c0 + cc]));
-    }
-    __syncthreads();                                     // before the copies of the chunk after next land here
   }
   if (!active) return;
 #pragma unroll
@@ -239,15 +274,15 @@ GB_OP(gb_op_selective_scan) {
   p.out = op_ptr<void>(a[17]); p.ldo = a[19];
   p.inner = (int)a[21]; p.N = (int)a[22];
   if (p.N < 1 || p.N > 256) GB_FAIL(GB_ERR_ARG, "selective_scan: %d state entries a channel (1 to 256)", p.N);
-  p.vec_bc = p.N % 4 == 0 && p.ldbc % 4 == 0 && (a[4] & 15) == 0 && (a[5] & 15) == 0;
-  p.vec_x = p.inner % 4 == 0 && p.ldx % 4 == 0 && p.lddt % 4 == 0 && (a[0] & 15) == 0 && (a[2] & 15) == 0;
+  p.vec = p.N % 4 == 0 && p.ldbc % 4 == 0 && p.inner % 4 == 0 && p.ldx % 4 == 0 && p.lddt % 4 == 0 && p.ldz % 4 == 0 &&
+          ((a[0] | a[2] | a[4] | a[5] | a[7]) & 15) == 0;
 #define SEL(SPLIT, PER, FAST, TO)                                                                                       \
   do {                                                                                                                  \
-    constexpr size_t smem = sizeof(float) * SEL_TOKENS * (4 * SPLIT * PER + 6 * (SEL_THREADS / SPLIT));                 \
+    constexpr int smem = SelCfg<SPLIT, PER>::SMEM;                                                                      \
     static bool raised = false;            /* once, before any stream capture replays the launch */                    \
     if (!raised && smem > 48 * 1024) {                                                                                  \
       GB_CUDA((cudaFuncSetAttribute(selective_scan_kernel<SPLIT, PER, FAST, TO>,                                        \
-                                    cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)));                          \
+                                    cudaFuncAttributeMaxDynamicSharedMemorySize, smem)));                               \
       raised = true;                                                                                                    \
     }                                                                                                                   \
     gb_launch(selective_scan_kernel<SPLIT, PER, FAST, TO>, dim3(R, gb_div_up(p.inner, SEL_THREADS / SPLIT)),             \

@@ -41,6 +41,71 @@ __global__ void causal_conv_silu_kernel(const float* in, long long ld, const flo
   if (copy) copy[(size_t)t * ldcopy + c] = __float2bfloat16_rn(y);
 }
 
+// The same for rows that can be read in 16-byte pieces and few taps: a thread takes four channels and CONV_RUN
+// consecutive rows of the step, with the last K - 1 inputs sliding in registers (reloaded where a row begins another
+// request); the same arithmetic per value as above.
+constexpr int CONV_RUN = 8;
+
+__device__ __forceinline__ float4 conv_fma(float4 w, float4 v, float4 a) {
+  return make_float4(fmaf(w.x, v.x, a.x), fmaf(w.y, v.y, a.y), fmaf(w.z, v.z, a.z), fmaf(w.w, v.w, a.w));
+}
+
+template <int K>
+__global__ void __launch_bounds__(128)
+causal_conv_silu_run_kernel(const float* in, long long ld, const float* __restrict__ taps, const float* __restrict__ bias,
+                            const float* state, long long slot_stride, const int* slot_ids, const int* tok_req,
+                            const int* q_start, float* out, long long ldo, int n, int C, bf16* copy, long long ldcopy) {
+  pdl_trigger();
+  const int c = 4 * (blockIdx.x * blockDim.x + threadIdx.x);
+  if (c >= C) return;
+  const int t0 = blockIdx.y * CONV_RUN, t1 = min(n, t0 + CONV_RUN);
+  float4 w[K];
+#pragma unroll
+  for (int j = 0; j < K; ++j)
+    w[j] = make_float4(taps[(size_t)c * K + j], taps[(size_t)(c + 1) * K + j], taps[(size_t)(c + 2) * K + j],
+                       taps[(size_t)(c + 3) * K + j]);
+  const float4 b = bias ? *reinterpret_cast<const float4*>(bias + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+  pdl_wait();
+  float4 x[CONV_RUN];                                     // (all rows of the run are requested together)
+#pragma unroll
+  for (int u = 0; u < CONV_RUN; ++u)
+    if (t0 + u < t1) x[u] = *reinterpret_cast<const float4*>(in + (size_t)(t0 + u) * ld + c);
+  float4 win[K];                                          // win[0 .. K-2]: the inputs before the row
+  int req = -1;
+#pragma unroll
+  for (int u = 0; u < CONV_RUN; ++u) {
+    const int t = t0 + u;
+    if (t >= t1) break;
+    const int r = tok_req[t];
+    if (r != req) {
+      req = r;
+      const int first = q_start[r], li = t - first;
+      const float* st = state + (size_t)slot_ids[r] * slot_stride + c;
+#pragma unroll
+      for (int j = 0; j < K - 1; ++j) {
+        const int s = li - (K - 1) + j;
+        win[j] = s >= 0 ? *reinterpret_cast<const float4*>(in + (size_t)(first + s) * ld + c)
+                        : *reinterpret_cast<const float4*>(st + (size_t)(K - 1 + s) * C);
+      }
+    }
+    win[K - 1] = x[u];
+    float4 acc = b;
+#pragma unroll
+    for (int j = 0; j < K; ++j) acc = conv_fma(w[j], win[j], acc);
+#pragma unroll
+    for (int j = 0; j < K - 1; ++j) win[j] = win[j + 1];
+    const float4 y = make_float4(hy_silu(acc.x), hy_silu(acc.y), hy_silu(acc.z), hy_silu(acc.w));
+    *reinterpret_cast<float4*>(out + (size_t)t * ldo + c) = y;
+    if (copy) {
+      __nv_bfloat162 lo = __floats2bfloat162_rn(y.x, y.y), hi = __floats2bfloat162_rn(y.z, y.w);
+      uint2 pk;
+      pk.x = *reinterpret_cast<unsigned*>(&lo);
+      pk.y = *reinterpret_cast<unsigned*>(&hi);
+      *reinterpret_cast<uint2*>(copy + (size_t)t * ldcopy + c) = pk;
+    }
+  }
+}
+
 // A step in which every request brings one token: convolution and state in one kernel, a thread per (request, channel)
 // (the same arithmetic as in the two kernels around it).
 __global__ void causal_conv_silu_decode_kernel(const float* in, long long ld, const float* __restrict__ taps,
@@ -329,10 +394,22 @@ GB_OP(gb_op_causal_conv_silu) {
     GB_CHECK_LAUNCH("causal_conv_silu (one token each)");
     return 1;
   }
+  const bool runs = K >= 2 && K <= 4 && C % 4 == 0 && a[1] % 4 == 0 && a[5] % 4 == 0 && a[11] % 4 == 0 && a[17] % 4 == 0 &&
+                    ((a[0] | a[3] | a[4] | a[10]) & 15) == 0 && (a[16] & 7) == 0 && gb_div_up(n, CONV_RUN) <= 65535;
+#define CONV_RUNS(K_)                                                                                                   \
+  gb_launch(causal_conv_silu_run_kernel<K_>, dim3(gb_div_up(C, 4 * 128), gb_div_up(n, CONV_RUN)), dim3(128), 0,          \
+            ctx->stream, op_ptr<const float>(a[0]), a[1], op_ptr<const float>(a[2]), op_ptr<const float>(a[3]),          \
+            op_ptr<const float>(a[4]), a[5], op_ptr<const int>(a[6]), op_ptr<const int>(a[7]), op_ptr<const int>(a[8]),  \
+            op_ptr<float>(a[10]), a[11], n, C, op_ptr<bf16>(a[16]), a[17])
+  if (runs && K == 2) CONV_RUNS(2);
+  else if (runs && K == 3) CONV_RUNS(3);
+  else if (runs && K == 4) CONV_RUNS(4);
+  else
   gb_launch(causal_conv_silu_kernel, dim3(gb_div_up((long long)n * C, 256)), dim3(256), 0, ctx->stream,
             op_ptr<const float>(a[0]), a[1], op_ptr<const float>(a[2]), op_ptr<const float>(a[3]), op_ptr<const float>(a[4]),
             a[5], op_ptr<const int>(a[6]), op_ptr<const int>(a[7]), op_ptr<const int>(a[8]), op_ptr<float>(a[10]), a[11], n,
             C, K, op_ptr<bf16>(a[16]), a[17]);
+#undef CONV_RUNS
   GB_CHECK_LAUNCH("causal_conv_silu");
   if (K == 1) return 1;
   gb_launch(conv_state_update_kernel, dim3(gb_div_up((long long)R * C, 256)), dim3(256), 0, ctx->stream,

@@ -198,14 +198,14 @@ int run_op(Walk& w, const PlanOp& o, bool force = false) {
       // symbol), a8 n, a9 k, a10 kernel (0 tensor cores, 1 FFMA), a11 mode (0 bf16, 1 f32, 2 add into f32, 3 SwiGLU),
       // a12 x dtype, a13 W dtype, a14 out dtype; mode 3 with f0 != 0: the gated unit's constants f0 alpha, f1 limit
       // (0: none), f2 what is added to u (all zero: SwiGLU), a15 the bits of a 32-bit float: the cubic term inside the
-      // gate's sigmoid (0: none)
+      // gate's sigmoid (0: none); mode 0: a16 a function of the finished sums (0: none, 1: the square of relu)
       const bool glu = a[11] == 3 && o.f[0] != 0.0;
       const int M = (int)val(w, a[7]);
       if (M <= 0) return 0;
       const float* bias = ptr<const float>(w, a[4]);
       const PlanOp* lazy = (o.flags & LF_NORMED) ? w.lazy_norm : nullptr;
       w.lazy_norm = nullptr;
-      if (a[10] == 0 && !glu && M <= w.decode_products &&
+      if (a[10] == 0 && !glu && a[16] == 0 && M <= w.decode_products &&
           ((LinearDecodeSupportedFn)g_fn[F_LINEAR_DECODE_SUPPORTED])(M, ptr<const void>(w, a[2]), a[3], (int)a[9])) {
         // up to 64 rows: K is split inside a cluster, and a norm that was left out runs inside the product
         const int n = (int)a[8], k = (int)a[9];
@@ -248,7 +248,7 @@ int run_op(Walk& w, const PlanOp& o, bool force = false) {
                            ((o.flags & LF_PARTIALS_IF_ONE_EACH) && one_each);
         // a large unsplit product into the residual stream is deferred as a whole (ops.DEFER_WHOLE_ROWS)
         const bool whole = (o.flags & LF_RESIDUAL) && splits == 1 && M >= w.defer_whole_rows;
-        const bool defer = (wants && splits > 1 && (a[11] == 0 || a[11] == 2)) || whole;
+        const bool defer = (wants && splits > 1 && a[11] <= 2 && a[16] == 0) || whole;
         if (glu)
           PLAN_CALL(w, F_LINEAR_TC_GLU, ((LinearTcGluFn)g_fn[F_LINEAR_TC_GLU])(
               ptr<const void>(w, a[0]), a[1], ptr<const void>(w, a[2]), a[3], bias, ptr<void>(w, a[5]), (int)a[11], a[6],
@@ -257,8 +257,8 @@ int run_op(Walk& w, const PlanOp& o, bool force = false) {
         else
         PLAN_CALL(w, F_LINEAR_TC, ((LinearTcFn)g_fn[F_LINEAR_TC])(
             ptr<const void>(w, a[0]), a[1], ptr<const void>(w, a[2]), a[3], bias, ptr<void>(w, a[5]), (int)a[11], a[6],
-            M, n, k, (splits > 1 || whole) ? w.ws : nullptr, whole ? 2 : (defer ? 1 : 0), w.tc_flags, w.status,
-            w.stream));
+            M, n, k, (splits > 1 || whole) ? w.ws : nullptr, whole ? 2 : (defer ? 1 : 0),
+            w.tc_flags | (int)(a[16] << 8), w.status, w.stream));
         if (o.flags & LF_RESIDUAL) {
           w.pend_splits = defer ? splits : 0;
           w.pend_bias = bias;
@@ -402,7 +402,13 @@ int run_registered(Walk& w, const PlanOp& o) {
   }
   w.ssq_parts = 0;
   w.lazy_norm = nullptr;
-  w.part_splits = 0;
+  const bool parts = (o.flags & GB_OP_TAKES_PARTIALS) != 0 && w.part_splits > 0;
+  if (w.part_splits > 0 && !parts) {
+    snprintf(gb_error_buffer(), 512, "gb_plan_run: '%s' does not take the partial tiles the product in front left",
+             g_registered[i].name);
+    w.failed_lib = 2;
+    return GB_ERR_ARG;
+  }
   long long a[24];
   for (int j = 0; j < 24; ++j) a[j] = val(w, o.a[j]);
   GbPlanCtx ctx;
@@ -416,6 +422,10 @@ int run_registered(Walk& w, const PlanOp& o) {
   ctx.pend_splits = takes ? w.pend_splits : 0;
   ctx.pend_bias = takes ? w.pend_bias : nullptr;
   w.pend_splits = 0;
+  ctx.part = parts ? w.ws : nullptr;
+  ctx.part_splits = parts ? w.part_splits : 0;
+  ctx.part_bias = parts ? w.part_bias : nullptr;
+  w.part_splits = 0;
   const int rc = g_registered[i].fn(&ctx, a, o.f, o.flags);
   if (rc < 0) {
     snprintf(gb_error_buffer(), 512, "gb_plan_run: the registered operation '%s' failed with code %d",

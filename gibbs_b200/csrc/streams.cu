@@ -54,6 +54,8 @@ __device__ __forceinline__ void store_normed(void* out, int dtype, size_t at, co
 struct StreamParams {
   float* x; long long ldx;                 // [rows, streams * dim]
   const float* y; long long ldy;           // a sublayer's output (mixing only)
+  const float* part; int splits;           // or its partial tiles [splits][rows][dim], added up in this order
+  long long part_stride; const float* part_bias;
   const float* mix;                        // [streams][streams], from x to
   const float* out_w;                      // [streams]
   const float* in_w;                       // [streams] weights of the next reader, or null: ones
@@ -120,7 +122,28 @@ __global__ void stream_kernel(StreamParams p, int streams) {
       if (S > 0 || s < n_s) old[s].load(x + (size_t)s * p.dim + (size_t)i * VEC);
     if constexpr (MIX) {
       Piece<VEC> yy, now[CAP];
-      yy.load(y + (size_t)i * VEC);
+      if (p.part == nullptr) {
+        yy.load(y + (size_t)i * VEC);
+      } else {
+        const float* at = p.part + (size_t)r * p.dim + (size_t)i * VEC;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) yy.v[e] = 0.f;
+        for (int s0 = 0; s0 < p.splits; s0 += 4) {         // (four requested together, added in order)
+          Piece<VEC> t[4];
+#pragma unroll
+          for (int u = 0; u < 4; ++u) t[u].load(at + (size_t)min(s0 + u, p.splits - 1) * p.part_stride);
+#pragma unroll
+          for (int u = 0; u < 4; ++u)
+            if (s0 + u < p.splits) {
+#pragma unroll
+              for (int e = 0; e < VEC; ++e) yy.v[e] += t[u].v[e];
+            }
+        }
+        if (p.part_bias) {
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) yy.v[e] += p.part_bias[(size_t)i * VEC + e];
+        }
+      }
 #pragma unroll
       for (int t = 0; t < CAP; ++t) {
         if (S == 0 && t >= n_s) break;
@@ -189,7 +212,7 @@ __global__ void stream_kernel(StreamParams p, int streams) {
 template <bool MIX>
 int launch_streams(const StreamParams& p, int n, int streams, cudaStream_t stream, const char* what) {
   if (streams < 1 || streams > MAX_STREAMS) GB_FAIL(GB_ERR_ARG, "%s: %d streams (1 to %d)", what, streams, MAX_STREAMS);
-  const uintptr_t bits = (uintptr_t)p.x | (uintptr_t)p.y | (uintptr_t)p.gain;
+  const uintptr_t bits = (uintptr_t)p.x | (uintptr_t)p.y | (uintptr_t)p.gain | (uintptr_t)p.part;
   const bool vec = p.dim % 4 == 0 && p.ldx % 4 == 0 && p.ldy % 4 == 0 && (bits & 15) == 0 &&
                    ((uintptr_t)p.out & (p.out_dtype == GB_BF16 ? 7 : 15)) == 0;
   const int pieces = vec ? p.dim / 4 : p.dim;
@@ -228,11 +251,16 @@ GB_OP(gb_op_stream_read) {
 // a0 x (f32 [rows, streams * dim], changed in place), a1 its row stride, a2 y (f32 [rows, dim]), a3 its row stride,
 // a4 mix [streams][streams] (f32: from the first index to the second), a5 weights of y [streams], a6 rows, a7 dim,
 // a8 streams; what the next sublayer reads of the new streams: a9 its weights [streams] or 0: ones, a10 its norm's gain
-// or 0: nothing is read, a11 out [rows, dim], a12 out dtype; f0 that norm's eps
+// or 0: nothing is read, a11 out [rows, dim], a12 out dtype; f0 that norm's eps.  A record with GB_OP_TAKES_PARTIALS: y
+// may be the partial tiles of the product in front
 GB_OP(gb_op_stream_mix) {
   if (a[6] <= 0) return 0;
   StreamParams p{};
   p.x = op_ptr<float>(a[0]); p.ldx = a[1]; p.y = op_ptr<const float>(a[2]); p.ldy = a[3];
+  if (ctx->part_splits > 0) {
+    p.part = ctx->part; p.splits = ctx->part_splits;
+    p.part_stride = a[6] * a[7]; p.part_bias = ctx->part_bias;
+  }
   p.mix = op_ptr<const float>(a[4]); p.out_w = op_ptr<const float>(a[5]);
   p.dim = (int)a[7]; p.in_w = op_ptr<const float>(a[9]); p.gain = op_ptr<const float>(a[10]);
   p.out = op_ptr<void>(a[11]); p.out_dtype = (int)a[12]; p.eps = (float)f[0];

@@ -174,11 +174,13 @@ class PlanBuilder:
         return out
 
     def linear(self, x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], out, mode: str,
-               rows_symbol: int = S_N, partials: str = "", role: str = "", glu=None) -> torch.Tensor:
+               rows_symbol: int = S_N, partials: str = "", role: str = "", glu=None, act: int = 0) -> torch.Tensor:
         """out (+)= x W^T + b.  mode: 'plain' (out in its own dtype), 'residual' (adds into the
         float32 residual; partial sums may be left to the next norm) or 'swiglu'.  ``partials``:
         '' | 'one_each' | 'always': when K is split, leave the partial tiles to the next
-        operation (a short convolution or q/k kernel that adds them itself).  ``glu`` (mode
+        operation (a short convolution or q/k kernel that adds them itself; or, for a 32-bit output, a registered
+        operation whose flags say that it takes them).  ``act`` (a bfloat16 output on the tensor cores): a function of
+        the finished sums, applied before they are rounded (``ops.EPILOGUES``).  ``glu`` (mode
         'swiglu'): (alpha, limit, add[, cubic]) of the gated unit g' sigmoid(alpha (g' + cubic g'^3)) (u' + add)
         with g' = min(g, limit), u' = clamp(u, -limit, limit); limit 0: none.  None: SwiGLU."""
         n, k = weight.shape
@@ -206,7 +208,9 @@ class PlanBuilder:
             code = 1                                                   # the step's float32 logits
         else:
             code = 0 if out.dtype == torch.bfloat16 else 1
-            if partials and use_tc and out.dtype == torch.bfloat16:
+            if act and (not use_tc or out.dtype != torch.bfloat16 or partials):
+                raise NotPlannable("a function in a product's epilogue: bfloat16 out on the tensor cores, not left in parts")
+            if partials and use_tc:
                 flags |= LF_PARTIALS if partials == "always" else LF_PARTIALS_IF_ONE_EACH
         if use_tc:
             # how K is split changes with the tile width (at 16, 32 and 64 rows) and then with
@@ -227,7 +231,7 @@ class PlanBuilder:
                              n if isinstance(out, int) else out.stride(0), sym(rows_symbol), n, k, 0 if use_tc else 1,
                              code, ops.dtype_code(x.dtype), ops.dtype_code(weight.dtype),
                              ops.F32 if isinstance(out, int) else ops.dtype_code(out.dtype),
-                             0 if glu is None or len(glu) < 4 else int(np.float32(glu[3]).view(np.uint32))],
+                             0 if glu is None or len(glu) < 4 else int(np.float32(glu[3]).view(np.uint32)), int(act)],
                   [] if glu is None else [float(v) for v in glu[:3]], flags=flags, label="linear:" + (role or mode))
         return out
 

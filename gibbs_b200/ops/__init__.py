@@ -266,8 +266,12 @@ _TC_FLAGS = 1 if os.environ.get("GIBBS_B200_EVICT_FIRST", "1") != "0" else 0
 DEFER_WHOLE_ROWS = 256
 
 
+# functions a product with a bfloat16 output can apply to its finished sums (the ``act`` of ``linear_tc``)
+EPILOGUES = {"relu2": 1}
+
+
 def linear_tc(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor,
-              accumulate: bool = False, swiglu: bool = False, defer: bool = False, glu=None):
+              accumulate: bool = False, swiglu: bool = False, defer: bool = False, glu=None, act: int = 0):
     """out (+)= a @ w.T (+ bias) for bfloat16 a and w on the tensor cores
     (csrc/gemm_tc.cu).  ``swiglu``: w holds gate and up rows alternating in
     blocks of 64 and out [m, n/2] gets (g * sigmoid(g)) * u.
@@ -276,7 +280,8 @@ def linear_tc(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], ou
     [splits, m, n] are returned instead, for the caller's next kernel to add
     (without the bias).  Otherwise returns ``out``.
     ``glu`` (with ``swiglu``): (alpha, limit, add[, cubic]) of the gated unit g' sigmoid(alpha (g' + cubic g'^3)) (u' + add)
-    with g' = min(g, limit), u' = clamp(u, -limit, limit); limit 0: none."""
+    with g' = min(g, limit), u' = clamp(u, -limit, limit); limit 0: none.
+    ``act`` (a plain bfloat16 product): a function of the finished sums (``EPILOGUES``), taken in 32-bit."""
     # (this wrapper runs some seventy times a step: its checks are the cheap ones)
     lib = _LIBS.get("tensorcore") or _lib("tensorcore")
     m, k = a.shape
@@ -323,7 +328,7 @@ def linear_tc(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], ou
         _c_void(out.data_ptr()), _c_int(mode), _c_ll(out.stride(0) if m > 1 else max(out.stride(0), n_out)), _c_int(m),
         _c_int(n), _c_int(k), _NULL if ws is None else _c_void(ws.data_ptr()),
         _c_int(2) if whole else (_ONE if defer else _ZERO),
-        _c_int(_TC_FLAGS),
+        _c_int(_TC_FLAGS | (act << 8)),
         _status_ptr(a), _STREAM if _STREAM is not None else _stream(), *extra)
     if rc < 0:
         check(lib, rc)

@@ -243,6 +243,7 @@ class HyperResidual(Block):
         return False
 
     def _run(self, rn, x, caches):
+        rn.partial_branches = True                 # (the mixing adds up the partial tiles a sublayer's last product leaves)
         h, self._handed = self._handed, None
         if h is None:
             h = self.mixer_streams.read(rn, x, self.mixer_norm)

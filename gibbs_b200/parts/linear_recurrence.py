@@ -54,7 +54,7 @@ class RecurrentHeads(BranchPart, Mixer):
         rn.linear(h, self.fused, None, u, role="rec_in")
         o = rn.buffer("rec_heads", self.heads_width)
         self.mix_heads(rn, u, caches, o)
-        (rn.add_linear if accumulate else rn.linear)(o, self.out_weight, None, out, role="rec_out")
+        rn.branch_linear(o, self.out_weight, None, out, accumulate, role="rec_out")
 
 
 class GatedWriteRecurrence(RecurrentHeads):
@@ -131,7 +131,7 @@ class MatrixMemory(RecurrentHeads):
         slots = rn.slots(rec)
         rn.op("exp_gates", [at(ic), u.stride(0), at(ic + H), u.stride(0), keep(rn, self.i_bias), keep(rn, self.f_bias),
                             keep(rn, top.state), top.state.stride(0), slots, rn.q_start, rn.q_len,
-                            *[t.data_ptr() for t in gates], rn.R, H], [self.cap])
+                            *[t.data_ptr() for t in gates], rn.R, H, rn.N], [self.cap])
         decay, write, floor = gates
         y = rn.buffer("rec_read", H * vdim, torch.float32)
         nq = rn.buffer("mm_norm", H, torch.float32)

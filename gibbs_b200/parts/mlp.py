@@ -5,7 +5,8 @@
 "relu", "relu2" (the square of relu).  The first product writes 32-bit values, the function (and the gate's
 product with the up rows) is taken in 32-bit and rounded to the compute dtype
 for the second product, which adds into the residual stream or writes for an
-arrangement that takes the output as it is.
+arrangement that takes the output as it is.  In bfloat16 the first product's
+epilogue applies a function it knows (``ops.EPILOGUES``).
 """
 from __future__ import annotations
 
@@ -21,7 +22,8 @@ ACTIVATIONS = {"gelu": 0, "gelu_tanh": 1, "silu": 2, "relu": 3, "relu2": 4, "non
 # act(g) = g * sigmoid(alpha * (g + cubic * g^3)) for the functions that have this form: (alpha, cubic).  The tanh form
 # of gelu has it because 0.5 (1 + tanh y) = sigmoid(2 y), with y = sqrt(2 / pi) (g + 0.044715 g^3).
 SIGMOID_FORMS = {"silu": (1.0, 0.0), "gelu_tanh": (1.5957691216057308, 0.044715)}
-FUSE_GATED_UNIT = True             # (the tests switch it off to compare the two ways)
+FUSE_GATED_UNIT = True             # (the tests switch them off to compare the two ways)
+FUSE_ACT = True
 
 
 class DenseMLP(BranchPart, FeedForward):
@@ -41,8 +43,11 @@ class DenseMLP(BranchPart, FeedForward):
         act = params.get("act", "gelu")
         if act not in ACTIVATIONS:
             raise ValueError(f"unknown activation '{act}'; known: {sorted(ACTIVATIONS)}")
-        self.act = ACTIVATIONS[act]
+        self.act, self.act_name = ACTIVATIONS[act], act
         self.up, self.down = tensors["up"].contiguous(), tensors["down"].contiguous()
+        # in bfloat16 the first product's epilogue applies a function it knows
+        self.fused = (FUSE_ACT and act in ops.EPILOGUES and rt.dtype == torch.bfloat16 and self.up.dtype == torch.bfloat16
+                      and self.hidden % 8 == 0)
         f32 = lambda n: tensors[n].to(torch.float32).contiguous() if params.get("bias") else None
         self.up_bias, self.down_bias = f32("up.b"), f32("down.b")
 
@@ -50,12 +55,15 @@ class DenseMLP(BranchPart, FeedForward):
         return tuple(set(ops.linear_libraries(self.up.dtype, self.rt.dtype)) | {"core", hybrid.LIBRARY})
 
     def run(self, rn: Runner, h, out, caches=None, accumulate: bool = False):
+        act = rn.buffer("mlp_act", self.inner)
+        if self.fused:
+            rn.act_linear(h, self.up, self.up_bias, act, self.act_name, role="mlp_up")
+            return rn.branch_linear(act, self.down, self.down_bias, out, accumulate, role="mlp_down")
         z = rn.buffer("mlp_up", self.inner, torch.float32)
         rn.linear(h, self.up, self.up_bias, z, role="mlp_up")
-        act = rn.buffer("mlp_act", self.inner)
         rn.op("act_rows", [z.data_ptr(), z.stride(0), act.data_ptr(), ops.dtype_code(act.dtype), act.stride(0), rn.N,
                            self.inner, self.act])
-        (rn.add_linear if accumulate else rn.linear)(act, self.down, self.down_bias, out, role="mlp_down")
+        rn.branch_linear(act, self.down, self.down_bias, out, accumulate, role="mlp_down")
 
 
 class GatedMLP(BranchPart, FeedForward):

@@ -75,7 +75,7 @@ class ParallelMixers(BranchPart, Mixer):
             side.mix_heads(rn, u[:, self.in_cols[i]:self.in_cols[i + 1]], caches[at:at + n],
                        o[:, self.out_cols[i]:self.out_cols[i + 1]], factor)
             at += n
-        (rn.add_linear if accumulate else rn.linear)(o, self.out_weight, None, out, role="par_out")
+        rn.branch_linear(o, self.out_weight, None, out, accumulate, role="par_out")
 
 
 register_part("mixer", "parallel_mixers", ParallelMixers)

@@ -44,6 +44,18 @@ class Runner:
         blocks of 64 (``parts.linear.interleave_gate_up``); ``glu`` = (alpha, limit, add)."""
         raise NotImplementedError
 
+    def act_linear(self, x, weight, bias, out, act: str, role: str = "") -> None:
+        """out = act(x weight^T (+ bias)) on the tensor cores, for a bfloat16 ``out`` and a function in
+        ``ops.EPILOGUES``: the product's epilogue applies it to the 32-bit sums."""
+        raise NotImplementedError
+
+    # set by an arrangement whose next kernel reads a sublayer's output and can add up partial tiles itself
+    partial_branches = False
+
+    def branch_linear(self, x, weight, bias, out, accumulate: bool = False, role: str = "") -> None:
+        """A sublayer's last product: written into ``out``, or added (``add_linear``)."""
+        (self.add_linear if accumulate else self.linear)(x, weight, bias, out, role=role)
+
     def op(self, name: str, a, f=(), label: str = "", flags: int = 0) -> None:
         raise NotImplementedError
 
@@ -76,6 +88,9 @@ class Eager(Runner):
 
     def glu_linear(self, x, weight, out, glu, role=""):
         ops.linear_tc(x[:self.N] if x.shape[0] != self.N else x, weight, None, out, swiglu=True, glu=glu)
+
+    def act_linear(self, x, weight, bias, out, act, role=""):
+        ops.linear_tc(x[:self.N] if x.shape[0] != self.N else x, weight, bias, out, act=ops.EPILOGUES[act])
 
     def op(self, name, a, f=(), label="", flags=0):
         hybrid.call(name, a, f, flags=flags, device=self.rt.device)
@@ -113,6 +128,15 @@ class Planned(Runner):
 
     def glu_linear(self, x, weight, out, glu, role=""):
         self.plan.linear(x, weight, None, out, "swiglu", role=role or "glu", glu=glu)
+
+    def act_linear(self, x, weight, bias, out, act, role=""):
+        self.plan.linear(x, weight, bias, out, "plain", role=role or "act", act=ops.EPILOGUES[act])
+
+    def branch_linear(self, x, weight, bias, out, accumulate=False, role=""):
+        if accumulate or not self.partial_branches:
+            return super().branch_linear(x, weight, bias, out, accumulate, role)
+        # (the sum of the partial tiles in their order is what the product's own reduction writes)
+        self.plan.linear(x, weight, bias, out, "plain", role=role or "plain", partials="always")
 
     def op(self, name, a, f=(), label="", flags=0):
         self.plan.emit(hybrid.plan_id(name), list(a), list(f), flags=flags, label=label or name)

@@ -88,7 +88,7 @@ class SelectiveScanMixer(BranchPart, Mixer):
                                  keep(rn, self.dt_bias), keep(rn, self.a_log), keep(rn, self.d_skip), keep(rn, rec.state),
                                  rec.state.stride(0), slots, rn.q_start, rn.q_len, y.data_ptr(), ops.dtype_code(y.dtype),
                                  y.stride(0), rn.R, inner, N])
-        rn.linear(y, self.w_out, None, out, role="scan_out")
+        rn.branch_linear(y, self.w_out, None, out, role="scan_out")
 
 
 register_part("mixer", "selective_scan", SelectiveScanMixer)

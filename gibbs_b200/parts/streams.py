@@ -52,7 +52,8 @@ class HyperConnection(Part):
         return out
 
     def add(self, rn, x: torch.Tensor, y: torch.Tensor, then=None):
-        """Mix the streams and add the sublayer's output y (float32 [rows, dim]).  ``then`` = (the next sublayer's
+        """Mix the streams and add the sublayer's output y (float32 [rows, dim]; in a plan the product in front may have
+        left it as partial tiles, which the kernel adds up).  ``then`` = (the next sublayer's
         HyperConnection, its norm): what that sublayer reads is taken in the same kernel and returned."""
         a = [x.data_ptr(), x.stride(0), y.data_ptr(), y.stride(0), keep(rn, self.mix_weights), keep(rn, self.write_weights),
              rn.N, self.dim, self.streams]
@@ -62,7 +63,7 @@ class HyperConnection(Part):
             out = rn.buffer("normed", self.dim)
             a += [keep(rn, following.read_weights), keep(rn, norm.gain), out.data_ptr(), ops.dtype_code(out.dtype)]
             f = [norm.eps]
-        rn.op("stream_mix", a, f, label="stream_mix")
+        rn.op("stream_mix", a, f, label="stream_mix", flags=hybrid.TAKES_PARTIALS)
         return out
 
 

@@ -791,3 +791,22 @@ def test_what_a_layer_reads_taken_by_the_layer_in_front_changes_nothing(dtype, m
         outs.append(run_trace_on_engine(eng, steps))
     for rid in reqs:
         assert np.array_equal(outs[0][rid], outs[1][rid]), rid
+
+
+@pytest.mark.parametrize("d,ff,rows", [(128, 256, 70), (96, 130, 5), (336, 64, 300), (64, 1024, 33), (2048, 512, 3), (512, 2048, 600)])
+def test_squared_relu_in_the_epilogue_of_its_product_against_the_kernel_of_its_own(d, ff, rows, monkeypatch):
+    """bfloat16: the first product applies the function to its 32-bit sums; against the 32-bit product followed by the
+    activation kernel (the same bits, as both round the same value once), also with K split and ragged edges."""
+    from gibbs_b200.parts import mlp
+    g = gen(31)
+    W = {"up": bf(torch.randn(ff, d, generator=g) / d ** 0.5), "down": bf(torch.randn(d, ff, generator=g) / ff ** 0.5)}
+    h = bf(torch.randn(rows, d, generator=g) * 1.5)
+    want = plain.dense_mlp(h.double(), dbl(W))
+    outs = {}
+    for fuse in (True, False):
+        monkeypatch.setattr(mlp, "FUSE_ACT", fuse)
+        part = make_part("feed_forward", "dense_mlp", {"hidden": d, "inner": ff, "act": "relu2"}, W, torch.bfloat16)
+        assert part.fused == fuse
+        outs[fuse] = PartHarness(part).feed("r", h)
+        check_rows(outs[fuse], want, "bfloat16", what=f"fused {fuse}", tol=1.5e-2)
+    assert rel_rows(outs[True], outs[False]).max() < 1e-3
