@@ -33,6 +33,10 @@ struct ScanParams {
   float* nq;                               // [t, heads]: n . q * q_scale, or null: no normaliser
   int H, dim, vdim, cols;                  // cols: vdim, or vdim + 1 with the normaliser
   float q_scale;
+  // a long portion in segments of seg_len tokens, computed side by side (SEGMENTS below)
+  int seg_len, segs;
+  float* seg_state;                        // [requests][segs][heads][cols][dim]
+  float* seg_decay;                        // [requests][segs][heads * dim] or [requests][segs][heads]
   int vec_rows, vec_v;                     // rows of q, k, g (of v) can be copied in 16-byte pieces
 };
 
@@ -49,6 +53,14 @@ template <int LEFT> __device__ __forceinline__ void ls_wait() {
 // together, every exchange halving what a lane still carries: one shuffle a token instead of log2(SPLIT).  A portion's
 // last tokens, fewer than GROUP, are added one by one in the same order of additions, so how a prompt is cut does not
 // change a bit.
+//
+// WHOLE: a block walks its request's whole portion.  A long prompt of one request has too few columns to fill the GPU, and
+// a warp that is alone on its scheduler waits for its own latencies: the portion is then cut into segments.  ENDS
+// computes, for every segment but the last, the state it leaves (from the slot's state for the first segment, from
+// zero for the others) and the product of its decays, without read-outs; SEGMENTS then starts every segment from
+// S = S_1;  S <- decay_j S + S_j for the segments j in between, and computes read-outs.  (The first segment's start
+// is copied aside by ENDS, because the last segment writes the slot.)
+enum ScanMode : int { WHOLE = 0, ENDS = 1, SEGMENTS = 2 };
 constexpr int LS_STAGES = 4;
 
 template <int SPLIT, int PER, int TOK, bool CHANNEL>
@@ -58,7 +70,7 @@ struct ScanCfg {
   static constexpr int SMEM = LS_STAGES * BUF * 4;
 };
 
-template <int SPLIT, int PER, int TOK, bool CHANNEL>
+template <int SPLIT, int PER, int TOK, bool CHANNEL, int MODE>
 __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(ScanParams p) {
   using C = ScanCfg<SPLIT, PER, TOK, CHANNEL>;
   constexpr int NR = C::NR, COLS = C::COLS, Q4 = PER / 4, ROWS = C::ROWS, BUF = C::BUF;
@@ -66,11 +78,26 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(ScanParams p) {
   extern __shared__ __align__(16) float ls_sm[];         // [LS_STAGES][BUF]
   pdl_trigger();
   const int col = threadIdx.x / SPLIT, q = threadIdx.x % SPLIT;
-  const int r = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * COLS, c = c0 + col;
+  const int r = MODE == WHOLE ? blockIdx.x : blockIdx.x / p.segs, seg = MODE == WHOLE ? 0 : blockIdx.x - r * p.segs;
+  const int h = blockIdx.y, c0 = blockIdx.z * COLS, c = c0 + col;
   const bool active = c < p.cols;
   const bool counts = c == p.vdim;                       // the normaliser's column: its value is always 1
-  const int first = p.q_start[r], len = p.q_len[r];
+  const int all = p.q_len[r];                            // the portion
+  const int first = p.q_start[r] + seg * p.seg_len;
+  const int len = MODE == WHOLE ? all : min(p.seg_len, all - seg * p.seg_len);
+  const bool last = MODE == WHOLE || (seg + 1) * p.seg_len >= all;
+  if (len <= 0 || (MODE == ENDS && last)) {              // (nobody starts from what the last segment leaves)
+    pdl_wait();                                          // a launch all of whose blocks leave still ends behind the one in front
+    return;
+  }
   float* S = p.state + (size_t)p.slot_ids[r] * p.slot_stride + ((size_t)h * p.cols + (active ? c : 0)) * p.dim;
+  // where segment i of this request starts from, for this column: the slot's state (0), the state segment 0 leaves (1), or
+  // what segment i - 1 leaves when it starts from zero
+  const size_t seg_stride = (size_t)p.H * p.cols * p.dim;
+  float* starts = MODE == WHOLE ? nullptr
+                                : p.seg_state + (size_t)r * p.segs * seg_stride + ((size_t)h * p.cols + (active ? c : 0)) * p.dim;
+  const size_t decay_stride = CHANNEL ? (size_t)p.H * p.dim : (size_t)p.H;
+  float* decays = MODE == WHOLE ? nullptr : p.seg_decay + (size_t)r * p.segs * decay_stride + (CHANNEL ? h * p.dim : h);
   const int vcols = max(0, min(COLS, p.vdim - c0));
   if (p.dim < NR || vcols < COLS)                        // what is never copied stays zero
     for (int i = threadIdx.x; i < LS_STAGES * BUF; i += LS_THREADS) ls_sm[i] = 0.f;
@@ -94,6 +121,7 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(ScanParams p) {
         r_src[j] = (which == 0 ? p.q : which == 1 ? p.k : p.g) + (size_t)first * r_ld[j] + (size_t)h * p.dim + c4;
         r_dst[j] = which * TOK * NR + c4;
         r_step[j] = NR;
+        if (MODE == ENDS && which == 0) r_src[j] = nullptr;        // (no read-out: no queries)
       } else if (i < ROWS * pieces + (vcols >> 2)) {
         const int c4 = 4 * (i - ROWS * pieces);
         r_ld[j] = p.ldv;
@@ -105,23 +133,58 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(ScanParams p) {
   }
   pdl_wait();
   const bool vec_state = (p.dim & 3) == 0 && (p.slot_stride & 3) == 0 && ((uintptr_t)p.state & 15) == 0;
-  float s[PER];
+  float s[PER] = {};
+  auto fetch4 = [&](const float* src, int n) {            // entries n .. n + 3 of a column, 0 beyond dim
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (active && n < p.dim) {
+      if (vec_state) {
+        v = *reinterpret_cast<const float4*>(src + n);
+      } else {
+        v.x = src[n];
+        if (n + 1 < p.dim) v.y = src[n + 1];
+        if (n + 2 < p.dim) v.z = src[n + 2];
+        if (n + 3 < p.dim) v.w = src[n + 3];
+      }
+    }
+    return v;
+  };
+  auto store4 = [&](float* dst, int i) {
+    const int n = 4 * (q + SPLIT * i);
+    if (!active || n >= p.dim) return;
+    if (vec_state) {
+      *reinterpret_cast<float4*>(dst + n) = make_float4(s[4 * i], s[4 * i + 1], s[4 * i + 2], s[4 * i + 3]);
+    } else {
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (n + e < p.dim) dst[n + e] = s[4 * i + e];
+    }
+  };
 #pragma unroll
   for (int i = 0; i < Q4; ++i) {
     const int n = 4 * (q + SPLIT * i);
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (active && n < p.dim) {
-      if (vec_state) {
-        v = *reinterpret_cast<const float4*>(S + n);
-      } else {
-        v.x = S[n];
-        if (n + 1 < p.dim) v.y = S[n + 1];
-        if (n + 2 < p.dim) v.z = S[n + 2];
-        if (n + 3 < p.dim) v.w = S[n + 3];
+    if (MODE == WHOLE || (MODE == SEGMENTS && seg == 0 && last) || (MODE == ENDS && seg == 0)) {
+      v = fetch4(S, n);
+    } else if (MODE == SEGMENTS) {
+      v = fetch4(starts + (seg == 0 ? 0 : seg_stride), n);
+      for (int j = 2; j <= seg; ++j) {
+        const float4 e = fetch4(starts + j * seg_stride, n);
+        float4 d;
+        if (CHANNEL) {
+          d = fetch4(decays + (j - 1) * decay_stride, n);
+        } else {
+          const float dh = decays[(j - 1) * decay_stride];
+          d = make_float4(dh, dh, dh, dh);
+        }
+        v = make_float4(fmaf(d.x, v.x, e.x), fmaf(d.y, v.y, e.y), fmaf(d.z, v.z, e.z), fmaf(d.w, v.w, e.w));
       }
     }
     s[4 * i] = v.x; s[4 * i + 1] = v.y; s[4 * i + 2] = v.z; s[4 * i + 3] = v.w;
+    if (MODE == ENDS && seg == 0) store4(starts, i);
   }
+  float prod[MODE == ENDS ? (CHANNEL ? PER : 1) : 1];      // the product of the segment's decays
+#pragma unroll
+  for (int i = 0; i < (int)(sizeof(prod) / sizeof(float)); ++i) prod[i] = 1.f;
   __syncthreads();
 
   const int chunks = (len + TOK - 1) / TOK;
@@ -146,7 +209,7 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(ScanParams p) {
         const size_t row0 = (size_t)(first + t0);
         for (int tt = 0; tt < nt; ++tt) {
           for (int i = threadIdx.x; i < p.dim; i += LS_THREADS) {
-            gb_cp_async_4(Q + tt * NR + i, p.q + (row0 + tt) * p.ldq + (size_t)h * p.dim + i);
+            if (MODE != ENDS) gb_cp_async_4(Q + tt * NR + i, p.q + (row0 + tt) * p.ldq + (size_t)h * p.dim + i);
             gb_cp_async_4(Q + (TOK + tt) * NR + i, p.k + (row0 + tt) * p.ldk + (size_t)h * p.dim + i);
             if (CHANNEL) gb_cp_async_4(Q + (2 * TOK + tt) * NR + i, p.g + (row0 + tt) * p.ldg + (size_t)h * p.dim + i);
           }
@@ -184,12 +247,24 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(ScanParams p) {
       const float2 gw = *reinterpret_cast<const float2*>(GW + 4 * tt);
       if (weighted) v *= gw.y;
       float d0 = 0.f, d1 = 0.f, d2 = 0.f, d3 = 0.f;      // four chains, added in a fixed order
+      if (MODE == ENDS && !CHANNEL) prod[0] *= gw.x;
 #pragma unroll
       for (int i = 0; i < Q4; ++i) {
         const float4 k4 = *reinterpret_cast<const float4*>(K + tt * NR + 4 * SPLIT * i);
-        const float4 q4 = *reinterpret_cast<const float4*>(Q + tt * NR + 4 * SPLIT * i);
+        float4 q4 = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (MODE != ENDS) q4 = *reinterpret_cast<const float4*>(Q + tt * NR + 4 * SPLIT * i);
         float4 g4 = make_float4(gw.x, gw.x, gw.x, gw.x);
         if (CHANNEL) g4 = *reinterpret_cast<const float4*>(G + tt * NR + 4 * SPLIT * i);
+        if constexpr (MODE == ENDS) {
+          s[4 * i] = fmaf(g4.x, s[4 * i], k4.x * v);
+          s[4 * i + 1] = fmaf(g4.y, s[4 * i + 1], k4.y * v);
+          s[4 * i + 2] = fmaf(g4.z, s[4 * i + 2], k4.z * v);
+          s[4 * i + 3] = fmaf(g4.w, s[4 * i + 3], k4.w * v);
+          if constexpr (CHANNEL) {
+            prod[4 * i] *= g4.x; prod[4 * i + 1] *= g4.y; prod[4 * i + 2] *= g4.z; prod[4 * i + 3] *= g4.w;
+          }
+          continue;
+        }
         s[4 * i] = fmaf(g4.x, s[4 * i], k4.x * v);             d0 = fmaf(s[4 * i], q4.x, d0);
         s[4 * i + 1] = fmaf(g4.y, s[4 * i + 1], k4.y * v);     d1 = fmaf(s[4 * i + 1], q4.y, d1);
         s[4 * i + 2] = fmaf(g4.z, s[4 * i + 2], k4.z * v);     d2 = fmaf(s[4 * i + 2], q4.z, d2);
@@ -230,6 +305,15 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(ScanParams p) {
       if (active && (q & (SPLIT / GROUP - 1)) == 0) put(tt + mine, o[0]);
     };
     int tt = 0;
+    if (MODE == ENDS) {
+      if (nt == TOK) {
+#pragma unroll
+        for (int u = 0; u < TOK; ++u) token(u);
+      } else {
+        for (int u = 0; u < nt; ++u) token(u);
+      }
+      continue;
+    }
     if (nt == TOK) {
 #pragma unroll
       for (; tt + GROUP <= TOK; tt += GROUP) group(tt);
@@ -243,17 +327,20 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(ScanParams p) {
       if (active && q == 0) put(tt, o);
     }
   }
-  if (!active) return;
+  if (MODE != ENDS && !last) return;
 #pragma unroll
-  for (int i = 0; i < Q4; ++i) {
-    const int n = 4 * (q + SPLIT * i);
-    if (n >= p.dim) continue;
-    if (vec_state) {
-      *reinterpret_cast<float4*>(S + n) = make_float4(s[4 * i], s[4 * i + 1], s[4 * i + 2], s[4 * i + 3]);
-    } else {
+  for (int i = 0; i < Q4; ++i) store4(MODE == ENDS ? starts + (seg + 1) * seg_stride : S, i);
+  if constexpr (MODE == ENDS) {
+    if (c != 0) return;                                  // (one column's lanes leave the decays)
+    float* d = decays + seg * decay_stride;
+    if constexpr (CHANNEL) {
 #pragma unroll
-      for (int e = 0; e < 4; ++e)
-        if (n + e < p.dim) S[n + e] = s[4 * i + e];
+      for (int i = 0; i < PER; ++i) {
+        const int n = 4 * (q + SPLIT * (i >> 2)) + (i & 3);
+        if (n < p.dim) d[n] = prod[i];
+      }
+    } else if (q == 0) {
+      d[0] = prod[0];
     }
   }
 }
@@ -345,11 +432,20 @@ __global__ void exp_gates_kernel(const float* zi, long long ldi, const float* zf
 
 }  // namespace
 
+// A portion is cut into at most LS_SEGMENTS segments of at least LS_MIN_SEGMENT tokens, in steps of LS_MIN_TOKENS or more.
+constexpr int LS_SEGMENTS = 8, LS_MIN_SEGMENT = 256, LS_MIN_TOKENS = 512;
+
+// Floats of workspace that let up to four requests of a step have their portions cut.
+GB_API long long gb_linear_scan_workspace(int heads, int dim, int vdim, int normalised) {
+  return 4ll * LS_SEGMENTS * heads * ((long long)(vdim + (normalised ? 1 : 0)) * dim + dim) + 4;
+}
+
 // a0 q (f32; head h of row t at t * a1 + h * dim), a1 row stride, a2 k (likewise), a3 row stride, a4 v (f32; head h at
 // h * vdim), a5 row stride, a6 decays (f32: [t, heads * dim], or [t, heads] with flag bit 0), a7 row stride, a8 write
 // weights (f32 [t, heads]) or 0, a9 row stride, a10 state of slot 0 ([heads][vdim (+ 1)][dim], f32), a11 elements
 // between slots, a12 slot ids, a13 first row per request, a14 rows per request, a15 out (f32 [t, heads * vdim]), a16 its
-// row stride, a17 n . q out (f32 [t, heads]) or 0: no normaliser, a18 requests, a19 heads, a20 dim, a21 vdim;
+// row stride, a17 n . q out (f32 [t, heads]) or 0: no normaliser, a18 requests, a19 heads, a20 dim, a21 vdim, a22
+// tokens, a23 workspace of gb_linear_scan_workspace floats (16-byte aligned) or 0: portions are never cut into segments;
 // f0 factor on the read-out; flags bit 0: one decay a head
 GB_OP(gb_op_linear_scan) {
   ScanParams p;
@@ -368,17 +464,41 @@ GB_OP(gb_op_linear_scan) {
   p.vec_rows = p.dim % 4 == 0 && p.ldq % 4 == 0 && p.ldk % 4 == 0 && (a[0] & 15) == 0 && (a[2] & 15) == 0 &&
                (!channel || (p.ldg % 4 == 0 && (a[6] & 15) == 0));
   p.vec_v = p.vdim % 4 == 0 && p.ldv % 4 == 0 && (a[4] & 15) == 0;
-#define SCAN_LAUNCH(SPLIT, PER, TOK, CHANNEL)                                                                          \
+  // segments: when a step of many tokens has too few columns to fill the GPU
+  const int n = (int)a[22];
+  const int lanes = p.dim <= 16 ? 4 : p.dim <= 32 ? 8 : p.dim <= 64 ? 16 : p.dim <= 128 ? 8 : 16;
+  const long long blocks = (long long)R * p.H * gb_div_up(p.cols, LS_THREADS / lanes);
+  p.segs = 1; p.seg_len = 0;
+  if (a[23] && n >= LS_MIN_TOKENS && blocks < 148 * 6) {
+    const int len = (gb_div_up(n, LS_SEGMENTS) + 15) / 16 * 16;
+    p.seg_len = len > LS_MIN_SEGMENT ? len : LS_MIN_SEGMENT;
+    p.segs = gb_div_up(n, p.seg_len);
+    const long long decays = (long long)R * p.segs * p.H * (channel ? p.dim : 1);
+    const long long floats = ((decays + 3) & ~3ll) + (long long)R * p.segs * p.H * p.cols * p.dim;
+    if (floats > gb_linear_scan_workspace(p.H, p.dim, p.vdim, p.nq != nullptr)) p.segs = 1;
+    p.seg_decay = op_ptr<float>(a[23]);
+    p.seg_state = p.seg_decay + ((decays + 3) & ~3ll);
+  }
+#define SCAN_MODE(SPLIT, PER, TOK, CHANNEL, MODE)                                                                      \
   do {                                                                                                                  \
     constexpr int smem = ScanCfg<SPLIT, PER, TOK, CHANNEL>::SMEM;                                                       \
     static bool raised = false;            /* once, before any stream capture replays the launch */                    \
     if (!raised && smem > 48 * 1024) {                                                                                  \
-      GB_CUDA((cudaFuncSetAttribute(linear_scan_kernel<SPLIT, PER, TOK, CHANNEL>,                                       \
+      GB_CUDA((cudaFuncSetAttribute(linear_scan_kernel<SPLIT, PER, TOK, CHANNEL, MODE>,                                 \
                                     cudaFuncAttributeMaxDynamicSharedMemorySize, smem)));                               \
       raised = true;                                                                                                    \
     }                                                                                                                   \
-    gb_launch(linear_scan_kernel<SPLIT, PER, TOK, CHANNEL>, dim3(R, p.H, gb_div_up(p.cols, LS_THREADS / SPLIT)),         \
-              dim3(LS_THREADS), smem, ctx->stream, p);                                                                  \
+    gb_launch(linear_scan_kernel<SPLIT, PER, TOK, CHANNEL, MODE>,                                                       \
+              dim3(R * p.segs, p.H, gb_div_up(p.cols, LS_THREADS / SPLIT)), dim3(LS_THREADS), smem, ctx->stream, p);    \
+  } while (0)
+#define SCAN_LAUNCH(SPLIT, PER, TOK, CHANNEL)                                                                          \
+  do {                                                                                                                  \
+    if (p.segs == 1) {                                                                                                  \
+      SCAN_MODE(SPLIT, PER, TOK, CHANNEL, WHOLE);                                                                       \
+    } else {                                                                                                            \
+      SCAN_MODE(SPLIT, PER, TOK, CHANNEL, ENDS);                                                                        \
+      SCAN_MODE(SPLIT, PER, TOK, CHANNEL, SEGMENTS);                                                                    \
+    }                                                                                                                   \
   } while (0)
 #define SCAN(SPLIT, PER, TOK)                                                                                           \
   do { if (channel) SCAN_LAUNCH(SPLIT, PER, TOK, true); else SCAN_LAUNCH(SPLIT, PER, TOK, false); } while (0)
@@ -389,8 +509,9 @@ GB_OP(gb_op_linear_scan) {
   else SCAN(16, 16, 8);
 #undef SCAN
 #undef SCAN_LAUNCH
+#undef SCAN_MODE
   GB_CHECK_LAUNCH("linear_scan");
-  return 1;
+  return p.segs == 1 ? 1 : 2;
 }
 
 // a0 q (f32, changed in place), a1 its row stride, a2 gate logits (f32, replaced by the decays), a3 their row stride, a4

@@ -67,8 +67,8 @@ struct StreamParams {
 
 constexpr int STREAM_CACHE = 4;            // pieces of u a thread keeps between the sum of squares and the norm
 
-// S streams (0: any number up to MAX_STREAMS, taken from `streams`).
-template <int S, int VEC, bool MIX>
+// S streams (0: any number up to MAX_STREAMS, taken from `streams`); PART: y comes as partial tiles.
+template <int S, int VEC, bool MIX, bool PART>
 __global__ void stream_kernel(StreamParams p, int streams) {
   constexpr int CAP = S > 0 ? S : MAX_STREAMS;
   __shared__ float scratch[32];
@@ -122,7 +122,7 @@ __global__ void stream_kernel(StreamParams p, int streams) {
       if (S > 0 || s < n_s) old[s].load(x + (size_t)s * p.dim + (size_t)i * VEC);
     if constexpr (MIX) {
       Piece<VEC> yy, now[CAP];
-      if (p.part == nullptr) {
+      if constexpr (!PART) {
         yy.load(y + (size_t)i * VEC);
       } else {
         const float* at = p.part + (size_t)r * p.dim + (size_t)i * VEC;
@@ -219,8 +219,13 @@ int launch_streams(const StreamParams& p, int n, int streams, cudaStream_t strea
   const dim3 block(pieces <= 64 ? 64 : pieces <= 256 ? 128 : 256);
 #define STREAMS(S)                                                                                       \
   do {                                                                                                   \
-    if (vec) gb_launch(stream_kernel<S, 4, MIX>, dim3(n), block, 0, stream, p, streams);                 \
-    else gb_launch(stream_kernel<S, 1, MIX>, dim3(n), block, 0, stream, p, streams);                     \
+    if (MIX && p.part) {                                                                                 \
+      if (vec) gb_launch(stream_kernel<S, 4, MIX, MIX>, dim3(n), block, 0, stream, p, streams);          \
+      else gb_launch(stream_kernel<S, 1, MIX, MIX>, dim3(n), block, 0, stream, p, streams);              \
+    } else {                                                                                             \
+      if (vec) gb_launch(stream_kernel<S, 4, MIX, false>, dim3(n), block, 0, stream, p, streams);        \
+      else gb_launch(stream_kernel<S, 1, MIX, false>, dim3(n), block, 0, stream, p, streams);            \
+    }                                                                                                    \
   } while (0)
   switch (streams) {
     case 1: STREAMS(1); break;

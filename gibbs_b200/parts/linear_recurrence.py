@@ -30,6 +30,7 @@ from .. import ops
 from ..ops import hybrid
 from .base import Mixer, SlotState, TensorDecl, VECTOR, register_part
 from .runner import BranchPart, Runner, keep
+from .selective_scan import segment_workspace
 
 
 def padded(rn: Runner, name: str, width: int) -> torch.Tensor:
@@ -89,7 +90,8 @@ class GatedWriteRecurrence(RecurrentHeads):
         y = rn.buffer("rec_read", H * vdim, torch.float32)
         rn.op("linear_scan", [q, u.stride(0), k.data_ptr(), k.stride(0), v, u.stride(0), f, u.stride(0), 0, 0,
                               keep(rn, rec.state), rec.state.stride(0), rn.slots(rec), rn.q_start, rn.q_len, y.data_ptr(),
-                              y.stride(0), 0, rn.R, H, dim, vdim], [1.0], label="linear_scan:channel")
+                              y.stride(0), 0, rn.R, H, dim, vdim, rn.N,
+                              segment_workspace(rn, "linear_scan", H, dim, vdim, 0).data_ptr()], [1.0], label="linear_scan:channel")
         rn.op("head_norm", [y.data_ptr(), y.stride(0), vdim, 0, keep(rn, self.gain), 0, 0, out.data_ptr(),
                             ops.dtype_code(out.dtype), out.stride(0), rn.N, H, vdim], [self.eps, 0.0, factor],
               label="rec_norm")
@@ -137,7 +139,8 @@ class MatrixMemory(RecurrentHeads):
         nq = rn.buffer("mm_norm", H, torch.float32)
         rn.op("linear_scan", [at(0), u.stride(0), at(kc), u.stride(0), at(vc), u.stride(0), decay.data_ptr(), H,
                               write.data_ptr(), H, keep(rn, rec.state), rec.state.stride(0), slots, rn.q_start, rn.q_len,
-                              y.data_ptr(), y.stride(0), nq.data_ptr(), rn.R, H, dim, vdim], [self.q_scale],
+                              y.data_ptr(), y.stride(0), nq.data_ptr(), rn.R, H, dim, vdim, rn.N,
+                              segment_workspace(rn, "linear_scan", H, dim, vdim, 1).data_ptr()], [self.q_scale],
               label="linear_scan:head", flags=1)
         rn.op("head_norm", [y.data_ptr(), y.stride(0), vdim, 0, keep(rn, self.gain), at(gc), u.stride(0), out.data_ptr(),
                             ops.dtype_code(out.dtype), out.stride(0), rn.N, H, vdim, nq.data_ptr(), floor.data_ptr()],

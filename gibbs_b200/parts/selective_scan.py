@@ -17,10 +17,13 @@ read rows of the compute dtype and write 32-bit rows.
 """
 from __future__ import annotations
 
+import ctypes
+
 import torch
 
 from .. import ops
 from ..ops import hybrid
+from ..ops.library import library
 from .base import Mixer, SlotState, TensorDecl, VECTOR, register_part
 from .mlp import ACTIVATIONS
 from .runner import BranchPart, Runner, keep
@@ -28,6 +31,13 @@ from .runner import BranchPart, Runner, keep
 
 def round_up(n: int, m: int) -> int:
     return -(-n // m) * m
+
+
+def segment_workspace(rn: Runner, op: str, *sizes: int) -> torch.Tensor:
+    """What a recurrence needs to cut a long portion into segments that are computed side by side."""
+    fn = getattr(library(hybrid.LIBRARY), f"gb_{op}_workspace")
+    fn.restype = ctypes.c_longlong
+    return rn.buffer("segments_" + op, 4, torch.float32, fixed_rows=-(-int(fn(*map(ctypes.c_int, sizes))) // 4))
 
 
 class SelectiveScanMixer(BranchPart, Mixer):
@@ -83,11 +93,11 @@ class SelectiveScanMixer(BranchPart, Mixer):
         dt = rn.buffer("sel_dt", inner, torch.float32)
         rn.linear(low, self.w_dt, None, dt, role="scan_dt")
         y = rn.buffer("sel_out", inner)
-        rn.op("selective_scan", [x.data_ptr(), x.stride(0), dt.data_ptr(), dt.stride(0), p.data_ptr() + 4 * R,
-                                 p.data_ptr() + 4 * (R + N), p.stride(0), u.data_ptr() + 4 * inner, u.stride(0),
+        ws = segment_workspace(rn, "selective_scan", inner, N)
+        rn.op("selective_scan", [x.data_ptr(), x.stride(0), dt.data_ptr(), dt.stride(0), p.data_ptr() + 4 * R, rn.N, p.stride(0), u.data_ptr() + 4 * inner, u.stride(0),
                                  keep(rn, self.dt_bias), keep(rn, self.a_log), keep(rn, self.d_skip), keep(rn, rec.state),
                                  rec.state.stride(0), slots, rn.q_start, rn.q_len, y.data_ptr(), ops.dtype_code(y.dtype),
-                                 y.stride(0), rn.R, inner, N])
+                                 y.stride(0), rn.R, inner, N, ws.data_ptr()])
         rn.branch_linear(y, self.w_out, None, out, role="scan_out")
 
 

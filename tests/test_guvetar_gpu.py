@@ -301,6 +301,38 @@ def test_linear_recurrence_in_every_size_class(dim, vdim, kind):
         assert not norm or torch.equal(again[1], whole[1])
 
 
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("kind,m", [("mamba1", scan(72, 16, 8, 4)), ("mamba1", scan(33, 5, 3, 2)), ("mamba1", scan(40, 70, 16, 4)),
+                                    ("mlstm", memory(2, 64, 20, 15.0)), ("mlstm", memory(1, 100, 7, 15.0)), ("mlstm", memory(3, 9, 5, 5.0)),
+                                    ("parallel", sides((2, 1, 16, 8, 0.2, (0.5, 100)), (2, 48, 24))),
+                                    ("parallel", sides((1, 1, 8, 8, 0.2, None), (1, 130, 12)))])
+def test_long_portions_are_computed_in_segments_side_by_side(kind, m, dtype):
+    """A portion of more than 512 tokens is cut into segments that start from one another's ends: whole, as a long portion
+    behind a short one and in front of single tokens, two long portions in one step, one beside a single token; and a step
+    of many tokens none of whose portions is long enough to be cut."""
+    d, T = 32, 1100
+    cfg = one_layer(kind, m, d)
+    W = make_weights(cfg, 12)
+    h = bf(torch.randn(T, d, generator=gen(12)))
+    want, noise = with_noise(lambda: plain_mixer(cfg, 0, W, h))
+    part = part_of(cfg, 0, W, dtype)
+    hz = PartHarness(part, n_pages=240, page_size=16, n_slots=4, max_context=2048)
+    tol = 1e-3 if dtype == "float32" else None
+    for rid, cuts in (("whole", [T]), ("behind", [3, 1040, 1]), ("twice", [530, 570])):
+        check_rows(hz.run_cut(rid, h, cuts), want, dtype, what=rid, noise=noise, tol=tol)
+        hz.close(rid)
+    one = hz.feed_many({"a": h[:600], "b": h[:1], "c": h[:700]})
+    two = hz.feed_many({"a": h[600:601], "b": h[1:T], "c": h[700:T]})
+    for rid in ("a", "b", "c"):
+        got = torch.cat([one[rid], two[rid]], 0)
+        n = got.shape[0]
+        check_rows(got, want[:n], dtype, what=f"together {rid}", noise=[x[:n] for x in noise], tol=tol)
+        hz.close(rid)
+    parts = hz.feed_many({r: h[:200] for r in "abcd"})
+    for rid in "abcd":
+        check_rows(parts[rid], want[:200], dtype, what=f"short {rid}", noise=[x[:200] for x in noise], tol=tol)
+
+
 def _recurrence(T, seed=3):
     """A gated write recurrence beside an attention that is switched off, whose first token is written strongly into
     channels that then hardly forget."""
