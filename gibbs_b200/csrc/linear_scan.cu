@@ -61,7 +61,7 @@ template <int LEFT> __device__ __forceinline__ void ls_wait() {
 // S = S_1;  S <- decay_j S + S_j for the segments j in between, and computes read-outs.  (The first segment's start
 // is copied aside by ENDS, because the last segment writes the slot.)
 enum ScanMode : int { WHOLE = 0, ENDS = 1, SEGMENTS = 2 };
-constexpr int LS_STAGES = 4;
+constexpr int LS_STAGES = 3;
 
 template <int SPLIT, int PER, int TOK, bool CHANNEL>
 struct ScanCfg {
