@@ -45,14 +45,14 @@ template <int LEFT> __device__ __forceinline__ void ls_wait() {
   asm volatile("cp.async.wait_group %0;" ::"n"(LEFT) : "memory");
 }
 
-// A column of S lies in the registers of SPLIT neighbouring lanes, PER of its dim values each (dim <= SPLIT * PER;
-// lane q holds rows 4 (q + SPLIT i) + e).  The inputs of TOK tokens at a time arrive by asynchronous copies in a ring of
-// STAGES buffers, of which all but one are on their way while one is consumed; what a thread copies is the same for every
-// token, so its source and place are worked out once.  GROUP tokens are computed one after the other, each
-// leaving this lane's share of its read-out in a register, and the shares of all of them are then added over the lanes
-// together, every exchange halving what a lane still carries: one shuffle a token instead of log2(SPLIT).  A portion's
-// last tokens, fewer than GROUP, are added one by one in the same order of additions, so how a prompt is cut does not
-// change a bit.
+// Columns of S lie in the registers of SPLIT neighbouring lanes: a lane holds PER of the dim values of CPL neighbouring
+// columns (dim <= SPLIT * PER; lane q holds rows 4 (q + SPLIT i) + e), so that what it reads of q, k and g from shared
+// memory, whose bandwidth is what this kernel lives on, serves CPL columns.  The inputs of TOK tokens at a time arrive by
+// asynchronous copies in a ring of LS_STAGES buffers, of which all but one are on their way while one is consumed; what a
+// thread copies is the same for every token, so its source and place are worked out once.  GROUP tokens are computed one
+// after the other, each leaving this lane's shares of CPL read-outs in registers, and the shares of all of them are then
+// added over the lanes together, every exchange halving what a lane still carries.  A portion's last tokens, fewer than
+// GROUP, are added one by one in the same order of additions, so how a prompt is cut does not change a bit.
 //
 // WHOLE: a block walks its request's whole portion.  A long prompt of one request has too few columns to fill the GPU, and
 // a warp that is alone on its scheduler waits for its own latencies: the portion is then cut into segments.  ENDS
@@ -61,27 +61,51 @@ template <int LEFT> __device__ __forceinline__ void ls_wait() {
 // S = S_1;  S <- decay_j S + S_j for the segments j in between, and computes read-outs.  (The first segment's start
 // is copied aside by ENDS, because the last segment writes the slot.)
 enum ScanMode : int { WHOLE = 0, ENDS = 1, SEGMENTS = 2 };
-constexpr int LS_STAGES = 3;
+constexpr int LS_STAGES = 3, CPL = 4, GROUP = 4;
 
 template <int SPLIT, int PER, int TOK, bool CHANNEL>
 struct ScanCfg {
-  static constexpr int NR = SPLIT * PER, COLS = LS_THREADS / SPLIT, ROWS = CHANNEL ? 3 : 2;
+  static constexpr int NR = SPLIT * PER, COLS = LS_THREADS / SPLIT * CPL, ROWS = CHANNEL ? 3 : 2;
   static constexpr int BUF = TOK * (ROWS * NR + COLS + 4);   // q [TOK][NR] | k | (g) | v [TOK][COLS] | (g, w, -, -) [TOK]
   static constexpr int SMEM = LS_STAGES * BUF * 4;
 };
+
+// V values a lane carries, added over SPLIT lanes: lanes whose bit is set keep the upper half, the others the lower half, as
+// long as there are halves.  Returns the index of the first value this lane ends up with (values 0 .. max(V / SPLIT, 1)
+// of o); when there are more lanes than values, several lanes end up with the same one.
+template <int SPLIT, int V>
+__device__ __forceinline__ int ls_reduce(float (&o)[V], int q) {
+  int mine = 0;
+#pragma unroll
+  for (int w = SPLIT / 2, carried = V; w > 0; w >>= 1) {
+    if (carried > 1) {
+      const int half = carried / 2;
+      const bool upper = q & w;
+#pragma unroll
+      for (int u = 0; u < V / 2; ++u) {
+        if (u < half) {
+          const float give = upper ? o[u] : o[u + half], keep = upper ? o[u + half] : o[u];
+          o[u] = keep + __shfl_xor_sync(0xffffffffu, give, w);
+        }
+      }
+      mine += upper ? half : 0;
+      carried = half;
+    } else {
+      o[0] += __shfl_xor_sync(0xffffffffu, o[0], w);
+    }
+  }
+  return mine;
+}
 
 template <int SPLIT, int PER, int TOK, bool CHANNEL, int MODE>
 __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(ScanParams p) {
   using C = ScanCfg<SPLIT, PER, TOK, CHANNEL>;
   constexpr int NR = C::NR, COLS = C::COLS, Q4 = PER / 4, ROWS = C::ROWS, BUF = C::BUF;
-  constexpr int GROUP = SPLIT < 8 ? SPLIT : 8;
   extern __shared__ __align__(16) float ls_sm[];         // [LS_STAGES][BUF]
   pdl_trigger();
-  const int col = threadIdx.x / SPLIT, q = threadIdx.x % SPLIT;
+  const int cg = threadIdx.x / SPLIT, q = threadIdx.x % SPLIT;
   const int r = MODE == WHOLE ? blockIdx.x : blockIdx.x / p.segs, seg = MODE == WHOLE ? 0 : blockIdx.x - r * p.segs;
-  const int h = blockIdx.y, c0 = blockIdx.z * COLS, c = c0 + col;
-  const bool active = c < p.cols;
-  const bool counts = c == p.vdim;                       // the normaliser's column: its value is always 1
+  const int h = blockIdx.y, c0 = blockIdx.z * COLS, c = c0 + cg * CPL;      // this lane's columns: c .. c + CPL - 1
   const int all = p.q_len[r];                            // the portion
   const int first = p.q_start[r] + seg * p.seg_len;
   const int len = MODE == WHOLE ? all : min(p.seg_len, all - seg * p.seg_len);
@@ -90,12 +114,11 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(ScanParams p) {
     pdl_wait();                                          // a launch all of whose blocks leave still ends behind the one in front
     return;
   }
-  float* S = p.state + (size_t)p.slot_ids[r] * p.slot_stride + ((size_t)h * p.cols + (active ? c : 0)) * p.dim;
-  // where segment i of this request starts from, for this column: the slot's state (0), the state segment 0 leaves (1), or
-  // what segment i - 1 leaves when it starts from zero
+  float* S = p.state + (size_t)p.slot_ids[r] * p.slot_stride + ((size_t)h * p.cols + c) * p.dim;
+  // where segment i of this request starts from, for these columns: the slot's state (0), the state segment 0 leaves (1),
+  // or what segment i - 1 leaves when it starts from zero
   const size_t seg_stride = (size_t)p.H * p.cols * p.dim;
-  float* starts = MODE == WHOLE ? nullptr
-                                : p.seg_state + (size_t)r * p.segs * seg_stride + ((size_t)h * p.cols + (active ? c : 0)) * p.dim;
+  float* starts = MODE == WHOLE ? nullptr : p.seg_state + (size_t)r * p.segs * seg_stride + ((size_t)h * p.cols + c) * p.dim;
   const size_t decay_stride = CHANNEL ? (size_t)p.H * p.dim : (size_t)p.H;
   float* decays = MODE == WHOLE ? nullptr : p.seg_decay + (size_t)r * p.segs * decay_stride + (CHANNEL ? h * p.dim : h);
   const int vcols = max(0, min(COLS, p.vdim - c0));
@@ -133,10 +156,10 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(ScanParams p) {
   }
   pdl_wait();
   const bool vec_state = (p.dim & 3) == 0 && (p.slot_stride & 3) == 0 && ((uintptr_t)p.state & 15) == 0;
-  float s[PER] = {};
+  float s[CPL][PER] = {};
   auto fetch4 = [&](const float* src, int n) {            // entries n .. n + 3 of a column, 0 beyond dim
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (active && n < p.dim) {
+    if (n < p.dim) {
       if (vec_state) {
         v = *reinterpret_cast<const float4*>(src + n);
       } else {
@@ -148,39 +171,55 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(ScanParams p) {
     }
     return v;
   };
-  auto store4 = [&](float* dst, int i) {
-    const int n = 4 * (q + SPLIT * i);
-    if (!active || n >= p.dim) return;
-    if (vec_state) {
-      *reinterpret_cast<float4*>(dst + n) = make_float4(s[4 * i], s[4 * i + 1], s[4 * i + 2], s[4 * i + 3]);
-    } else {
+  auto store_state = [&](float* dst) {
 #pragma unroll
-      for (int e = 0; e < 4; ++e)
-        if (n + e < p.dim) dst[n + e] = s[4 * i + e];
-    }
-  };
+    for (int e = 0; e < CPL; ++e) {
+      if (c + e >= p.cols) continue;
 #pragma unroll
-  for (int i = 0; i < Q4; ++i) {
-    const int n = 4 * (q + SPLIT * i);
-    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (MODE == WHOLE || (MODE == SEGMENTS && seg == 0 && last) || (MODE == ENDS && seg == 0)) {
-      v = fetch4(S, n);
-    } else if (MODE == SEGMENTS) {
-      v = fetch4(starts + (seg == 0 ? 0 : seg_stride), n);
-      for (int j = 2; j <= seg; ++j) {
-        const float4 e = fetch4(starts + j * seg_stride, n);
-        float4 d;
-        if (CHANNEL) {
-          d = fetch4(decays + (j - 1) * decay_stride, n);
+      for (int i = 0; i < Q4; ++i) {
+        const int n = 4 * (q + SPLIT * i);
+        float* d = dst + (size_t)e * p.dim + n;
+        if (n >= p.dim) continue;
+        if (vec_state) {
+          *reinterpret_cast<float4*>(d) = make_float4(s[e][4 * i], s[e][4 * i + 1], s[e][4 * i + 2], s[e][4 * i + 3]);
         } else {
-          const float dh = decays[(j - 1) * decay_stride];
-          d = make_float4(dh, dh, dh, dh);
+#pragma unroll
+          for (int x = 0; x < 4; ++x)
+            if (n + x < p.dim) d[x] = s[e][4 * i + x];
         }
-        v = make_float4(fmaf(d.x, v.x, e.x), fmaf(d.y, v.y, e.y), fmaf(d.z, v.z, e.z), fmaf(d.w, v.w, e.w));
       }
     }
-    s[4 * i] = v.x; s[4 * i + 1] = v.y; s[4 * i + 2] = v.z; s[4 * i + 3] = v.w;
-    if (MODE == ENDS && seg == 0) store4(starts, i);
+  };
+  const bool from_slot = MODE == WHOLE || (MODE == SEGMENTS && seg == 0 && last) || (MODE == ENDS && seg == 0);
+  if (MODE != ENDS || seg == 0) {
+#pragma unroll
+    for (int e = 0; e < CPL; ++e) {
+      if (c + e >= p.cols) continue;
+#pragma unroll
+      for (int i = 0; i < Q4; ++i) {
+        const int n = 4 * (q + SPLIT * i);
+        const size_t at = (size_t)e * p.dim;
+        float4 v;
+        if (from_slot) {
+          v = fetch4(S + at, n);
+        } else {
+          v = fetch4(starts + (seg == 0 ? 0 : seg_stride) + at, n);
+          for (int j = 2; j <= seg; ++j) {
+            const float4 x = fetch4(starts + j * seg_stride + at, n);
+            float4 d;
+            if (CHANNEL) {
+              d = fetch4(decays + (j - 1) * decay_stride, n);
+            } else {
+              const float dh = decays[(j - 1) * decay_stride];
+              d = make_float4(dh, dh, dh, dh);
+            }
+            v = make_float4(fmaf(d.x, v.x, x.x), fmaf(d.y, v.y, x.y), fmaf(d.z, v.z, x.z), fmaf(d.w, v.w, x.w));
+          }
+        }
+        s[e][4 * i] = v.x; s[e][4 * i + 1] = v.y; s[e][4 * i + 2] = v.z; s[e][4 * i + 3] = v.w;
+      }
+    }
+    if (MODE == ENDS) store_state(starts);
   }
   float prod[MODE == ENDS ? (CHANNEL ? PER : 1) : 1];      // the product of the segment's decays
 #pragma unroll
@@ -239,99 +278,82 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(ScanParams p) {
     const float* Q = ls_sm + (chunk % LS_STAGES) * BUF + 4 * q;
     const float* K = Q + TOK * NR;
     const float* G = K + TOK * NR;
-    const float* V = ls_sm + (chunk % LS_STAGES) * BUF + ROWS * TOK * NR + col;
+    const float* V = ls_sm + (chunk % LS_STAGES) * BUF + ROWS * TOK * NR + cg * CPL;
     const float* GW = ls_sm + (chunk % LS_STAGES) * BUF + TOK * (ROWS * NR + COLS);
-    // one token: the state's step, and this lane's share of the read-out
-    auto token = [&](int tt) {
-      float v = counts ? 1.f : V[tt * COLS];
+    // one token: the state's step, and this lane's shares of the read-outs
+    auto token = [&](int tt, float* o) {
+      const float4 v4 = *reinterpret_cast<const float4*>(V + tt * COLS);
       const float2 gw = *reinterpret_cast<const float2*>(GW + 4 * tt);
-      if (weighted) v *= gw.y;
-      float d0 = 0.f, d1 = 0.f, d2 = 0.f, d3 = 0.f;      // four chains, added in a fixed order
+      float v[CPL] = {v4.x, v4.y, v4.z, v4.w};
+#pragma unroll
+      for (int e = 0; e < CPL; ++e) {
+        if (c + e == p.vdim) v[e] = 1.f;                   // the normaliser's column
+        if (weighted) v[e] *= gw.y;
+        if (MODE != ENDS) o[e] = 0.f;
+      }
       if (MODE == ENDS && !CHANNEL) prod[0] *= gw.x;
 #pragma unroll
       for (int i = 0; i < Q4; ++i) {
         const float4 k4 = *reinterpret_cast<const float4*>(K + tt * NR + 4 * SPLIT * i);
-        float4 q4 = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (MODE != ENDS) q4 = *reinterpret_cast<const float4*>(Q + tt * NR + 4 * SPLIT * i);
-        float4 g4 = make_float4(gw.x, gw.x, gw.x, gw.x);
+        float4 g4 = make_float4(gw.x, gw.x, gw.x, gw.x), q4 = g4;
         if (CHANNEL) g4 = *reinterpret_cast<const float4*>(G + tt * NR + 4 * SPLIT * i);
-        if constexpr (MODE == ENDS) {
-          s[4 * i] = fmaf(g4.x, s[4 * i], k4.x * v);
-          s[4 * i + 1] = fmaf(g4.y, s[4 * i + 1], k4.y * v);
-          s[4 * i + 2] = fmaf(g4.z, s[4 * i + 2], k4.z * v);
-          s[4 * i + 3] = fmaf(g4.w, s[4 * i + 3], k4.w * v);
-          if constexpr (CHANNEL) {
-            prod[4 * i] *= g4.x; prod[4 * i + 1] *= g4.y; prod[4 * i + 2] *= g4.z; prod[4 * i + 3] *= g4.w;
-          }
-          continue;
+        if (MODE != ENDS) q4 = *reinterpret_cast<const float4*>(Q + tt * NR + 4 * SPLIT * i);
+        if constexpr (MODE == ENDS && CHANNEL) {
+          prod[4 * i] *= g4.x; prod[4 * i + 1] *= g4.y; prod[4 * i + 2] *= g4.z; prod[4 * i + 3] *= g4.w;
         }
-        s[4 * i] = fmaf(g4.x, s[4 * i], k4.x * v);             d0 = fmaf(s[4 * i], q4.x, d0);
-        s[4 * i + 1] = fmaf(g4.y, s[4 * i + 1], k4.y * v);     d1 = fmaf(s[4 * i + 1], q4.y, d1);
-        s[4 * i + 2] = fmaf(g4.z, s[4 * i + 2], k4.z * v);     d2 = fmaf(s[4 * i + 2], q4.z, d2);
-        s[4 * i + 3] = fmaf(g4.w, s[4 * i + 3], k4.w * v);     d3 = fmaf(s[4 * i + 3], q4.w, d3);
-      }
-      return (d0 + d1) + (d2 + d3);
-    };
-    auto put = [&](int tt, float o) {
-      const size_t row = (size_t)(first + t0 + tt);
-      if (counts) p.nq[row * p.H + h] = o * p.q_scale;
-      else p.out[row * p.ldo + (size_t)h * p.vdim + c] = o * p.q_scale;
-    };
-    // lanes whose bit `w` is set keep the upper half of the tokens they carry, the others the lower half
-    auto group = [&](int tt) {
-      float o[GROUP];
 #pragma unroll
-      for (int u = 0; u < GROUP; ++u) o[u] = token(tt + u);
-      int mine = 0;
-#pragma unroll
-      for (int w = SPLIT / 2, carried = GROUP; w > 0; w >>= 1) {
-        if (carried > 1) {
-          const int half = carried / 2;
-          const bool upper = q & w;
-#pragma unroll
-          for (int u = 0; u < GROUP / 2; ++u) {
-            if (u < half) {
-              const float give = upper ? o[u] : o[u + half], keep = upper ? o[u + half] : o[u];
-              o[u] = keep + __shfl_xor_sync(0xffffffffu, give, w);
-            }
-          }
-          mine += upper ? half : 0;
-          carried = half;
-        } else {
-          o[0] += __shfl_xor_sync(0xffffffffu, o[0], w);
+        for (int e = 0; e < CPL; ++e) {
+          float* se = s[e] + 4 * i;
+          se[0] = fmaf(g4.x, se[0], k4.x * v[e]);
+          se[1] = fmaf(g4.y, se[1], k4.y * v[e]);
+          se[2] = fmaf(g4.z, se[2], k4.z * v[e]);
+          se[3] = fmaf(g4.w, se[3], k4.w * v[e]);
+          if (MODE != ENDS)
+            o[e] = fmaf(se[3], q4.w, fmaf(se[2], q4.z, fmaf(se[1], q4.y, fmaf(se[0], q4.x, o[e]))));
         }
       }
-      // (several lanes carry the same token when there are more lanes than tokens: the first of them stores)
-      if (active && (q & (SPLIT / GROUP - 1)) == 0) put(tt + mine, o[0]);
     };
-    int tt = 0;
-    if (MODE == ENDS) {
+    // value number i of tokens tt ..: column i % CPL of token tt + i / CPL
+    auto put = [&](int tt, int i, float o) {
+      const size_t row = (size_t)(first + t0 + tt + i / CPL);
+      const int cc = c + i % CPL;
+      if (cc < p.vdim) p.out[row * p.ldo + (size_t)h * p.vdim + cc] = o * p.q_scale;
+      else if (cc < p.cols) p.nq[row * p.H + h] = o * p.q_scale;
+    };
+    if constexpr (MODE == ENDS) {
+      float none[CPL];
       if (nt == TOK) {
-#pragma unroll
-        for (int u = 0; u < TOK; ++u) token(u);
+#pragma unroll 4
+        for (int u = 0; u < TOK; ++u) token(u, none);
       } else {
-        for (int u = 0; u < nt; ++u) token(u);
+        for (int u = 0; u < nt; ++u) token(u, none);
       }
-      continue;
-    }
-    if (nt == TOK) {
-#pragma unroll
-      for (; tt + GROUP <= TOK; tt += GROUP) group(tt);
     } else {
-      for (; tt + GROUP <= nt; tt += GROUP) group(tt);
-    }
-    for (; tt < nt; ++tt) {
-      float o = token(tt);
+      int tt = 0;
+#pragma unroll 1
+      for (; tt + GROUP <= nt; tt += GROUP) {
+        float o[GROUP * CPL];
 #pragma unroll
-      for (int w = SPLIT / 2; w > 0; w >>= 1) o += __shfl_xor_sync(0xffffffffu, o, w);
-      if (active && q == 0) put(tt, o);
+        for (int u = 0; u < GROUP; ++u) token(tt + u, o + u * CPL);
+        const int mine = ls_reduce<SPLIT, GROUP * CPL>(o, q);
+        constexpr int LEFT = GROUP * CPL > SPLIT ? GROUP * CPL / SPLIT : 1;
+        if (SPLIT <= GROUP * CPL || (q & (SPLIT / (GROUP * CPL) - 1)) == 0) {
+#pragma unroll
+          for (int i = 0; i < LEFT; ++i) put(tt, mine + i, o[i]);
+        }
+      }
+      for (; tt < nt; ++tt) {
+        float o[CPL];
+        token(tt, o);
+        const int mine = ls_reduce<SPLIT, CPL>(o, q);
+        if ((q & (SPLIT / CPL - 1)) == 0) put(tt, mine, o[0]);
+      }
     }
   }
   if (MODE != ENDS && !last) return;
-#pragma unroll
-  for (int i = 0; i < Q4; ++i) store4(MODE == ENDS ? starts + (seg + 1) * seg_stride : S, i);
+  store_state(MODE == ENDS ? starts + (seg + 1) * seg_stride : S);
   if constexpr (MODE == ENDS) {
-    if (c != 0) return;                                  // (one column's lanes leave the decays)
+    if (c != 0) return;                                  // (one group of columns leaves the decays)
     float* d = decays + seg * decay_stride;
     if constexpr (CHANNEL) {
 #pragma unroll
@@ -433,11 +455,11 @@ __global__ void exp_gates_kernel(const float* zi, long long ldi, const float* zf
 }  // namespace
 
 // A portion is cut into at most LS_SEGMENTS segments of at least LS_MIN_SEGMENT tokens, in steps of LS_MIN_TOKENS or more.
-constexpr int LS_SEGMENTS = 8, LS_MIN_SEGMENT = 256, LS_MIN_TOKENS = 512;
+constexpr int LS_SEGMENTS = 16, LS_MIN_SEGMENT = 128, LS_MIN_TOKENS = 512;
 
-// Floats of workspace that let up to four requests of a step have their portions cut.
+// Floats of workspace that hold 32 segments (a step that would need more is not cut).
 GB_API long long gb_linear_scan_workspace(int heads, int dim, int vdim, int normalised) {
-  return 4ll * LS_SEGMENTS * heads * ((long long)(vdim + (normalised ? 1 : 0)) * dim + dim) + 4;
+  return 32ll * heads * ((long long)(vdim + (normalised ? 1 : 0)) * dim + dim) + 4;
 }
 
 // a0 q (f32; head h of row t at t * a1 + h * dim), a1 row stride, a2 k (likewise), a3 row stride, a4 v (f32; head h at
@@ -466,11 +488,12 @@ GB_OP(gb_op_linear_scan) {
   p.vec_v = p.vdim % 4 == 0 && p.ldv % 4 == 0 && (a[4] & 15) == 0;
   // segments: when a step of many tokens has too few columns to fill the GPU
   const int n = (int)a[22];
-  const int lanes = p.dim <= 16 ? 4 : p.dim <= 32 ? 8 : p.dim <= 64 ? 16 : p.dim <= 128 ? 8 : 16;
-  const long long blocks = (long long)R * p.H * gb_div_up(p.cols, LS_THREADS / lanes);
+  const int lanes = p.dim <= 16 ? 4 : p.dim <= 32 ? 8 : p.dim <= 128 ? 16 : 32;
+  const long long blocks = (long long)R * p.H * gb_div_up(p.cols, LS_THREADS / lanes * CPL);
   p.segs = 1; p.seg_len = 0;
-  if (a[23] && n >= LS_MIN_TOKENS && blocks < 148 * 6) {
-    const int len = (gb_div_up(n, LS_SEGMENTS) + 15) / 16 * 16;
+  if (a[23] && n >= LS_MIN_TOKENS && blocks < 148 * 4) {
+    const int wanted = gb_div_up(148 * 8, blocks);        // (about as many blocks as the GPU holds)
+    const int len = (gb_div_up(n, wanted < LS_SEGMENTS ? wanted : LS_SEGMENTS) + 15) / 16 * 16;
     p.seg_len = len > LS_MIN_SEGMENT ? len : LS_MIN_SEGMENT;
     p.segs = gb_div_up(n, p.seg_len);
     const long long decays = (long long)R * p.segs * p.H * (channel ? p.dim : 1);
@@ -489,7 +512,7 @@ GB_OP(gb_op_linear_scan) {
       raised = true;                                                                                                    \
     }                                                                                                                   \
     gb_launch(linear_scan_kernel<SPLIT, PER, TOK, CHANNEL, MODE>,                                                       \
-              dim3(R * p.segs, p.H, gb_div_up(p.cols, LS_THREADS / SPLIT)), dim3(LS_THREADS), smem, ctx->stream, p);    \
+              dim3(R * p.segs, p.H, gb_div_up(p.cols, LS_THREADS / SPLIT * CPL)), dim3(LS_THREADS), smem, ctx->stream, p);    \
   } while (0)
 #define SCAN_LAUNCH(SPLIT, PER, TOK, CHANNEL)                                                                          \
   do {                                                                                                                  \
@@ -505,8 +528,8 @@ GB_OP(gb_op_linear_scan) {
   if (p.dim <= 16) SCAN(4, 4, 16);
   else if (p.dim <= 32) SCAN(8, 4, 16);
   else if (p.dim <= 64) SCAN(16, 4, 16);
-  else if (p.dim <= 128) SCAN(8, 16, 8);
-  else SCAN(16, 16, 8);
+  else if (p.dim <= 128) SCAN(16, 8, 8);
+  else SCAN(32, 8, 8);
 #undef SCAN
 #undef SCAN_LAUNCH
 #undef SCAN_MODE
