@@ -182,8 +182,11 @@ class GatedAttention(Mixer):
             raise RuntimeError(f"pages of {tuple(kp.shape[1:])} / {tuple(vp.shape[1:])} for {G} kv heads of {dim} / {vdim}")
         table, bt_stride = rn.table(kv)
         pages_bf16 = kp.dtype == torch.bfloat16
-        # bfloat16 pages and sizes the tensor-core kernel is built for: queries in bfloat16 as well
-        tc = pages_bf16 and self.rt.dtype == torch.bfloat16 and USE_TENSOR_CORES and _tensor_cores_take(H, G, dim, vdim)
+        if out is None:
+            out = rn.buffer("ga_heads_out", H * vdim)
+        # bfloat16 pages, sizes the tensor-core kernel is built for and rows it can write in pairs: queries in bfloat16 too
+        tc = (pages_bf16 and self.rt.dtype == torch.bfloat16 and USE_TENSOR_CORES and _tensor_cores_take(H, G, dim, vdim)
+              and out.stride(0) % 2 == 0 and out.data_ptr() % 4 == 0)
         q = rn.buffer("ga_query", H * dim, torch.bfloat16 if tc else torch.float32)
         write = not self.shares_kv
         rn.op("qk_prep", [fused.data_ptr(), fused.stride(0), self.k_col, self.v_col, keep(rn, self.q_gain),
@@ -193,8 +196,6 @@ class GatedAttention(Mixer):
               [self.eps, self.temp_coef, self.temp_every],
               flags=(1 if self.whole_norm else 0) | (8 if self.head_norm else 0) | (2 if tc else 0) | (4 if pages_bf16 else 0) |
                     (16 if self.rot_halves else 0) | (32 if self.norm_after_rot else 0))
-        if out is None:
-            out = rn.buffer("ga_heads_out", H * vdim)
         if factor != 1.0 and not self.sigmoid:
             raise ValueError("a factor on the heads' outputs is taken by unnormalised weights only")
         # (unnormalised weights: an operation of their own, whose last constant is the factor on the output)

@@ -68,7 +68,8 @@ class ParallelMixers(BranchPart, Mixer):
     def run(self, rn: Runner, h, out, caches, accumulate: bool = False):
         u = padded(rn, "par_in", self.fused.shape[0])
         rn.linear(h, self.fused, None, u, role="par_in")
-        o = rn.buffer("par_heads", self.out_cols[-1])
+        # (rows on 16-byte boundaries: what the kernels that write into columns of them may ask for)
+        o = rn.buffer("par_heads", -(-self.out_cols[-1] // 8) * 8)[:, :self.out_cols[-1]]
         at = 0
         for i, (side, factor) in enumerate(zip(self.sides, self.factors)):
             n = len(side.cache_needs())

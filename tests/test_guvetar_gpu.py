@@ -555,12 +555,13 @@ def test_temperature_bias_norms_and_factors_show(dtype):
         assert steps == [p for p in range(1, 210) if (p + 1) % every == 0]
 
 
-@pytest.mark.parametrize("heads,kv_heads,dim,vdim", [(8, 2, 64, 64), (4, 1, 128, 32), (6, 2, 32, 96), (20, 1, 32, 64), (3, 3, 96, 128)])
-def test_tensor_core_sigmoid_attention_against_the_generic_kernel(heads, kv_heads, dim, vdim, monkeypatch):
+@pytest.mark.parametrize("heads,kv_heads,dim,vdim,right", [(8, 2, 64, 64, (2, 8, 16)), (4, 1, 128, 32, (3, 8, 5)), (6, 2, 32, 96, (1, 4, 1)),
+                                                         (20, 1, 32, 64, (2, 8, 3)), (3, 3, 96, 128, (2, 8, 16))])
+def test_tensor_core_sigmoid_attention_against_the_generic_kernel(heads, kv_heads, dim, vdim, right, monkeypatch):
     """bfloat16: the two kernels read the same pages; the tensor-core one reads the queries in bfloat16 too.  Whole, cut
-    at odd places, decoded, and a portion beside single tokens."""
+    at odd places, decoded, and a portion beside single tokens; beside mixers whose outputs make the joint rows odd."""
     from gibbs_b200.parts import gated_attention
-    cfg = one_layer("parallel", sides((heads, kv_heads, dim, vdim, dim ** -0.5, (0.5, 30)), (2, 8, 16), (0.8, 0.1)), 96)
+    cfg = one_layer("parallel", sides((heads, kv_heads, dim, vdim, dim ** -0.5, (0.5, 30)), right, (0.8, 0.1)), 96)
     W = make_weights(cfg, 5)
     T = 300
     h = bf(torch.randn(T, 96, generator=gen(6)))
