@@ -29,7 +29,8 @@ LIBRARIES = {
     "core": ["errors.cu", "elementwise.cu", "gemm_simt.cu", "conv.cu", "attention.cu", "sampling.cu"],
     "tensorcore": ["errors.cu", "gemm_tc.cu", "gemm_tc_decode.cu", "attention_tc.cu", "attention_tcgen05.cu"],
     "runtime": ["errors.cu", "step_plan.cu"],
-    # layer norms, clamped gated units, latent and gated attention, state-space and delta-rule recurrences, routed experts: every entry
+    # layer norms, clamped gated units, latent, gated and sigmoid attention, state-space, delta-rule and linear recurrences, residual
+    # streams, routed experts: every entry
     # point has the signature of a step-plan operation (hybrid.cuh)
     "hybrid": ["errors.cu", "norms.cu", "latent_attention.cu", "latent_attention_tc.cu", "gated_attention.cu", "gated_attention_tc.cu",
                "sigmoid_attention_tc.cu", "ssm.cu", "selective_scan.cu", "delta_rule.cu", "linear_scan.cu", "streams.cu", "moe.cu",

@@ -1,6 +1,7 @@
 """Bindings of the "hybrid" kernel library (csrc/norms.cu, latent_attention.cu,
-gated_attention.cu, gated_attention_tc.cu, ssm.cu, delta_rule.cu, moe.cu): layer norms, clamped gated units, latent
-attention, gated attention with a sink, state-space and delta-rule recurrences and routed experts.
+gated_attention.cu, gated_attention_tc.cu, sigmoid_attention_tc.cu, ssm.cu, selective_scan.cu, delta_rule.cu,
+linear_scan.cu, streams.cu, moe.cu): layer norms, clamped gated units, latent attention, gated attention with a sink,
+attention without a softmax, state-space, delta-rule and linear recurrences, residual streams and routed experts.
 
 Every operation of that library has the signature of a step-plan operation,
 ``int op(ctx, a[24], f[3], flags)``.  So an operation is described ONCE, by
