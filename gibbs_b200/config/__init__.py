@@ -6,6 +6,7 @@ from .petelix import PetelixConfig
 from .sisadra import SisadraConfig
 from .selivik import SelivikConfig
 from .guvetar import GuvetarConfig
+from .nutopel import NutopelConfig
 
 register_architecture("Lfm2ForCausalLM", Lfm2Config.from_dict, model_types=("lfm2",))
 register_architecture("Potivik", PotivikConfig.from_dict, model_types=("potivik",))
@@ -13,8 +14,9 @@ register_architecture("Petelix", PetelixConfig.from_dict, model_types=("petelix"
 register_architecture("Sisadra", SisadraConfig.from_dict, model_types=("sisadra",))
 register_architecture("Selivik", SelivikConfig.from_dict, model_types=("selivik",))
 register_architecture("Guvetar", GuvetarConfig.from_dict, model_types=("guvetar",))
+register_architecture("Nutopel", NutopelConfig.from_dict, model_types=("nutopel",))
 
 __all__ = ["ModelPlan", "LayerSpec", "OrderEntry", "PartSpec", "prenorm_layer", "register_architecture", "known_architectures",
            "detect", "parse_config", "Lfm2Config", "PotivikConfig", "PetelixConfig", "SisadraConfig", "SelivikConfig",
-           "GuvetarConfig",
+           "GuvetarConfig", "NutopelConfig",
            "ConfigError"]

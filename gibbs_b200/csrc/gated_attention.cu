@@ -84,10 +84,10 @@ enum { PREP_NORM_WHOLE = 1, PREP_Q_BF16 = 2, PREP_PAGES_BF16 = 4, PREP_NORM_HEAD
 // One normed and rotated element of a projection: entry d of a head of `dim` entries that starts at `base`.
 // `gain` is indexed like the projection (norm over the whole projection) or by d (`gain_per_head`: one gain
 // vector shared by all heads).  The first `rot_dims` entries turn by pos * inv_freq[i], in adjacent pairs
-// (2i, 2i+1) or, with `halves`, in pairs (i, i + rot_dims/2).
+// (2i, 2i+1) or, with `halves`, in pairs (i, i + rot_dims/2); cosines and sines are multiplied by mscale.
 __device__ __forceinline__ float prep_element(const float* x, const float* __restrict__ gain, bool gain_per_head,
                                               float rstd, int base, int d, int rot_dims, bool halves,
-                                              const float* __restrict__ inv_freq, int pos) {
+                                              const float* __restrict__ inv_freq, int pos, float mscale) {
   const int gb = gain_per_head ? 0 : base;
   const float own = x[base + d] * rstd * (gain ? gain[gb + d] : 1.f);
   if (d >= rot_dims) return own;
@@ -97,7 +97,7 @@ __device__ __forceinline__ float prep_element(const float* x, const float* __res
   const int fi = halves ? (second ? d - half : d) : (d >> 1);
   const float other = x[base + partner] * rstd * (gain ? gain[gb + partner] : 1.f);
   const float ang = (float)pos * inv_freq[fi];
-  const float c = cosf(ang), s = sinf(ang);
+  const float c = cosf(ang) * mscale, s = sinf(ang) * mscale;
   // the pair (u, v) becomes (u c - v s, v c + u s)
   return second ? own * c + other * s : own * c - other * s;
 }
@@ -123,6 +123,7 @@ __global__ void qk_prep_kernel(const float* fused, long long ld, int k_col, int 
   const bool after = mode & PREP_NORM_AFTER;
   // a query grows with its position: 1 + coef * ln(floor((pos + 1) / every) + 1)
   const float temp = temp_every > 0.f ? fmaf(temp_coef, logf(floorf((float)(pos + 1) / temp_every) + 1.f), 1.f) : 1.f;
+  const float mscale = rot_dims > 0 ? inv_freq[rot_dims >> 1] : 1.f;
   int page = -1;
   if (writes) page = block_table[(size_t)tok_req[t] * bt_stride + pos / page_size];
   pdl_wait();
@@ -151,14 +152,14 @@ __global__ void qk_prep_kernel(const float* fused, long long ld, int k_col, int 
     if (after) {
       float ss = 0.f;
       for (int d = lane; d < dim; d += 32) {
-        const float v = prep_element(row, nullptr, true, 1.f, h * dim, d, rot_dims, halves, inv_freq, pos);
+        const float v = prep_element(row, nullptr, true, 1.f, h * dim, d, rot_dims, halves, inv_freq, pos, mscale);
         ss += v * v;
       }
       post = temp / sqrtf(warp_sum(ss) / (float)dim + eps);
     }
     for (int d = lane; d < dim; d += 32)
       q_out[(size_t)t * ldq + h * dim + d] = from_f32<TQ>(post * prep_element(row, normed ? q_gain : nullptr, per_head, rstd,
-                                                                              h * dim, d, rot_dims, halves, inv_freq, pos));
+                                                                              h * dim, d, rot_dims, halves, inv_freq, pos, mscale));
   }
   if (!writes) return;
   if (page < 0 || page >= n_pages) {
@@ -179,14 +180,14 @@ __global__ void qk_prep_kernel(const float* fused, long long ld, int k_col, int 
     if (after) {
       float ss = 0.f;
       for (int d = lane; d < dim; d += 32) {
-        const float v = prep_element(row + k_col, nullptr, true, 1.f, h * dim, d, rot_dims, halves, inv_freq, pos);
+        const float v = prep_element(row + k_col, nullptr, true, 1.f, h * dim, d, rot_dims, halves, inv_freq, pos, mscale);
         ss += v * v;
       }
       post = 1.0f / sqrtf(warp_sum(ss) / (float)dim + eps);
     }
     for (int d = lane; d < dim; d += 32)
       dst[d] = from_f32<TC>(post * prep_element(row + k_col, normed ? k_gain : nullptr, per_head, rstd, h * dim, d, rot_dims,
-                                                halves, inv_freq, pos));
+                                                halves, inv_freq, pos, mscale));
   }
   for (int i = threadIdx.x; i < G * vdim; i += blockDim.x) {
     const int g = i / vdim, d = i - g * vdim;
@@ -482,7 +483,7 @@ GB_OP(gb_op_embed_scaled) {
 
 // a0 fused rows (f32) [q (heads * maps * dim) | ...], a1 their stride, a2 column of the keys (kv_heads * maps * dim),
 // a3 column of the values (kv_heads * vdim), a4 gain of the query norm or 0, a5 gain of the key norm or 0, a6 inv_freq
-// [rot_dims / 2], a7 rot_dims, a8 token -> request, a9 token -> position, a10 block table, a11 its entries per request,
+// [rot_dims / 2] and behind them a factor on cosines and sines, a7 rot_dims, a8 token -> request, a9 token -> position, a10 block table, a11 its entries per request,
 // a12 page size, a13 key pages or 0 (a layer that reads another layer's cache writes none), a14 value pages, a15 number
 // of pages, a16 tokens, a17 heads, a18 kv heads, a19 dim, a20 vdim, a21 q out [tokens, heads * maps * dim], a22 maps
 // (heads of `dim` entries side by side in one query or key head; 0 means 1); flags bit 0: norm over the whole

@@ -90,11 +90,13 @@ struct GemmParams {
 };
 
 // The function of a feed-forward without a gate, in the epilogue of its first product.
-enum Act : int { ACT_NONE = 0, ACT_RELU2 = 1 };
+enum Act : int { ACT_NONE = 0, ACT_RELU2 = 1, ACT_GELU = 2 };      // (gelu: the exact one)
 __device__ __forceinline__ float apply_act(int act, float v) {
   if (act == ACT_RELU2) {
     v = fmaxf(v, 0.f);
     v *= v;
+  } else if (act == ACT_GELU) {
+    v = 0.5f * v * (1.0f + erff(v * 0.7071067811865476f));
   }
   return v;
 }
@@ -1215,7 +1217,7 @@ static int linear_tc_impl(const void* X, long long ldx, const void* W, long long
   if (defer && mode == OUT_SWIGLU)
     GB_FAIL(GB_ERR_ARG, "gb_linear_tc: only a plain or an accumulating product can be deferred");
   const int act = (flags >> 8) & 255;
-  if (act > ACT_RELU2 || (act && (mode != OUT_BF16 || defer)))
+  if (act > ACT_GELU || (act && (mode != OUT_BF16 || defer)))
     GB_FAIL(GB_ERR_ARG, "gb_linear_tc: function %d of an output of mode %d (deferred: %d)", act, mode, defer);
 
   CUtensorMap tw, tx;

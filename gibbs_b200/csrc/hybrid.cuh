@@ -10,6 +10,8 @@
 // directly with the same operand list.  It launches on ctx->stream and returns the number of kernels
 // launched, or a negative code with the message in gb_last_error().
 #pragma once
+#include <cstring>
+
 #include "common.cuh"
 #include "gb_plan_op.h"
 
@@ -20,6 +22,7 @@ template <typename T> static inline T* op_ptr(long long v) { return reinterpret_
 __device__ __forceinline__ float hy_sigmoid(float x) { return 1.0f / (1.0f + expf(-x)); }
 __device__ __forceinline__ float hy_silu(float x) { return x / (1.0f + expf(-x)); }
 __device__ __forceinline__ float hy_softplus(float x) { return x > 20.f ? x : log1pf(expf(x)); }
+__device__ __forceinline__ float hy_gelu(float z) { return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f)); }
 __device__ __forceinline__ float hy_gelu_tanh(float z) {
   return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
@@ -28,6 +31,107 @@ __device__ __forceinline__ float hy_clamped_glu(float g, float u, float alpha, f
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
   return g * hy_sigmoid(alpha * g) * (u + up_add);
+}
+
+// Functions of a feed-forward's units by number.
+enum { ACT_GELU_ERF = 0, ACT_GELU_TANH = 1, ACT_SILU = 2, ACT_RELU = 3, ACT_RELU2 = 4, ACT_NONE = 5 };
+
+__device__ __forceinline__ float hy_act(float z, int kind) {
+  switch (kind) {
+    case ACT_GELU_ERF: return hy_gelu(z);
+    case ACT_GELU_TANH: return hy_gelu_tanh(z);
+    case ACT_SILU: return hy_silu(z);
+    case ACT_RELU: return fmaxf(z, 0.f);
+    case ACT_RELU2: z = fmaxf(z, 0.f); return z * z;
+    default: return z;
+  }
+}
+
+enum { NORM_LAYER = 0, NORM_RMS = 1 };
+
+// `then`: the norm in front of the NEXT sublayer, taken of the new rows while they are in registers
+// (out = norm(x) * gain), so that it needs no kernel and no second trip of its own.
+struct ThenNorm {
+  const float* gain;
+  void* out;
+  int out_dtype, kind;
+  float eps;
+};
+
+// (as five operands of an operation, the last one the bits of the 32-bit eps)
+static inline ThenNorm hy_then_of(long long gain, long long out, long long dtype, long long kind, long long eps_bits) {
+  ThenNorm t;
+  t.gain = op_ptr<const float>(gain);
+  t.out = op_ptr<void>(out);
+  t.out_dtype = (int)dtype;
+  t.kind = (int)kind;
+  const unsigned b = (unsigned)eps_bits;
+  memcpy(&t.eps, &b, sizeof(float));
+  return t;
+}
+static inline bool hy_then_vec(const ThenNorm& t) {
+  return t.gain == nullptr || (((uintptr_t)t.gain | (uintptr_t)t.out) & 15) == 0;
+}
+// Threads of a block that holds a row of `dim` values in pieces of four (up to 256, whole warps).
+static inline int hy_row_threads(int dim) {
+  const int t = (dim / 4 + 31) / 32 * 32;
+  return t < 32 ? 32 : t > 256 ? 256 : t;
+}
+
+// A row in the block's registers, NV pieces of four values a thread (piece i at 4 * (threadIdx.x + i * blockDim.x)).
+template <int NV>
+__device__ __forceinline__ void hy_then_norm(const float4 (&v)[NV], int dim, const ThenNorm& then, size_t row, float* scratch) {
+  float mean = 0.f;
+  if (then.kind == NORM_LAYER) {
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+      if (4 * (int)(threadIdx.x + i * blockDim.x) < dim) s += (v[i].x + v[i].y) + (v[i].z + v[i].w);
+    mean = block_sum(s, scratch) / (float)dim;
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    if (4 * (int)(threadIdx.x + i * blockDim.x) >= dim) continue;
+    const float p = v[i].x - mean, q = v[i].y - mean, c = v[i].z - mean, e = v[i].w - mean;
+    ss += (p * p + q * q) + (c * c + e * e);
+  }
+  const float rstd = 1.0f / sqrtf(block_sum(ss, scratch) / (float)dim + then.eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int d = 4 * (threadIdx.x + i * blockDim.x);
+    if (d >= dim) continue;
+    const float4 g = *reinterpret_cast<const float4*>(then.gain + d);
+    const float r0 = (v[i].x - mean) * rstd * g.x, r1 = (v[i].y - mean) * rstd * g.y;
+    const float r2 = (v[i].z - mean) * rstd * g.z, r3 = (v[i].w - mean) * rstd * g.w;
+    if (then.out_dtype == GB_BF16) {
+      __nv_bfloat162 lo = __floats2bfloat162_rn(r0, r1), hi = __floats2bfloat162_rn(r2, r3);
+      uint2 w;
+      w.x = *reinterpret_cast<unsigned*>(&lo);
+      w.y = *reinterpret_cast<unsigned*>(&hi);
+      *reinterpret_cast<uint2*>((bf16*)then.out + row * dim + d) = w;
+    } else {
+      *reinterpret_cast<float4*>((float*)then.out + row * dim + d) = make_float4(r0, r1, r2, r3);
+    }
+  }
+}
+
+// The same for a row of any length that this block's threads have just written, each its own entries threadIdx.x + i * blockDim.x.
+__device__ __forceinline__ void hy_then_norm_row(const float* o, int dim, const ThenNorm& then, size_t row, float* scratch) {
+  float mean = 0.f;
+  if (then.kind == NORM_LAYER) {
+    float s = 0.f;
+    for (int d = threadIdx.x; d < dim; d += blockDim.x) s += o[d];
+    mean = block_sum(s, scratch) / (float)dim;
+  }
+  float ss = 0.f;
+  for (int d = threadIdx.x; d < dim; d += blockDim.x) ss += (o[d] - mean) * (o[d] - mean);
+  const float rstd = 1.0f / sqrtf(block_sum(ss, scratch) / (float)dim + then.eps);
+  for (int d = threadIdx.x; d < dim; d += blockDim.x) {
+    const float h = (o[d] - mean) * rstd * then.gain[d];
+    if (then.out_dtype == GB_BF16) ((bf16*)then.out)[row * dim + d] = __float2bfloat16_rn(h);
+    else ((float*)then.out)[row * dim + d] = h;
+  }
 }
 
 // A 64 x 64 tile of C = A . B^T on the CUDA cores in 32-bit, for 256 threads.  Row i of the tile is

@@ -9,6 +9,8 @@
 //  gb_op_linear_scan         the recurrence
 //  gb_op_forget_write_gates  what enters it when the forget gate decides what is written: per channel
 //                            f = l + (1 - l) sigmoid(z + bias), g = f, k = 1 - f; and q = silu(q).  All in 32-bit.
+//  gb_op_low_rank_decays     g = sigmoid(W z + bias)^(1 / tau) per channel, z a few entries a token: the second half of a
+//                            low-rank projection and the decay in one kernel.  All in 32-bit.
 //  gb_op_exp_gates           what enters it with exponential gates kept in range by a running maximum, per head:
 //                            i = cap tanh((zi + bi) / cap), f = log sigmoid(cap tanh((zf + bf) / cap)),
 //                            m_t = max(f + m_(t-1), i), g = exp(f + m_(t-1) - m_t), w = exp(i - m_t), and exp(-m_t)
@@ -383,6 +385,43 @@ __global__ void forget_write_gates_kernel(float* q, long long ldq, float* f, lon
   k[(size_t)t * ldk + c] = (1.f - l) * hy_sigmoid(-z);   // (1 - f without the cancellation where f is near one)
 }
 
+// A thread takes one channel of LD_TOK tokens: its row of W is read once for them, z from shared memory.
+constexpr int LD_TOK = 8, LD_THREADS = 128;
+
+template <typename TW>
+__global__ void __launch_bounds__(LD_THREADS)
+low_rank_decays_kernel(const float* z, long long ldz, const TW* __restrict__ W, const float* __restrict__ bias, float* g,
+                       long long ldg, int n, int width, int rank, float inv_tau) {
+  extern __shared__ __align__(16) float zs[];                        // [rank][LD_TOK]
+  pdl_trigger();
+  const int c = blockIdx.x * LD_THREADS + threadIdx.x, t0 = blockIdx.y * LD_TOK;
+  const float b = c < width ? bias[c] : 0.f;
+  pdl_wait();
+  for (int i = threadIdx.x; i < rank * LD_TOK; i += LD_THREADS) {
+    const int tt = i / rank, r = i - tt * rank;
+    zs[r * LD_TOK + tt] = t0 + tt < n ? z[(size_t)(t0 + tt) * ldz + r] : 0.f;
+  }
+  __syncthreads();
+  if (c >= width) return;
+  float acc[LD_TOK];
+#pragma unroll
+  for (int u = 0; u < LD_TOK; ++u) acc[u] = b;
+  const TW* w = W + (size_t)c * rank;
+#pragma unroll 8
+  for (int r = 0; r < rank; ++r) {
+    const float wr = to_f32(w[r]);
+    const float4 a = *reinterpret_cast<const float4*>(zs + r * LD_TOK), e = *reinterpret_cast<const float4*>(zs + r * LD_TOK + 4);
+    acc[0] = fmaf(wr, a.x, acc[0]); acc[1] = fmaf(wr, a.y, acc[1]); acc[2] = fmaf(wr, a.z, acc[2]); acc[3] = fmaf(wr, a.w, acc[3]);
+    acc[4] = fmaf(wr, e.x, acc[4]); acc[5] = fmaf(wr, e.y, acc[5]); acc[6] = fmaf(wr, e.z, acc[6]); acc[7] = fmaf(wr, e.w, acc[7]);
+  }
+#pragma unroll
+  for (int u = 0; u < LD_TOK; ++u) {
+    // log sigmoid(x) = min(x, 0) - log1p(exp(-|x|))
+    const float x = acc[u];
+    if (t0 + u < n) g[(size_t)(t0 + u) * ldg + c] = expf((fminf(x, 0.f) - log1pf(expf(-fabsf(x)))) * inv_tau);
+  }
+}
+
 // A block per (request, head).  m -> max(m + F, I) is closed under composition ((F1, I1) then (F2, I2) is
 // (F1 + F2, max(I1 + F2, I2))), so a round of tokens, one a thread, is combined by scans over the lanes of each warp and
 // then over the warps.
@@ -563,5 +602,23 @@ GB_OP(gb_op_exp_gates) {
             op_ptr<const int>(a[8]), op_ptr<const int>(a[9]), op_ptr<const int>(a[10]), op_ptr<float>(a[11]),
             op_ptr<float>(a[12]), op_ptr<float>(a[13]), H, (float)f[0]);
   GB_CHECK_LAUNCH("exp_gates");
+  return 1;
+}
+
+// a0 z (f32 [t, rank] at a row stride), a1 that stride, a2 W [width, rank], a3 its dtype, a4 bias [width] (f32), a5 decays
+// out (f32), a6 their row stride, a7 tokens, a8 width, a9 rank; f0 tau
+GB_OP(gb_op_low_rank_decays) {
+  const int n = (int)a[7], width = (int)a[8], rank = (int)a[9];
+  if (n <= 0) return 0;
+  if (!(f[0] > 0.0)) GB_FAIL(GB_ERR_ARG, "low_rank_decays: a temperature of %g", f[0]);
+  const size_t smem = sizeof(float) * LD_TOK * (size_t)rank;
+  if (rank < 1 || smem > 48 * 1024) GB_FAIL(GB_ERR_ARG, "low_rank_decays: rank %d (1 to 1536)", rank);
+  const dim3 grid(gb_div_up(width, LD_THREADS), gb_div_up(n, LD_TOK));
+#define DECAYS(TW)                                                                                                      \
+  gb_launch(low_rank_decays_kernel<TW>, grid, dim3(LD_THREADS), smem, ctx->stream, op_ptr<const float>(a[0]), a[1],      \
+            op_ptr<const TW>(a[2]), op_ptr<const float>(a[4]), op_ptr<float>(a[5]), a[6], n, width, rank, (float)(1.0 / f[0]))
+  if (a[3] == GB_BF16) DECAYS(bf16); else DECAYS(float);
+#undef DECAYS
+  GB_CHECK_LAUNCH("low_rank_decays");
   return 1;
 }

@@ -9,11 +9,12 @@
 //  gb_op_moe_sort      (token, choice) pairs ordered by expert: offsets[E + 1], the pair behind every
 //                      row, the row of every pair
 //  gb_op_moe_gather    rows[row] = weight * h[token]: the weight multiplies the expert's INPUT
-//  gb_op_moe_experts   per expert, over its rows: either act = glu(rows W_gate^T, rows W_up^T) with
-//                      clamps, or out = rows W_down^T (32-bit)
+//  gb_op_moe_experts   per expert, over its rows: act = glu(rows W_gate^T, rows W_up^T) with clamps, or act =
+//                      function(rows W_up^T) for experts without a gate, or out = rows W_down^T (32-bit)
 //  gb_op_moe_combine   y[token] = sum over its choices of out[row] (+ gate * shared[token])
 //  gb_op_moe_combine_weighted  y[token] (+)= sum over its choices of weight * out[row], where the weight multiplies
-//                      the expert's OUTPUT; a choice beyond the real experts contributes weight * h[token]
+//                      the expert's OUTPUT; a choice beyond the real experts contributes weight * h[token]; optionally
+//                      + shared[token], and the norm in front of the next sublayer taken of the new rows
 //
 // A row's result does not depend on which rows share its tile (one accumulator per output walking k
 // upwards), so the order in which pairs land inside an expert's range does not matter.
@@ -60,11 +61,12 @@ __global__ void moe_route_kernel(const float* logits, long long ld, int n, int E
 // `normalise`: 0 a chosen output's weight is its score, 1 the score divided by the sum of the chosen scores, 2 the
 // softmax over the chosen scores alone.  The choice is made on
 // score + correction; with `groups` > 1 the outputs form that many equal groups of neighbours, a group's mark is
-// its largest choice score, and only outputs of the `keep` best groups can be chosen.  The weight of a chosen
-// output is its score without the correction, not renormalised.  Ties go to the lower index.
+// its largest choice score (or, with `mark_two`, the sum of its two largest), and only outputs of the `keep` best groups
+// can be chosen.  The weight of a chosen output is its score without the correction, not renormalised, times
+// `weight_scale`.  Ties go to the lower index.
 __global__ void moe_route_grouped_kernel(const float* logits, long long ld, int n, int n_out, int top, int scores,
                                          const float* __restrict__ correction, int groups, int keep, int* idx,
-                                         float* weight, int normalise) {
+                                         float* weight, int normalise, int mark_two, float weight_scale) {
   extern __shared__ float route_sm[];                    // per warp: scores [n_out], choice scores [n_out], group marks
   pdl_trigger();
   pdl_wait();
@@ -97,9 +99,12 @@ __global__ void moe_route_grouped_kernel(const float* logits, long long ld, int 
   const int gs = n_out / groups;
   if (groups > 1 && keep < groups) {
     for (int g = lane; g < groups; g += 32) {
-      float b = -INFINITY;
-      for (int e = g * gs; e < (g + 1) * gs; ++e) b = fmaxf(b, c[e]);
-      mark[g] = b;
+      float b = -INFINITY, second = -INFINITY;
+      for (int e = g * gs; e < (g + 1) * gs; ++e) {
+        second = fmaxf(second, fminf(b, c[e]));
+        b = fmaxf(b, c[e]);
+      }
+      mark[g] = mark_two && gs > 1 ? b + second : b;
     }
     __syncwarp();
     // the `keep` best groups stay open: the mark of a group that is picked becomes +infinity, which no score
@@ -140,7 +145,7 @@ __global__ void moe_route_grouped_kernel(const float* logits, long long ld, int 
     }
     if (lane == 0) {
       idx[(size_t)t * top + k] = be;
-      weight[(size_t)t * top + k] = s[be];
+      weight[(size_t)t * top + k] = normalise ? s[be] : s[be] * weight_scale;
       c[be] = -INFINITY;                                   // taken
     }
     __syncwarp();
@@ -157,7 +162,7 @@ __global__ void moe_route_grouped_kernel(const float* logits, long long ld, int 
     } else {
       for (int k = 0; k < top; ++k) sum += w[k];
     }
-    for (int k = 0; k < top; ++k) w[k] = w[k] / sum;
+    for (int k = 0; k < top; ++k) w[k] = w[k] / sum * weight_scale;
   }
 }
 
@@ -251,9 +256,10 @@ __global__ void moe_experts_glu_kernel(const TA* rows, long long ldr, const TW* 
   }
 }
 
-template <typename TA, typename TW>
+// out = rows W^T (32-bit), or function(rows W^T) in the rows' type
+template <typename TA, typename TW, typename TO>
 __global__ void moe_experts_down_kernel(const TA* act, long long lda, const TW* __restrict__ W, const int* offsets, int E,
-                                        float* out, long long ldo, int width, int ff) {
+                                        TO* out, long long ldo, int width, int ff, int fn) {
   pdl_trigger();
   pdl_wait();
   int e, r0, r1;
@@ -272,7 +278,7 @@ __global__ void moe_experts_down_kernel(const TA* act, long long lda, const TW* 
 #pragma unroll
     for (int c = 0; c < 4; ++c) {
       const int col = c0 + tx * 4 + c;
-      if (col < width) out[(size_t)row * ldo + col] = acc[r][c];
+      if (col < width) out[(size_t)row * ldo + col] = from_f32<TO>(hy_act(acc[r][c], fn));
     }
   }
 }
@@ -291,23 +297,81 @@ __global__ void moe_combine_kernel(const float* out, long long ldo, const int* p
   }
 }
 
+// rows of any length; `then`: the norm in front of the next sublayer, of the new row
 template <typename T>
-__global__ void moe_combine_weighted_kernel(const float* out, long long ldo, const int* pair_row, const int* idx,
-                                            const float* weight, const T* h, long long ldh, float* y, long long ldy,
-                                            int width, int top, int E, int accumulate) {
+__global__ void moe_combine_weighted_any_kernel(const float* out, long long ldo, const int* pair_row, const int* idx,
+                                                const float* weight, const T* h, long long ldh, float* y, long long ldy,
+                                                int width, int top, int E, int accumulate, const float* shared,
+                                                long long lds, ThenNorm then) {
+  __shared__ float scratch[32];
   pdl_trigger();
   pdl_wait();
-  const int t = blockIdx.x;
+  const size_t t = blockIdx.x;
+  float* o = y + t * ldy;
   for (int d = threadIdx.x; d < width; d += blockDim.x) {
     float v = 0.f;
     for (int k = 0; k < top; ++k) {
-      const size_t p = (size_t)t * top + k;
-      const float src = idx[p] < E ? out[(size_t)pair_row[p] * ldo + d] : to_f32(h[(size_t)t * ldh + d]);
+      const size_t p = t * top + k;
+      const float src = idx[p] < E ? out[(size_t)pair_row[p] * ldo + d] : to_f32(h[t * ldh + d]);
       v = fmaf(weight[p], src, v);
     }
-    float* o = y + (size_t)t * ldy + d;
-    *o = accumulate ? *o + v : v;
+    if (shared) v += shared[t * lds + d];
+    o[d] = accumulate ? o[d] + v : v;
   }
+  if (then.gain != nullptr) hy_then_norm_row(o, width, then, t, scratch);
+}
+
+__device__ __forceinline__ float4 load4_f32(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4_f32(const bf16* p) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+  const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+  return make_float4(lo.x, lo.y, hi.x, hi.y);
+}
+
+// The same arithmetic per value for rows of 16-byte pieces, the new row in the block's registers.
+template <typename T, int NV>
+__global__ void __launch_bounds__(256)
+moe_combine_weighted_kernel(const float* out, long long ldo, const int* pair_row, const int* idx, const float* weight,
+                            const T* h, long long ldh, float* y, long long ldy, int width, int top, int E, int accumulate,
+                            const float* shared, long long lds, ThenNorm then) {
+  __shared__ float scratch[32];
+  pdl_trigger();
+  pdl_wait();
+  const size_t t = blockIdx.x;
+  float* o = y + t * ldy;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 v[NV], own[NV], sh[NV];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int d = 4 * (threadIdx.x + i * blockDim.x);
+    v[i] = zero;
+    own[i] = d < width && accumulate ? load4_f32(o + d) : zero;
+    sh[i] = d < width && shared ? load4_f32(shared + t * lds + d) : zero;
+  }
+  for (int k = 0; k < top; ++k) {
+    const size_t p = t * top + k;
+    const float w = weight[p];
+    const bool real = idx[p] < E;
+    const float* src = out + (size_t)pair_row[p] * ldo;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int d = 4 * (threadIdx.x + i * blockDim.x);
+      if (d >= width) continue;
+      const float4 x = real ? load4_f32(src + d) : load4_f32(h + t * ldh + d);
+      v[i].x = fmaf(w, x.x, v[i].x); v[i].y = fmaf(w, x.y, v[i].y);
+      v[i].z = fmaf(w, x.z, v[i].z); v[i].w = fmaf(w, x.w, v[i].w);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int d = 4 * (threadIdx.x + i * blockDim.x);
+    if (d >= width) continue;
+    if (shared) { v[i].x += sh[i].x; v[i].y += sh[i].y; v[i].z += sh[i].z; v[i].w += sh[i].w; }
+    if (accumulate) { v[i].x += own[i].x; v[i].y += own[i].y; v[i].z += own[i].z; v[i].w += own[i].w; }
+    *reinterpret_cast<float4*>(o + d) = v[i];
+  }
+  if (then.gain != nullptr) hy_then_norm<NV>(v, width, then, t, scratch);
 }
 
 }  // namespace
@@ -315,7 +379,8 @@ __global__ void moe_combine_weighted_kernel(const float* out, long long ldo, con
 // a0 logits (f32), a1 their row stride, a2 tokens, a3 router outputs (experts and identity outputs), a4 top, a5 scores
 // (0 sigmoid, 1 softmax, 2 the logits), a6 correction [outputs] (f32) or 0, a7 groups (1: none), a8 groups kept, a9 chosen
 // outputs [tokens, top] (int32), a10 their weights (f32), a11 how the chosen scores become weights: 0 as they are, 1
-// divided by their sum, 2 their softmax
+// divided by their sum, 2 their softmax, a12 a group's mark: 0 its largest choice score, 1 the sum of its two largest;
+// f0 factor on the weights (0 means 1)
 GB_OP(gb_op_moe_route_grouped) {
   const int n = (int)a[2], n_out = (int)a[3], top = (int)a[4];
   int groups = (int)a[7], keep = (int)a[8];
@@ -330,7 +395,7 @@ GB_OP(gb_op_moe_route_grouped) {
   const size_t smem = sizeof(float) * warps * (2 * (size_t)n_out + groups);
   gb_launch(moe_route_grouped_kernel, dim3(gb_div_up(n, warps)), dim3(32 * warps), smem, ctx->stream,
             op_ptr<const float>(a[0]), a[1], n, n_out, top, (int)a[5], op_ptr<const float>(a[6]), groups, keep,
-            op_ptr<int>(a[9]), op_ptr<float>(a[10]), (int)a[11]);
+            op_ptr<int>(a[9]), op_ptr<float>(a[10]), (int)a[11], (int)a[12], f[0] != 0.0 ? (float)f[0] : 1.f);
   GB_CHECK_LAUNCH("moe_route_grouped");
   return 1;
 }
@@ -377,8 +442,9 @@ GB_OP(gb_op_moe_gather) {
 
 // a0 input rows, a1 their stride, a2 their dtype, a3 weights [E, out features, in features], a4 their dtype,
 // a5 offsets [E + 1], a6 experts, a7 out, a8 its row stride, a9 tokens, a10 features out (GLU: ff), a11 features in,
-// a12 mode (0: GLU over [gate rows | up rows], out in the input's dtype; 1: plain, out f32), a13 top, a14 (GLU) 1 when
-// gate and up rows alternate in blocks of 64 instead; f0 alpha, f1 limit, f2 what is added to u
+// a12 mode (0: GLU over [gate rows | up rows], out in the input's dtype; 1: plain, out f32; 2: a function of the sums, out
+// in the input's dtype), a13 top, a14 (GLU) 1 when gate and up rows alternate in blocks of 64 instead, (mode 2) the
+// function's number; f0 alpha, f1 limit, f2 what is added to u
 GB_OP(gb_op_moe_experts) {
   const int pairs = (int)(a[9] * a[13]), E = (int)a[6], n_out = (int)a[10], n_in = (int)a[11], mode = (int)a[12];
   if (pairs <= 0) return 0;
@@ -389,14 +455,19 @@ GB_OP(gb_op_moe_experts) {
   gb_launch(moe_experts_glu_kernel<TA, TW>, dim3(gb_div_up(n_out, 32), tiles), dim3(256), 0, ctx->stream,          \
             op_ptr<const TA>(a[0]), a[1], op_ptr<const TW>(a[3]), op_ptr<const int>(a[5]), E, op_ptr<TA>(a[7]), a[8], \
             n_out, n_in, (float)f[0], (float)f[1], (float)f[2], (int)a[14])
-#define DOWN(TA, TW)                                                                                                \
-  gb_launch(moe_experts_down_kernel<TA, TW>, dim3(gb_div_up(n_out, 64), tiles), dim3(256), 0, ctx->stream,         \
-            op_ptr<const TA>(a[0]), a[1], op_ptr<const TW>(a[3]), op_ptr<const int>(a[5]), E, op_ptr<float>(a[7]),   \
-            a[8], n_out, n_in)
+#define DOWN(TA, TW, TO, FN)                                                                                        \
+  gb_launch(moe_experts_down_kernel<TA, TW, TO>, dim3(gb_div_up(n_out, 64), tiles), dim3(256), 0, ctx->stream,     \
+            op_ptr<const TA>(a[0]), a[1], op_ptr<const TW>(a[3]), op_ptr<const int>(a[5]), E, op_ptr<TO>(a[7]),      \
+            a[8], n_out, n_in, FN)
   if (mode == 0) {
     if (abf) GLU(bf16, bf16); else if (wbf) GLU(float, bf16); else GLU(float, float);
+  } else if (mode == 2) {
+    const int fn = (int)a[14];
+    if (fn < 0 || fn > ACT_NONE) GB_FAIL(GB_ERR_ARG, "moe_experts: function %d", fn);
+    if (abf) DOWN(bf16, bf16, bf16, fn); else if (wbf) DOWN(float, bf16, float, fn); else DOWN(float, float, float, fn);
   } else {
-    if (abf) DOWN(bf16, bf16); else if (wbf) DOWN(float, bf16); else DOWN(float, float);
+    if (abf) DOWN(bf16, bf16, float, ACT_NONE); else if (wbf) DOWN(float, bf16, float, ACT_NONE);
+    else DOWN(float, float, float, ACT_NONE);
   }
 #undef GLU
 #undef DOWN
@@ -418,19 +489,30 @@ GB_OP(gb_op_moe_combine) {
 
 // a0 expert outputs by row (f32), a1 their stride, a2 pair -> row, a3 chosen outputs [tokens, top], a4 their weights,
 // a5 the feed-forward's input h, a6 its row stride, a7 its dtype, a8 y (f32), a9 its row stride, a10 tokens, a11 width,
-// a12 top, a13 real experts (a choice from here on returns h); flags bit 0: add into y
+// a12 top, a13 real experts (a choice from here on returns h), a14 an output added for every token (f32) or 0, a15 its row
+// stride, a16 gain of a norm taken of the new rows or 0: none, a17 its output [tokens, width], a18 that dtype, a19 its kind
+// (0 layer norm, 1 RMS norm), a20 its eps (the bits of a 32-bit float); flags bit 0: add into y
 GB_OP(gb_op_moe_combine_weighted) {
   const int n = (int)a[10], width = (int)a[11];
   if (n <= 0) return 0;
-  const dim3 grid(n), block(width <= 256 ? 64 : 256);
-  if (a[7] == GB_BF16)
-    gb_launch(moe_combine_weighted_kernel<bf16>, grid, block, 0, ctx->stream, op_ptr<const float>(a[0]), a[1],
-              op_ptr<const int>(a[2]), op_ptr<const int>(a[3]), op_ptr<const float>(a[4]), op_ptr<const bf16>(a[5]), a[6],
-              op_ptr<float>(a[8]), a[9], width, (int)a[12], (int)a[13], flags & 1);
-  else
-    gb_launch(moe_combine_weighted_kernel<float>, grid, block, 0, ctx->stream, op_ptr<const float>(a[0]), a[1],
-              op_ptr<const int>(a[2]), op_ptr<const int>(a[3]), op_ptr<const float>(a[4]), op_ptr<const float>(a[5]), a[6],
-              op_ptr<float>(a[8]), a[9], width, (int)a[12], (int)a[13], flags & 1);
+  const ThenNorm then = hy_then_of(a[16], a[17], a[18], a[19], a[20]);
+  const bool vec = width % 4 == 0 && width <= 4096 && a[1] % 4 == 0 && a[6] % 4 == 0 && a[9] % 4 == 0 && a[15] % 4 == 0 &&
+                   ((a[0] | a[8] | a[14]) & 15) == 0 && (a[5] & (a[7] == GB_BF16 ? 7 : 15)) == 0 && hy_then_vec(then);
+#define COMBINE(T, KERNEL, THREADS)                                                                                     \
+  gb_launch(KERNEL, dim3(n), dim3(THREADS), 0, ctx->stream, op_ptr<const float>(a[0]), a[1], op_ptr<const int>(a[2]),    \
+            op_ptr<const int>(a[3]), op_ptr<const float>(a[4]), op_ptr<const T>(a[5]), a[6], op_ptr<float>(a[8]), a[9],  \
+            width, (int)a[12], (int)a[13], flags & 1, op_ptr<const float>(a[14]), a[15], then)
+  const int threads = hy_row_threads(width);
+#define COMBINE_OF(T)                                                                                                   \
+  do {                                                                                                                  \
+    if (!vec) COMBINE(T, moe_combine_weighted_any_kernel<T>, width <= 256 ? 64 : 256);                                  \
+    else if (width <= 4 * threads) COMBINE(T, (moe_combine_weighted_kernel<T, 1>), threads);                            \
+    else if (width <= 8 * threads) COMBINE(T, (moe_combine_weighted_kernel<T, 2>), threads);                            \
+    else COMBINE(T, (moe_combine_weighted_kernel<T, 4>), threads);                                                      \
+  } while (0)
+  if (a[7] == GB_BF16) COMBINE_OF(bf16); else COMBINE_OF(float);
+#undef COMBINE_OF
+#undef COMBINE
   GB_CHECK_LAUNCH("moe_combine_weighted");
   return 1;
 }

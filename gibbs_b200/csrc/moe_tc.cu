@@ -11,8 +11,9 @@
 // for those is not stored.
 //
 // The weight is the M side of the MMA (128 weight rows per tile, one accumulator lane each), the
-// token rows the N side (BN per tile), as in gemm_tc.cu.  Two epilogues:
+// token rows the N side (BN per tile), as in gemm_tc.cu.  Three epilogues:
 //   plain   out[row, n] = acc            (32-bit; the experts' down projections)
+//   unit    act[row, n] = function(acc)  (bfloat16; the first product of experts without a gate)
 //   GLU     act[row, f] = g' sigmoid(alpha g') (u' + up_add), g' = min(g, limit), u' = clamp(u, +-limit),
 //           for weights whose rows alternate in blocks of 64 between gate and up of the same 64 features
 //           (lanes 0-63 of a tile hold g, lanes 64-127 u).
@@ -33,7 +34,8 @@ constexpr int STATUS_TIMEOUT = 24;
 struct GroupedParams {
   const int* offsets;
   int E, rows_per_expert, n_valid;   // weight rows per expert in the stacked matrix; rows that exist per expert
-  int mode;                          // 0 GLU, 1 plain
+  int mode;                          // 0 GLU, 1 plain, 2 a function of the sums
+  int fn;                            // (mode 2) the function's number
   void* out; long long ldo;
   int total_kb;
   float alpha, limit, up_add;
@@ -165,6 +167,19 @@ moe_experts_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_c
             if (c0 + j < cols) out[(size_t)(r0 + c0 + j) * p.ldo + n] = v[j];
         }
       }
+    } else if (good && p.mode == 2) {
+      const int n = blockIdx.x * BM + row;
+      bf16* out = (bf16*)p.out;
+#pragma unroll 1
+      for (int c0 = 0; c0 < cols; c0 += 16) {
+        float v[16];
+        tmem_ld_16(tmem_base + ((uint32_t)(32 * q) << 16) + (uint32_t)c0, v);
+        if (n < p.n_valid) {
+#pragma unroll
+          for (int j = 0; j < 16; ++j)
+            if (c0 + j < cols) out[(size_t)(r0 + c0 + j) * p.ldo + n] = __float2bfloat16_rn(hy_act(v[j], p.fn));
+        }
+      }
     } else if (good) {
       // u of one 16-column chunk through shared memory (the pipeline's first stage is free once the
       // accumulator is complete); the threads of lanes 0-63 hold g and finish the unit
@@ -261,7 +276,7 @@ int launch(const CUtensorMap& tw, const CUtensorMap& tx, const GroupedParams& p,
 }  // namespace
 
 // Whether gb_op_moe_experts_tc takes these sizes (mode 0: GLU, the weights' gate and up rows alternating
-// in blocks of 64; mode 1: plain).  K: features in; ld: row strides of the rows and of the weights.
+// in blocks of 64; mode 1: plain; mode 2: a function of the sums).  K: features in; ld: row strides of the rows and of the weights.
 GB_API int gb_moe_experts_tc_supported(int mode, int n_out, int K, long long ld_rows, long long ld_w) {
   if (K % 8 || ld_rows % 8 || ld_w % 8) return 0;
   if (mode == 0 && n_out % 64) return 0;
@@ -270,8 +285,8 @@ GB_API int gb_moe_experts_tc_supported(int mode, int n_out, int K, long long ld_
 
 // a0 input rows (bf16), a1 their stride, a2 rows the matrix has room for, a3 weights [E, rows per expert, K]
 // (bf16, contiguous), a4 unused, a5 offsets [E + 1], a6 experts, a7 out, a8 its row stride, a9 tokens, a10 features out
-// (GLU: ff), a11 features in (K), a12 mode (0: GLU, out bf16 [rows, ff]; 1: plain, out f32), a13 top; f0 alpha,
-// f1 limit, f2 what is added to u
+// (GLU: ff), a11 features in (K), a12 mode (0: GLU, out bf16 [rows, ff]; 1: plain, out f32; 2: a function of the sums, out
+// bf16), a13 top, a14 (mode 2) the function's number; f0 alpha, f1 limit, f2 what is added to u
 GB_OP(gb_op_moe_experts_tc) {
   const int pairs = (int)(a[9] * a[13]), E = (int)a[6], n_out = (int)a[10], K = (int)a[11], mode = (int)a[12];
   if (pairs <= 0) return 0;
@@ -296,7 +311,8 @@ GB_OP(gb_op_moe_experts_tc) {
     GB_FAIL(GB_ERR_CUDA, "moe_experts_tc: cuTensorMapEncodeTiled failed (rows)");
   GroupedParams p;
   p.offsets = op_ptr<const int>(a[5]);
-  p.E = E; p.rows_per_expert = rows_per_expert; p.n_valid = n_out; p.mode = mode;
+  p.E = E; p.rows_per_expert = rows_per_expert; p.n_valid = n_out; p.mode = mode; p.fn = (int)a[14];
+  if (mode < 0 || mode > 2 || (mode == 2 && (p.fn < 0 || p.fn > ACT_NONE))) GB_FAIL(GB_ERR_ARG, "moe_experts_tc: mode %d, function %d", mode, p.fn);
   p.out = op_ptr<void>(a[7]); p.ldo = a[8];
   p.total_kb = gb_div_up(K, BK);
   p.alpha = (float)f[0]; p.limit = (float)f[1]; p.up_add = (float)f[2];

@@ -11,12 +11,13 @@
 //  gb_op_scaled_sum      x += mult * (s1 * y1 + s2 * y2): two sublayers' outputs, scaled per channel, into the stream
 //  gb_op_head_norm       per head: out = rmsnorm(x - lambda * x2) * gain * sigmoid(gate) * factor, each of x2,
 //                        gain and gate optional: the norm behind a recurrence or behind two attention maps; or of
-//                        x / (max(|den|, floor) + add) with two numbers per head: a read-out divided by its normaliser
+//                        x / (max(|den|, floor) + add) with two numbers per head: a read-out divided by its normaliser;
+//                        the gate's function is the sigmoid or silu
+//  gb_op_normed_sum      x (+)= f1 * rmsnorm(y1) * gain1 + f2 * rmsnorm(y2) * gain2: the outputs of mixers side by side,
+//                        each normed over the row before they are added
 #include "hybrid.cuh"
 
 namespace {
-
-enum { NORM_LAYER = 0, NORM_RMS = 1 };
 
 // Rows of up to NORM_CACHE * blockDim.x values are read once and kept in registers; longer rows are read
 // again from memory (an L2 hit) for every pass.
@@ -175,15 +176,6 @@ row_norm_warp_kernel(const float* x, long long ldx, const float* __restrict__ ga
     }
   }
 }
-
-// `then`: the norm in front of the NEXT sublayer, taken of the new rows while they are in registers
-// (out2 = norm2(x) * gain2), so that it needs no kernel and no second trip of its own.
-struct ThenNorm {
-  const float* gain;
-  void* out;
-  int out_dtype, kind;
-  float eps;
-};
 
 __global__ void norm_add_kernel(float* x, long long ldx, const float* y, long long ldy, const float* __restrict__ gain,
                                 int dim, int kind, float eps, bf16* copy, ThenNorm then) {
@@ -418,19 +410,6 @@ __global__ void gated_group_norm_kernel(const float* y, long long ldy, const flo
     o[d] = from_f32<TO>(yr[d] * hy_silu(zr[d]) * rstd * gain[c0 + d]);
 }
 
-enum { ACT_GELU_ERF = 0, ACT_GELU_TANH = 1, ACT_SILU = 2, ACT_RELU = 3, ACT_RELU2 = 4, ACT_NONE = 5 };
-
-__device__ __forceinline__ float act_value(float z, int kind) {
-  switch (kind) {
-    case ACT_GELU_ERF: return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f));
-    case ACT_GELU_TANH: return hy_gelu_tanh(z);
-    case ACT_SILU: return hy_silu(z);
-    case ACT_RELU: return fmaxf(z, 0.f);
-    case ACT_RELU2: z = fmaxf(z, 0.f); return z * z;
-    default: return z;
-  }
-}
-
 template <typename TO>
 __global__ void act_rows_kernel(const float* x, long long ld, TO* out, long long ldo, int n, int inner, int kind,
                                 int up) {
@@ -439,7 +418,7 @@ __global__ void act_rows_kernel(const float* x, long long ld, TO* out, long long
   const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= (long long)n * inner) return;
   const int t = (int)(i / inner), c = (int)(i - (long long)t * inner);
-  const float v = act_value(x[(size_t)t * ld + c], kind);
+  const float v = hy_act(x[(size_t)t * ld + c], kind);
   // (`up` > 0: a gated unit whose second factor lies `up` columns further in the row)
   out[(size_t)t * ldo + c] = from_f32<TO>(up > 0 ? v * x[(size_t)t * ld + up + c] : v);
 }
@@ -455,7 +434,7 @@ __global__ void act_rows4_kernel(const float* x, long long ld, TO* out, long lon
   if (i >= (long long)n * inner4) return;
   const int t = (int)(i / inner4), c = 4 * (int)(i - (long long)t * inner4);
   const float4 v = *reinterpret_cast<const float4*>(x + (size_t)t * ld + c);
-  float r0 = act_value(v.x, kind), r1 = act_value(v.y, kind), r2 = act_value(v.z, kind), r3 = act_value(v.w, kind);
+  float r0 = hy_act(v.x, kind), r1 = hy_act(v.y, kind), r2 = hy_act(v.z, kind), r3 = hy_act(v.w, kind);
   if (up > 0) {
     const float4 u = *reinterpret_cast<const float4*>(x + (size_t)t * ld + up + c);
     r0 *= u.x; r1 *= u.y; r2 *= u.z; r3 *= u.w;
@@ -479,7 +458,7 @@ template <typename TO>
 __global__ void head_norm_kernel(const float* x, long long ldx, long long xh, const float* x2,
                                  const float* __restrict__ gain, const float* gate, long long ld_gate, TO* out,
                                  long long ldo, int n, int H, int vdim, float eps, float lambda, float factor,
-                                 const float* den, const float* floor_, int gain_whole) {
+                                 const float* den, const float* floor_, int gain_whole, int gate_silu) {
   // (with `den`, lambda is what is added to the divisor)
   pdl_trigger();
   pdl_wait();
@@ -505,9 +484,92 @@ __global__ void head_norm_kernel(const float* x, long long ldx, long long xh, co
     if (d >= vdim) continue;
     float o = v[i] * rstd;
     if (gain) o *= gain[gain_whole ? h * vdim + d : d];
-    if (gate) o *= hy_sigmoid(gate[(size_t)t * ld_gate + (size_t)h * vdim + d]);
+    if (gate) {
+      const float z = gate[(size_t)t * ld_gate + (size_t)h * vdim + d];
+      o *= gate_silu ? hy_silu(z) : hy_sigmoid(z);
+    }
     out[(size_t)t * ldo + (size_t)h * vdim + d] = from_f32<TO>(o);
   }
+}
+
+// One block a row: x (+)= f1 * rms(y1) * g1 + f2 * rms(y2) * g2 (y2: optional), both rows in registers as NV pieces of
+// four values a thread (rows of 16-byte pieces); `then`: the norm in front of the next sublayer, of the new row.
+template <int NV>
+__global__ void __launch_bounds__(256)
+normed_sum_kernel(float* x, long long ldx, const float* y1, long long ld1, const float* __restrict__ g1, const float* y2,
+                  long long ld2, const float* __restrict__ g2, int dim, float eps, float f1, float f2, int accumulate,
+                  ThenNorm then) {
+  __shared__ float scratch[32];
+  pdl_trigger();
+  const size_t row = blockIdx.x;
+  float4 w1[NV], w2[NV];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int d = 4 * (threadIdx.x + i * blockDim.x);
+    w1[i] = d < dim ? *reinterpret_cast<const float4*>(g1 + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+    w2[i] = d < dim && y2 ? *reinterpret_cast<const float4*>(g2 + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+    gb_pin(w1[i]);
+    gb_pin(w2[i]);
+  }
+  pdl_wait();
+  float* o = x + row * ldx;
+  const float* a = y1 + row * ld1;
+  const float* b = y2 ? y2 + row * ld2 : nullptr;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 v[NV], ya[NV], yb[NV];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int d = 4 * (threadIdx.x + i * blockDim.x);
+    const bool in = d < dim;
+    ya[i] = in ? *reinterpret_cast<const float4*>(a + d) : zero;
+    yb[i] = in && b ? *reinterpret_cast<const float4*>(b + d) : zero;
+    v[i] = in && accumulate ? *reinterpret_cast<const float4*>(o + d) : zero;
+  }
+  float s1 = 0.f, s2 = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    s1 += (ya[i].x * ya[i].x + ya[i].y * ya[i].y) + (ya[i].z * ya[i].z + ya[i].w * ya[i].w);
+    s2 += (yb[i].x * yb[i].x + yb[i].y * yb[i].y) + (yb[i].z * yb[i].z + yb[i].w * yb[i].w);
+  }
+  const float r1 = f1 / sqrtf(block_sum(s1, scratch) / (float)dim + eps);
+  const float r2 = b ? f2 / sqrtf(block_sum(s2, scratch) / (float)dim + eps) : 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int d = 4 * (threadIdx.x + i * blockDim.x);
+    if (d >= dim) continue;
+    v[i].x += fmaf(yb[i].x * r2, w2[i].x, ya[i].x * r1 * w1[i].x);
+    v[i].y += fmaf(yb[i].y * r2, w2[i].y, ya[i].y * r1 * w1[i].y);
+    v[i].z += fmaf(yb[i].z * r2, w2[i].z, ya[i].z * r1 * w1[i].z);
+    v[i].w += fmaf(yb[i].w * r2, w2[i].w, ya[i].w * r1 * w1[i].w);
+    *reinterpret_cast<float4*>(o + d) = v[i];
+  }
+  if (then.gain != nullptr) hy_then_norm<NV>(v, dim, then, row, scratch);
+}
+
+// The same for rows of any length and alignment, read again for every pass.
+__global__ void normed_sum_any_kernel(float* x, long long ldx, const float* y1, long long ld1, const float* __restrict__ g1,
+                                      const float* y2, long long ld2, const float* __restrict__ g2, int dim, float eps,
+                                      float f1, float f2, int accumulate, ThenNorm then) {
+  __shared__ float scratch[32];
+  pdl_trigger();
+  pdl_wait();
+  const size_t row = blockIdx.x;
+  float* o = x + row * ldx;
+  const float* a = y1 + row * ld1;
+  const float* b = y2 ? y2 + row * ld2 : nullptr;
+  float s1 = 0.f, s2 = 0.f;
+  for (int d = threadIdx.x; d < dim; d += blockDim.x) {
+    s1 += a[d] * a[d];
+    if (b) s2 += b[d] * b[d];
+  }
+  const float r1 = f1 / sqrtf(block_sum(s1, scratch) / (float)dim + eps);
+  const float r2 = b ? f2 / sqrtf(block_sum(s2, scratch) / (float)dim + eps) : 0.f;
+  for (int d = threadIdx.x; d < dim; d += blockDim.x) {
+    float s = a[d] * r1 * g1[d];
+    if (b) s = fmaf(b[d] * r2, g2[d], s);
+    o[d] = accumulate ? o[d] + s : s;
+  }
+  if (then.gain != nullptr) hy_then_norm_row(o, dim, then, row, scratch);
 }
 
 inline int norm_threads(int dim) { return dim <= 256 ? 64 : dim <= 1024 ? 128 : 256; }
@@ -722,7 +784,8 @@ GB_OP(gb_op_act_rows) {
 // out as x) or 0, a4 gain [vdim] (shared by the heads) or 0, a5 gate logits (f32, [t, h * vdim + d] at a row stride)
 // or 0, a6 that stride, a7 out [rows, heads * vdim], a8 out dtype, a9 its row stride, a10 rows, a11 heads, a12 vdim,
 // a13 den [rows, heads] (f32) or 0: x is first divided by max(|den|, floor) + f1 (then no x2), a14 floor [rows, heads];
-// flags bit 0: the gain is [heads * vdim], not shared; f0 eps, f1 lambda, f2 factor
+// flags bit 0: the gain is [heads * vdim], not shared, bit 1: the gate's function is silu (else the sigmoid); f0 eps, f1
+// lambda, f2 factor
 GB_OP(gb_op_head_norm) {
   const int n = (int)a[10], H = (int)a[11], vdim = (int)a[12];
   if (n <= 0) return 0;
@@ -732,11 +795,35 @@ GB_OP(gb_op_head_norm) {
   if (a[8] == GB_BF16)
     gb_launch(head_norm_kernel<bf16>, grid, block, 0, ctx->stream, op_ptr<const float>(a[0]), a[1], a[2],
               op_ptr<const float>(a[3]), op_ptr<const float>(a[4]), op_ptr<const float>(a[5]), a[6], op_ptr<bf16>(a[7]), a[9],
-              n, H, vdim, (float)f[0], (float)f[1], (float)f[2], op_ptr<const float>(a[13]), op_ptr<const float>(a[14]), flags & 1);
+              n, H, vdim, (float)f[0], (float)f[1], (float)f[2], op_ptr<const float>(a[13]), op_ptr<const float>(a[14]), flags & 1, (flags >> 1) & 1);
   else
     gb_launch(head_norm_kernel<float>, grid, block, 0, ctx->stream, op_ptr<const float>(a[0]), a[1], a[2],
               op_ptr<const float>(a[3]), op_ptr<const float>(a[4]), op_ptr<const float>(a[5]), a[6], op_ptr<float>(a[7]), a[9],
-              n, H, vdim, (float)f[0], (float)f[1], (float)f[2], op_ptr<const float>(a[13]), op_ptr<const float>(a[14]), flags & 1);
+              n, H, vdim, (float)f[0], (float)f[1], (float)f[2], op_ptr<const float>(a[13]), op_ptr<const float>(a[14]), flags & 1, (flags >> 1) & 1);
   GB_CHECK_LAUNCH("head_norm");
+  return 1;
+}
+
+// a0 x (f32), a1 its row stride, a2 y1 (f32), a3 its row stride, a4 its gain [dim], a5 y2 (f32) or 0, a6 its row stride,
+// a7 its gain, a8 rows, a9 dim, a10 gain of a norm taken of the new rows or 0: none, a11 its output [rows, dim], a12 that
+// dtype, a13 its kind (0 layer norm, 1 RMS norm), a14 its eps (the bits of a 32-bit float); f0 eps of y1's and y2's norm,
+// f1 factor on the first, f2 on the second; flags bit 0: add into x (else it is overwritten)
+GB_OP(gb_op_normed_sum) {
+  const int n = (int)a[8], dim = (int)a[9];
+  if (n <= 0) return 0;
+  const ThenNorm then = hy_then_of(a[10], a[11], a[12], a[13], a[14]);
+  const bool vec = dim % 4 == 0 && dim <= 4096 && a[1] % 4 == 0 && a[3] % 4 == 0 && a[6] % 4 == 0 &&
+                   ((a[0] | a[2] | a[4] | a[5] | a[7]) & 15) == 0 && hy_then_vec(then);
+#define NORMED_SUM(KERNEL, THREADS)                                                                                     \
+  gb_launch(KERNEL, dim3(n), dim3(THREADS), 0, ctx->stream, op_ptr<float>(a[0]), a[1], op_ptr<const float>(a[2]), a[3],  \
+            op_ptr<const float>(a[4]), op_ptr<const float>(a[5]), a[6], op_ptr<const float>(a[7]), dim, (float)f[0],      \
+            (float)f[1], (float)f[2], flags & 1, then)
+  const int threads = hy_row_threads(dim);
+  if (!vec) NORMED_SUM(normed_sum_any_kernel, norm_threads(dim));
+  else if (dim <= 4 * threads) NORMED_SUM(normed_sum_kernel<1>, threads);
+  else if (dim <= 8 * threads) NORMED_SUM(normed_sum_kernel<2>, threads);
+  else NORMED_SUM(normed_sum_kernel<4>, threads);
+#undef NORMED_SUM
+  GB_CHECK_LAUNCH("normed_sum");
   return 1;
 }

@@ -267,7 +267,7 @@ DEFER_WHOLE_ROWS = 256
 
 
 # functions a product with a bfloat16 output can apply to its finished sums (the ``act`` of ``linear_tc``)
-EPILOGUES = {"relu2": 1}
+EPILOGUES = {"relu2": 1, "gelu": 2}
 
 
 def linear_tc(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor,

@@ -9,30 +9,89 @@ from .norm import RowNorm
 from .runner import Eager, Planned, stream_tensor
 
 
+FUSE_NEXT_NORM = True            # (the tests switch it off to compare the two ways)
+
+
 class PreNormResidual(Block):
     """x += mixer(norm(x)); x += ffn(norm(x))
-    (MisterTK/gibbs arch/families/lfm2.json5:76-89)."""
+    (MisterTK/gibbs arch/families/lfm2.json5:76-89).
+
+    A sublayer that says ``takes_then`` does the residual sum in a kernel that can also take the norm of the new rows: the
+    norm in front of the next sublayer, in this layer or (``hands_over``, which the model calls for neighbours in its order)
+    in the layer that runs next, then needs no kernel of its own when it is a ``RowNorm`` kind."""
     ROLES = (("mixer_norm", "norm"), ("mixer", "mixer"), ("ffn_norm", "norm"), ("ffn", "feed_forward"))
     OPTIONAL_ROLES = ("ffn_norm", "ffn")       # a layer may have no feed-forward (then neither its norm)
 
     # A mixer or feed-forward that says ``fuses_norm`` hands its input straight to a product
     # (``parts.linear.Linear``), which may then run the norm itself.
 
+    def __init__(self, parts, rt, params=None):
+        super().__init__(parts, rt, params)
+        self._next = None          # the block that runs next, when its norm is taken here
+        self._handed = None        # the normed rows the block in front left for this one
+
+    def hands_over(self, following) -> bool:
+        last = self.parts["ffn"] if "ffn" in self.parts else self.parts["mixer"]
+        if isinstance(following, PreNormResidual) and self._takes(last, following.mixer_norm):
+            self._next = following
+            return True
+        return False
+
+    @staticmethod
+    def _takes(part, norm) -> bool:
+        return FUSE_NEXT_NORM and bool(getattr(part, "takes_then", False)) and isinstance(norm, RowNorm)
+
+    def _behind(self, role: str):
+        """The norm that the kernel completing the sublayer in ``role`` takes, or None."""
+        if role == "mixer" and "ffn" in self.parts:
+            return self.ffn_norm if self._takes(self.mixer, self.ffn_norm) else None
+        return self._next.mixer_norm if self._next is not None else None
+
+    def _sublayers(self, run_norm, plain, summing):
+        """Both sublayers in order; ``run_norm(norm, consumer)``, ``plain(role, h)`` and ``summing(role, h, then)`` are the two
+        ways' own."""
+        h, self._handed = self._handed, None
+        for role in ("mixer", "ffn"):
+            if role not in self.parts:
+                break
+            part = self.parts[role]
+            if h is None:
+                h = run_norm(self.parts[role + "_norm"], part)
+            then = self._behind(role)
+            if then is None:
+                plain(role, h)
+                h = None
+            else:
+                h = summing(role, h, then)
+        if self._next is not None:
+            self._next._handed = h
+
     def forward(self, x, step, caches):
-        h = self.mixer_norm.lazy(x) if getattr(self.mixer, "fuses_norm", False) else self.mixer_norm.forward(x)
-        self.mixer.forward(h, x, step, self.caches_of("mixer", caches))
-        if "ffn" not in self.parts:
-            return
-        h = self.ffn_norm.lazy(x) if getattr(self.ffn, "fuses_norm", False) else self.ffn_norm.forward(x)
-        self.ffn.forward(h, x, step)
+        def run_norm(norm, part):
+            return norm.lazy(x) if getattr(part, "fuses_norm", False) else norm.forward(x)
+
+        def plain(role, h):
+            if role == "mixer":
+                self.mixer.forward(h, x, step, self.caches_of("mixer", caches))
+            else:
+                self.ffn.forward(h, x, step)
+
+        def summing(role, h, then):
+            return self.parts[role].run(Eager(self.rt, step), h, stream_tensor(x),
+                                        self.caches_of("mixer", caches) if role == "mixer" else None, accumulate=True, then=then)
+        self._sublayers(run_norm, plain, summing)
 
     def plan_ops(self, plan, caches):
-        h = self._norm_ops(plan, self.mixer_norm, self.mixer)
-        plan_ops_of(self.mixer)(plan, h, self.caches_of("mixer", caches))
-        if "ffn" not in self.parts:
-            return
-        h = self._norm_ops(plan, self.ffn_norm, self.ffn)
-        plan_ops_of(self.ffn)(plan, h)
+        def plain(role, h):
+            if role == "mixer":
+                plan_ops_of(self.mixer)(plan, h, self.caches_of("mixer", caches))
+            else:
+                plan_ops_of(self.ffn)(plan, h)
+
+        def summing(role, h, then):
+            return self.parts[role].run(Planned(plan), h, plan.residual,
+                                        self.caches_of("mixer", caches) if role == "mixer" else None, accumulate=True, then=then)
+        self._sublayers(lambda norm, part: self._norm_ops(plan, norm, part), plain, summing)
 
     @staticmethod
     def _norm_ops(plan, norm, consumer):
@@ -145,9 +204,6 @@ class ScaledSum(Part):
 
 
 register_part("branch_sum", "scaled_sum", ScaledSum)
-
-
-FUSE_NEXT_NORM = True            # (the tests switch it off to compare the two ways)
 
 
 class ParallelResidual(Block):

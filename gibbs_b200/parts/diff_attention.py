@@ -96,7 +96,7 @@ class DifferentialAttention(BranchPart, Mixer):
         lam = [float((tensors[a].double() * tensors[b].double()).sum()) for a, b in (("lq1", "lk1"), ("lq2", "lk2"))]
         self.lam = math.exp(lam[0]) - math.exp(lam[1]) + self.diff
         inv = stretched_inv_freq(self.rot_dims, float(p.get("rot_base", 10000.0)), p.get("rot_scaling"))
-        self.inv_freq = torch.cat([torch.from_numpy(inv), torch.zeros(1)]).to(torch.float32).to(rt.device)
+        self.inv_freq = torch.cat([torch.from_numpy(inv), torch.ones(1)]).to(torch.float32).to(rt.device)
 
     def kernel_libraries(self):
         return tuple(set(ops.linear_libraries(self.fused.dtype, self.rt.dtype)) | {"core", hybrid.LIBRARY})

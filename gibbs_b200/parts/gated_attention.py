@@ -24,6 +24,10 @@ j < n (at their true positions), and the pages of those positions stay;
 ``qk_norm`` "head": every head of q and k is normed over ``dim`` with a gain
 shared by the heads (before the rotation); ``q_temp`` {coef, every}: the query
 at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1);
+``mask`` ("blocks", n): position i sees the
+j <= i of its own block of n positions, blocks counted from position 0 of the sequence (pages of blocks a request has left go
+back); ``rot_yarn`` {factor, original, fast, slow}: the frequencies and a factor on cosines and sines of
+``parts.position.yarn_inv_freq``;
 ``weights`` "sigmoid": no softmax, p_j = sigmoid(s_j + pb_h) with a number per
 head (tensor ``pb``), not normalised over keys.  With ``shares_kv`` the layer has no key/value projections and reads the
 pages another entry of the model's order writes (keys as that entry stored
@@ -43,6 +47,7 @@ from .. import ops
 from ..ops import hybrid
 from .base import Mixer, PagedKV, Residual, TensorDecl, VECTOR, register_part
 from .linear import Linear
+from .position import yarn_inv_freq
 from .runner import BranchPart, Eager, Planned, Runner, keep
 
 
@@ -101,6 +106,10 @@ class GatedAttention(Mixer):
         self.softcap = float(p.get("softcap") or 0.0)
         self.window = int(p["window"]) if p.get("window") else None
         self.retain = p.get("retain", self.window)
+        mask = p.get("mask")
+        if mask and (self.window or p.get("shares_kv") or str(mask[0]) != "blocks" or int(mask[1]) < 1):
+            raise ValueError(f"mask {mask!r}: ('blocks', n) with n >= 1, for a layer with keys of its own and without a window")
+        self.block = int(mask[1]) if mask else None
         self.sink, self.gated = bool(p.get("sink", False)), bool(p.get("gate", True))
         self.sink_scores = tensors["sink"].to(torch.float32).contiguous() if p.get("sink") == "learned" else None
         self.keep_first = int(p.get("keep_first") or 0) if self.window else 0
@@ -143,17 +152,26 @@ class GatedAttention(Mixer):
         self.out_proj = Linear(self.out_weight, None, rt)
         i = np.arange(self.rot_dims // 2, dtype=np.float64)
         inv = np.power(float(p.get("rot_base", 10000.0)), -2.0 * i / max(self.rot_dims, 1)) / float(p.get("rot_factor") or 1.0)
-        self.inv_freq = torch.from_numpy(np.concatenate([inv, [0.0]]).astype(np.float32)).to(rt.device)
+        mscale = 1.0                               # (behind the frequencies: the factor on cosines and sines)
+        if p.get("rot_yarn") and self.rot_dims:
+            if p.get("rot_factor"):
+                raise ValueError("frequencies stretched in two ways")
+            inv, mscale = yarn_inv_freq(self.rot_dims, float(p.get("rot_base", 10000.0)),
+                                        *(float(p["rot_yarn"][k]) for k in ("factor", "original", "fast", "slow")))
+        self.inv_freq = torch.from_numpy(np.concatenate([inv, [mscale]]).astype(np.float32)).to(rt.device)
 
     def kernel_libraries(self):
         return tuple(set(ops.linear_libraries(self.fused.dtype, self.rt.dtype)) | {"core", hybrid.LIBRARY})
 
     def cache_needs(self):
         return [] if self.shares_kv else [PagedKV(self.kv_heads, self.dim, self.retain, self.vdim,
-                                                  keep_first=self.keep_first if self.retain else 0)]
+                                                  block=self.block, keep_first=self.keep_first if self.retain else 0)]
 
     def attention_flops(self, n_tokens: int) -> int:
         pairs = n_tokens * (n_tokens + 1) // 2
+        if self.block:
+            full, rest = divmod(n_tokens, self.block)
+            pairs = full * (self.block * (self.block + 1) // 2) + rest * (rest + 1) // 2
         if self.window and n_tokens > self.window:
             far = n_tokens - self.window                  # positions with keys in front of their window
             pairs -= far * (far + 1) // 2
@@ -201,19 +219,21 @@ class GatedAttention(Mixer):
         # (unnormalised weights: an operation of their own, whose last constant is the factor on the output)
         op, per_head, last = ("sigmoid_attention", self.score_bias, factor) if self.sigmoid else \
             ("sink_attention", self.sink_scores, self.keep_first)
+        span = self.block or self.window or 0
         ws = rn.buffer("ga_partial", vdim + 2, torch.float32, fixed_rows=_workspace_rows())
         gate = fused.data_ptr() + 4 * self.gate_col if self.gated else 0
         if tc:
             rn.op(op + "_tc", [q.data_ptr(), keep(rn, kp), keep(rn, vp), table, bt_stride, kv.page_size, kp.shape[0],
                                rn.tok_req, rn.tok_pos, gate, fused.stride(0), out.data_ptr(), out.stride(0), rn.N, H, G, dim,
-                               vdim, self.window or 0, rn.max_context, ws.data_ptr(), rn.R, rn.q_start, keep(rn, per_head)],
-                  [self.scale, self.softcap, last], label=op, flags=1 if self.sink else 0)
+                               vdim, span, rn.max_context, ws.data_ptr(), rn.R, rn.q_start, keep(rn, per_head)],
+                  [self.scale, self.softcap, last], label=op, flags=(1 if self.sink else 0) | (4 if self.block else 0))
             return out
         rn.op(op, [q.data_ptr(), keep(rn, kp), keep(rn, vp), table, bt_stride, kv.page_size, kp.shape[0], rn.tok_req,
-                   rn.tok_pos, gate, fused.stride(0), out.data_ptr(), out.stride(0), rn.N, H, G, dim, vdim, self.window or 0,
+                   rn.tok_pos, gate, fused.stride(0), out.data_ptr(), out.stride(0), rn.N, H, G, dim, vdim, span,
                    rn.max_context, ws.data_ptr(), 1, keep(rn, per_head)],
               [self.scale, self.softcap, last],
-              flags=(1 if self.sink else 0) | (4 if pages_bf16 else 0) | (8 if out.dtype == torch.bfloat16 else 0))
+              flags=(1 if self.sink else 0) | (4 if pages_bf16 else 0) | (8 if out.dtype == torch.bfloat16 else 0) |
+                    (16 if self.block else 0))
         return out
 
     def run(self, rn: Runner, h, out, caches, accumulate: bool = False):

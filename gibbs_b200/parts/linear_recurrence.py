@@ -16,10 +16,16 @@ input h (H heads, keys of ``dim`` channels, values of ``vdim`` entries):
     o = S^T q / (max(|n . q|, exp(-m_t)) + div_eps)
     out = W_o (rmsnorm(o_1 .. o_H, each head by itself) * gain * sigmoid(W_g h))                gain: all heads' size
 
+``gated_linear_attention`` (GLA; Yang et al.): one decay per head and key channel from a low-rank projection:
+
+    q = W_q h * dim^-1/2,  k = W_k h,  v = W_v h,  a = sigmoid(W_a2 (W_a1 h) + b)^(1 / tau)
+    S <- diag(a) S + k v^T,   o = S^T q
+    out = W_o [rmsnorm(o_h) * gain] * silu(W_g h)                             per head over ``vdim``; one gain vector
+
 S, n and m live in the request's slot, in 32-bit and zero for a new request.
 Everything behind the projections is 32-bit in every compute dtype.
 
-Both are made of an input product, the work between the products (``mix_heads``) and an output product, so that they can
+All are made of an input product, the work between the products (``mix_heads``) and an output product, so that they can
 also stand beside another mixer that reads the same input (``parts.parallel_mixers``).
 """
 from __future__ import annotations
@@ -147,5 +153,50 @@ class MatrixMemory(RecurrentHeads):
               [self.eps, self.div_eps, factor], label="rec_norm", flags=1)
 
 
+class GatedLinearAttention(RecurrentHeads):
+    @classmethod
+    def declare(cls, params):
+        d, H, dim, vdim, ra = (params[k] for k in ("hidden", "heads", "dim", "vdim", "decay_rank"))
+        return {"q": TensorDecl.of(H * dim, d), "k": TensorDecl.of(H * dim, d), "v": TensorDecl.of(H * vdim, d),
+                "g": TensorDecl.of(H * vdim, d), "a1": TensorDecl.of(ra, d), "a2": TensorDecl.of(H * dim, ra),
+                "a2.b": TensorDecl.of(H * dim, role=VECTOR), "norm": TensorDecl.of(vdim, role=VECTOR),
+                "o": TensorDecl.of(d, H * vdim)}
+
+    def __init__(self, params, tensors, rt):
+        super().__init__(params, tensors, rt)
+        self.hidden = int(params["hidden"])
+        self.H, self.dim, self.vdim = int(params["heads"]), int(params["dim"]), int(params["vdim"])
+        self.eps, self.tau = float(params["eps"]), float(params["tau"])
+        self.q_scale = float(params.get("q_scale", self.dim ** -0.5))
+        self.heads_width = self.H * self.vdim
+        self.fused = torch.cat([tensors[n] for n in ("q", "k", "v", "g", "a1")], 0).contiguous()
+        self.a2, self.out_weight = tensors["a2"].contiguous(), tensors["o"].contiguous()
+        f32 = lambda n: tensors[n].to(torch.float32).contiguous()
+        self.a_bias, self.gain = f32("a2.b"), f32("norm")
+
+    def cache_needs(self):
+        return [SlotState((self.H, self.vdim, self.dim), torch.float32)]
+
+    def mix_heads(self, rn, u, caches, out, factor=1.0):
+        rec = caches[0]
+        H, dim, vdim = self.H, self.dim, self.vdim
+        at = lambda col: u.data_ptr() + 4 * col
+        vc = 2 * H * dim
+        gc, ac = vc + H * vdim, vc + 2 * H * vdim
+        decay = padded(rn, "rec_decay", H * dim)
+        rn.op("low_rank_decays", [at(ac), u.stride(0), keep(rn, self.a2), ops.dtype_code(self.a2.dtype), keep(rn, self.a_bias),
+                                  decay.data_ptr(), decay.stride(0), rn.N, H * dim, self.a2.shape[1]], [self.tau])
+        y = rn.buffer("rec_read", H * vdim, torch.float32)
+        rn.op("linear_scan", [at(0), u.stride(0), at(H * dim), u.stride(0), at(vc), u.stride(0), decay.data_ptr(),
+                              decay.stride(0), 0, 0, keep(rn, rec.state), rec.state.stride(0), rn.slots(rec), rn.q_start,
+                              rn.q_len, y.data_ptr(), y.stride(0), 0, rn.R, H, dim, vdim, rn.N,
+                              segment_workspace(rn, "linear_scan", H, dim, vdim, 0).data_ptr()], [self.q_scale],
+              label="linear_scan:channel")
+        rn.op("head_norm", [y.data_ptr(), y.stride(0), vdim, 0, keep(rn, self.gain), at(gc), u.stride(0), out.data_ptr(),
+                            ops.dtype_code(out.dtype), out.stride(0), rn.N, H, vdim], [self.eps, 0.0, factor],
+              label="rec_norm", flags=2)
+
+
+register_part("mixer", "gated_linear_attention", GatedLinearAttention)
 register_part("mixer", "gated_write_recurrence", GatedWriteRecurrence)
 register_part("mixer", "matrix_memory", MatrixMemory)

@@ -11,6 +11,7 @@ design that keeps its norm weights around zero sets 1 and the rows are multiplie
 taken once, in 32-bit, when the part is built."""
 from __future__ import annotations
 
+import numpy as np
 import torch
 
 from .. import ops
@@ -61,6 +62,16 @@ class RMSNorm(Norm):
 
 
 register_part("norm", "rmsnorm", RMSNorm)
+
+
+def then_operands(rn: Runner, then):
+    """(five operands, output buffer or None) for a kernel that completes rows and takes a ``RowNorm`` of them (``then``; None:
+    it takes none): gain, output, its dtype, kind and the bits of the 32-bit eps."""
+    if then is None:
+        return [0, 0, 0, 0, 0], None
+    out = rn.buffer("normed", then.dim)
+    return [keep(rn, then.gain), out.data_ptr(), ops.dtype_code(out.dtype), then.KIND,
+            int(np.float32(then.eps).view(np.uint32))], out
 
 
 class RowNorm(Norm):

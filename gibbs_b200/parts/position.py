@@ -2,6 +2,8 @@
 kernel applies it to q and k together with the per-head norm."""
 from __future__ import annotations
 
+import math
+
 import numpy as np
 import torch
 
@@ -31,6 +33,21 @@ def stretched_inv_freq(rotary_dim: int, base: float, scaling=None) -> np.ndarray
         mid = (1.0 - s) * f / factor + s * f
         f = np.where(wl < orig / high, f, np.where(wl > orig / low, f / factor, mid))
     return f.astype(np.float32)
+
+
+def yarn_inv_freq(rotary_dim: int, base: float, factor: float, original: float, fast: float, slow: float):
+    """(frequencies, factor on cosines and sines) of a context stretched by ``factor`` the way YaRN (Peng et al.) does it:
+    pairs that turn more than ``fast`` times within ``original`` positions keep f_i = base^(-2i / rotary_dim), those that turn
+    less than ``slow`` times get f_i / factor, with a linear ramp over the pair's index in between.  64-bit, rounded once."""
+    i = np.arange(rotary_dim // 2, dtype=np.float64)
+    f = np.power(float(base), -2.0 * i / max(rotary_dim, 1))
+
+    def index_of(turns: float) -> float:          # the index whose pair turns this many times
+        return rotary_dim * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+
+    lo, hi = max(math.floor(index_of(fast)), 0), min(math.ceil(index_of(slow)), rotary_dim - 1)
+    ramp = np.clip((i - lo) / max(hi - lo, 0.001), 0.0, 1.0)
+    return (f / factor * ramp + f * (1.0 - ramp)).astype(np.float32), 0.1 * math.log(factor) + 1.0
 
 
 class RotaryHalfSplit(PositionEncoding):
