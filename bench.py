@@ -161,6 +161,30 @@ def guvetar_shape(size: str) -> dict:
             "layers": [{"type": k, "mixer": m, "mlp": mlp} for k, m in four * 2]}
 
 
+def nutopel_shape(size: str) -> dict:
+    """Layer sizes that resemble a real model's, for the Nutopel design: chunked attention beside a delta rule in turn with
+    gated linear attention; routed experts and a shared one behind each."""
+    if size == "1k":
+        d, vocab, chunk = 1024, 32768, 512
+        gla = {"heads": 8, "dim": 64, "vdim": 128, "tau": 16.0, "decay_rank": 16}
+        left = {"heads": 8, "kv_heads": 2, "dim": 64, "vdim": 64, "scale": 0.125}
+        right = {"heads": 8, "kv_heads": 4, "dim": 64, "vdim": 64, "conv": 4}
+        moe = {"kind": "moe", "router": {"experts": 16, "top": 2, "scale": 2.5, "groups": {"count": 4, "keep": 2}},
+               "expert": {"ff": 1024}, "shared": {"ff": 1024}}
+    else:
+        d, vocab, chunk = 2048, 65536, 1024
+        gla = {"heads": 8, "dim": 128, "vdim": 256, "tau": 16.0, "decay_rank": 16}
+        left = {"heads": 16, "kv_heads": 4, "dim": 64, "vdim": 64, "scale": 0.125}
+        right = {"heads": 8, "kv_heads": 4, "dim": 128, "vdim": 128, "conv": 4}
+        moe = {"kind": "moe", "router": {"experts": 32, "top": 4, "scale": 2.5, "groups": {"count": 8, "keep": 4}},
+               "expert": {"ff": 1024}, "shared": {"ff": 1024}}
+    left.update(mask={"size": chunk}, rot={"base": 500000.0, "dims": 64, "scaling": {"factor": 4.0, "original": 8192,
+                                                                                      "fast": 32.0, "slow": 1.0}})
+    both = {"left": left, "right": right}
+    return {"architecture": "Nutopel", "vocab": vocab, "width": d, "norm": {"eps": 1e-6}, "logit_scale": 1.0,
+            "layers": [{"type": k, "mixer": m, "mlp": moe} for k, m in [("parallel", both), ("gla", gla)] * 4]}
+
+
 def potivik_workload(a):
     """Prompt and decode throughput of the Potivik design at two sizes (random weights), beside an LFM2
     model of equal width, depth and feed-forward width, with the time per kind of operation of one
@@ -171,7 +195,9 @@ def potivik_workload(a):
     depth and feed-forward width.  'selivik': the Selivik design beside an LFM2 model, a Petelix model (windowed
     attention with a sink and routed experts) and a Potivik model (latent attention with a rotated part) of equal
     width and depth.  'guvetar': the Guvetar design beside an LFM2 model, a Sisadra model (a delta rule, attention on the
-    same tensor-core kernel, a dense feed-forward: the closest design) and a Potivik model (a state-space scan)."""
+    same tensor-core kernel, a dense feed-forward: the closest design) and a Potivik model (a state-space scan).  'nutopel':
+    the Nutopel design beside an LFM2 model, a Sisadra model (a delta rule, attention in blocks), a Guvetar model (the same
+    linear recurrence) and a Petelix model (routed experts) of equal width and depth."""
     import torch
     from gibbs_b200 import Engine, Lfm2Config, parse_config, random_model
     from gibbs_b200.engine import benchmark as B
@@ -190,8 +216,8 @@ def potivik_workload(a):
             twin = dict(LFM2_1P2B, hidden_size=d, num_hidden_layers=8, num_attention_heads=d // 64, num_key_value_heads=d // 256,
                         head_dim=64, vocab_size=pot["vocab"], intermediate_size=4 * d, block_auto_adjust_ff_dim=False,
                         full_attn_idxs=[1, 3, 5, 7], max_position_embeddings=4096)
-        elif a.workload in ("selivik", "guvetar"):
-            pot = selivik_shape(size) if a.workload == "selivik" else guvetar_shape(size)
+        elif a.workload in ("selivik", "guvetar", "nutopel"):
+            pot = {"selivik": selivik_shape, "guvetar": guvetar_shape, "nutopel": nutopel_shape}[a.workload](size)
             d = pot["width"]
             twin = dict(LFM2_1P2B, hidden_size=d, num_hidden_layers=8, num_attention_heads=d // 64, num_key_value_heads=d // 256,
                         head_dim=64, vocab_size=pot["vocab"], intermediate_size=4 * d, block_auto_adjust_ff_dim=False,
@@ -208,6 +234,10 @@ def potivik_workload(a):
         if a.workload == "guvetar":
             models.append(("Sisadra of equal size", parse_config(sisadra_shape(size))))
             models.append(("Potivik of equal size", parse_config(potivik_shape(size))))
+        if a.workload == "nutopel":
+            models.append(("Sisadra of equal size", parse_config(sisadra_shape(size))))
+            models.append(("Guvetar of equal size", parse_config(guvetar_shape(size))))
+            models.append(("Petelix of equal size", parse_config(petelix_shape(size))))
         if a.workload == "selivik":
             models.append(("Petelix of equal size", parse_config(petelix_shape(size))))
             models.append(("Potivik of equal size", parse_config(potivik_shape(size))))
@@ -302,10 +332,11 @@ def main():
                     help="float32: the engine's true 32-bit twin on the same (bfloat16-rounded) weights; "
                          "with --only prefill or --only decode (the benchmark line itself is bfloat16)")
     ap.add_argument("--skip-points", action="store_true", help="skip batch 1 and 64")
-    ap.add_argument("--workload", choices=["serve700m", "long2p6b", "sweep", "potivik", "petelix", "sisadra", "selivik", "guvetar"], default=None,
+    ap.add_argument("--workload", choices=["serve700m", "long2p6b", "sweep", "potivik", "petelix", "sisadra", "selivik", "guvetar", "nutopel"],
+                    default=None,
                     help="run one of the other workloads instead (prints its own JSON lines); 'potivik' / 'petelix' / "
-                         "'sisadra' / 'selivik' / 'guvetar': that design at layer sizes of a real model, beside an LFM2 model of equal size")
-    ap.add_argument("--size", default=None, help="with --workload potivik, petelix, sisadra, selivik or guvetar: '1k', '2k' or both with a comma (default both)")
+                         "'sisadra' / 'selivik' / 'guvetar' / 'nutopel': that design at layer sizes of a real model, beside an LFM2 model of equal size")
+    ap.add_argument("--size", default=None, help="with --workload potivik, petelix, sisadra, selivik, guvetar or nutopel: '1k', '2k' or both with a comma (default both)")
     ap.add_argument("--no-twins", action="store_true", help="with such a workload: the design alone, without the models beside it")
     ap.add_argument("--prompt-tokens", type=int, default=None,
                     help="with --only prefill / prefill-timeline / products: another prompt length than 2,048")
@@ -329,7 +360,7 @@ def main():
     from gibbs_b200 import Generator, Lfm2Config, random_model
     from gibbs_b200.engine import benchmark as B
 
-    if a.workload in ("potivik", "petelix", "sisadra", "selivik", "guvetar"):
+    if a.workload in ("potivik", "petelix", "sisadra", "selivik", "guvetar", "nutopel"):
         return potivik_workload(a)
     if a.workload:
         return other_workload(a)

@@ -33,7 +33,7 @@ LIBRARIES = {
     # streams, routed experts: every entry
     # point has the signature of a step-plan operation (hybrid.cuh)
     "hybrid": ["errors.cu", "norms.cu", "latent_attention.cu", "latent_attention_tc.cu", "gated_attention.cu", "gated_attention_tc.cu",
-               "sigmoid_attention_tc.cu", "ssm.cu", "selective_scan.cu", "delta_rule.cu", "linear_scan.cu", "streams.cu", "moe.cu",
+               "sigmoid_attention_tc.cu", "ssm.cu", "selective_scan.cu", "delta_rule.cu", "delta_chunks.cu", "linear_scan.cu", "streams.cu", "moe.cu",
                "moe_tc.cu"],
 }
 

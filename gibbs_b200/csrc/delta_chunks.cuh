@@ -1,0 +1,31 @@
+// The chunked form of the delta rule's recurrence (delta_chunks.cu), launched by gb_op_delta_scan.
+#pragma once
+#include "hybrid.cuh"
+
+constexpr int DELTA_CHUNK = 32;
+constexpr int DELTA_CHUNK_MAX_DIM = 128;
+
+struct DeltaChunkParams {
+  const float* qk; long long ld_qk;        // rows [q | k | v]: q and k normed per key head
+  int k_col, v_col;
+  const float* decay;                      // [t, heads]
+  const float* beta;                       // [t, heads]
+  float* state; long long slot_stride;     // slot 0: [heads][dim][vdim]
+  const int* slot_ids; const int* q_start; const int* q_len;
+  float* out; long long ldo;               // [t, heads * vdim]
+  int R, H, G, dim, vdim;
+  // workspace, set by gb_delta_chunks
+  float* w;                                // [t, heads, dim]
+  float* u0;                               // [t, heads, vdim]
+  float* read;                             // [t, heads, DELTA_CHUNK]
+  float* gains;                            // [t, heads, 2]: product of the chunk's decays up to t, and behind it
+};
+
+// Floats of workspace per token.
+static inline long long gb_delta_chunks_floats(int heads, int dim, int vdim) {
+  return (long long)heads * (dim + vdim + DELTA_CHUNK + 2);
+}
+
+// Rows of 16-byte pieces (dim, vdim and every column and stride a multiple of four), dim at most DELTA_CHUNK_MAX_DIM; n tokens.
+// Returns the number of launches or an error.
+int gb_delta_chunks(DeltaChunkParams p, float* ws, int n, cudaStream_t stream);

@@ -18,7 +18,7 @@
 //                     their shares of the two products with S by shuffles
 //
 // State layout in a slot: [heads][dim][vdim].
-#include "hybrid.cuh"
+#include "delta_chunks.cuh"
 
 namespace {
 
@@ -51,6 +51,7 @@ __global__ void delta_prep_kernel(float* qk, long long ld_qk, int k_col, const f
   for (int h = threadIdx.x; h < H; h += blockDim.x) beta[(size_t)t * H + h] = hy_sigmoid(b[(size_t)t * ld_b + h]);
 }
 
+constexpr int DS_CHUNKED_FROM = 48; // tokens of a portion from which on chunks pay (one decay a head)
 constexpr int DS_TOKENS = 16;       // tokens whose q, k and decay are staged in shared memory at a time
 
 // Block: (request, head, DS_COLS columns of S).  Thread j owns column c0 + j: S[i][c], i < dim, in registers
@@ -329,8 +330,10 @@ GB_OP(gb_op_delta_prep) {
 // a4 decays [tokens, heads * dim] (f32), a5 their row stride, a6 beta [tokens, heads] (f32), a7 recurrent state of
 // slot 0 ([heads][dim][vdim], f32), a8 elements between slots, a9 slot ids, a10 first row per request, a11 rows per
 // request, a12 out [tokens, heads * vdim] (f32), a13 its row stride, a14 requests, a15 heads, a16 kv heads, a17 dim,
-// a18 vdim; flags bit 0: the kernel with one thread a column, whatever the sizes, bit 1: one decay a head (a4 [tokens,
-// heads])
+// a18 vdim, a19 longest portion of the step (0: not known), a20 workspace of gb_delta_chunks_floats(heads, dim, vdim) floats a
+// token (16-byte aligned) or 0, a21 tokens; flags bit 0: the kernel with one thread a column, whatever the sizes, bit 1: one
+// decay a head (a4 [tokens, heads]): with a workspace and a portion of DS_CHUNKED_FROM tokens or more the recurrence then takes
+// chunks of tokens at a time (delta_chunks.cu)
 GB_OP(gb_op_delta_scan) {
   const int R = (int)a[14], H = (int)a[15], G = (int)a[16], dim = (int)a[17], vdim = (int)a[18];
   if (R <= 0) return 0;
@@ -340,6 +343,17 @@ GB_OP(gb_op_delta_scan) {
   // rows that can be copied in 16-byte pieces: a column of S over several lanes, inputs staged ahead
   if (!(flags & 1) && dim % 4 == 0 && vdim % 4 == 0 && a[1] % 4 == 0 && a[2] % 4 == 0 && a[3] % 4 == 0 &&
       (a[0] & 15) == 0 && (head || (a[5] % 4 == 0 && (a[4] & 15) == 0))) {
+    if (head && a[20] && (a[20] & 15) == 0 && a[19] >= DS_CHUNKED_FROM && dim <= DELTA_CHUNK_MAX_DIM && a[13] % 2 == 0 &&
+        (a[12] & 7) == 0 && a[5] == H) {
+      DeltaChunkParams p;
+      p.qk = op_ptr<const float>(a[0]); p.ld_qk = a[1]; p.k_col = (int)a[2]; p.v_col = (int)a[3];
+      p.decay = op_ptr<const float>(a[4]); p.beta = op_ptr<const float>(a[6]);
+      p.state = op_ptr<float>(a[7]); p.slot_stride = a[8];
+      p.slot_ids = op_ptr<const int>(a[9]); p.q_start = op_ptr<const int>(a[10]); p.q_len = op_ptr<const int>(a[11]);
+      p.out = op_ptr<float>(a[12]); p.ldo = a[13];
+      p.R = R; p.H = H; p.G = G; p.dim = dim; p.vdim = vdim;
+      return gb_delta_chunks(p, op_ptr<float>(a[20]), (int)a[21], ctx->stream);
+    }
 #define COLS_SCAN(SPLIT, PER, TOK)                                                                                      \
     do { if (head) COLS_SCAN_OF(SPLIT, PER, TOK, true); else COLS_SCAN_OF(SPLIT, PER, TOK, false); } while (0)
 #define COLS_SCAN_OF(SPLIT, PER, TOK, HEAD)                                                                             \
@@ -375,4 +389,10 @@ GB_OP(gb_op_delta_scan) {
 #undef SCAN_OF
   GB_CHECK_LAUNCH("delta_scan");
   return 1;
+}
+
+// Floats of workspace per token for the chunked form (0: these sizes have none).
+GB_API long long gb_delta_scan_workspace(int heads, int dim, int vdim) {
+  if (dim % 4 || vdim % 4 || dim > DELTA_CHUNK_MAX_DIM) return 0;
+  return gb_delta_chunks_floats(heads, dim, vdim);
 }

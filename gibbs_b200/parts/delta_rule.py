@@ -24,6 +24,8 @@ ranks of the two low-rank projections are read from their tensors' shapes.
 """
 from __future__ import annotations
 
+import ctypes
+
 import torch
 
 from .. import ops
@@ -31,7 +33,16 @@ from ..ops import hybrid
 from .base import Mixer, SlotState, TensorDecl, VECTOR, register_part
 from .runner import BranchPart, Runner, keep
 
-SPLIT_COLUMNS = True             # (the tests switch it off to compare the recurrence's two kernels)
+SPLIT_COLUMNS = True             # (the tests switch them off to compare the recurrence's kernels)
+CHUNKS = True
+
+
+def _chunk_floats(heads: int, dim: int, vdim: int) -> int:
+    """Floats of workspace per token for the recurrence in chunks of tokens; 0: these sizes have no such form."""
+    from ..ops.library import library
+    fn = library(hybrid.LIBRARY).gb_delta_scan_workspace
+    fn.restype = ctypes.c_longlong
+    return int(fn(heads, dim, vdim))
 
 
 class GatedDeltaRule(BranchPart, Mixer):
@@ -124,9 +135,12 @@ class GatedDeltaRule(BranchPart, Mixer):
                              keep(rn, self.dt_bias), keep(rn, self.a_log), beta.data_ptr(), rn.N, H, G, dim,
                              decay.data_ptr() if self.head_decay else 0], [self.unit_eps, self.q_scale])
         y = rn.buffer("dr_out", H * vdim, torch.float32)
+        # one decay a head: long portions in chunks of tokens (csrc/delta_chunks.cu)
+        floats = _chunk_floats(H, dim, vdim) if self.head_decay and CHUNKS and SPLIT_COLUMNS else 0
+        ws = rn.buffer("dr_chunks", floats, torch.float32).data_ptr() if floats else 0
         rn.op("delta_scan", [qkv.data_ptr(), qkv.stride(0), G * dim, 2 * G * dim, decay.data_ptr(), decay.stride(0),
                              beta.data_ptr(), keep(rn, rec.state), rec.state.stride(0), slots, rn.q_start, rn.q_len,
-                             y.data_ptr(), y.stride(0), rn.R, H, G, dim, vdim],
+                             y.data_ptr(), y.stride(0), rn.R, H, G, dim, vdim, rn.max_portion, ws, rn.N],
               flags=(0 if SPLIT_COLUMNS else 1) | (2 if self.head_decay else 0))
         rn.op("head_norm", [y.data_ptr(), y.stride(0), vdim, 0, keep(rn, self.gain), gate, ld_gate, out.data_ptr(),
                             ops.dtype_code(out.dtype), out.stride(0), rn.N, H, vdim], [self.eps, 0.0, factor],

@@ -22,6 +22,7 @@ class Runner:
     # rows in the step, requests, wanted rows; addresses of the step's metadata
     N = R = W = 0
     max_context = 0      # the longest context of the step after it (inside a CUDA graph: an upper bound)
+    max_portion = 0      # the longest portion of the step
     token_ids = tok_req = tok_pos = q_start = q_len = start_pos = want_rows = 0
 
     def buffer(self, name: str, width: int, dtype=None, per_token: int = 1, fixed_rows: Optional[int] = None):
@@ -73,6 +74,7 @@ class Eager(Runner):
         self.rt, self.step = rt, step
         self.N, self.R, self.W = step.n_tokens, step.n_requests, step.n_want
         self.max_context = max(int(step.max_ctx_len), 1)
+        self.max_portion = int(getattr(step, "max_q_len", 0))
         for k in ("token_ids", "tok_req", "tok_pos", "q_start", "q_len", "start_pos", "want_rows"):
             setattr(self, k, getattr(step, k).data_ptr())
 
@@ -111,7 +113,7 @@ class Planned(Runner):
         self.token_ids, self.tok_req, self.tok_pos = P.sym(P.S_TOKEN_IDS), P.sym(P.S_TOK_REQ), P.sym(P.S_TOK_POS)
         self.q_start, self.q_len, self.start_pos = P.sym(P.S_Q_START), P.sym(P.S_Q_LEN), P.sym(P.S_START_POS)
         self.want_rows = P.sym(P.S_WANT_ROWS)
-        self.max_context = P.sym(P.S_MAXCTX)
+        self.max_context, self.max_portion = P.sym(P.S_MAXCTX), P.sym(P.S_MAXQ)
         self._P = P
 
     def buffer(self, name, width, dtype=None, per_token=1, fixed_rows=None):

@@ -274,3 +274,34 @@ def test_trace_run_guvetar_with_and_without_dependent_launch(tmp_path):
     for rid in results["serial"]:
         for p in results["serial"][rid]:
             assert np.array_equal(results["serial"][rid][p], results["overlapped"][rid][p]), (rid, p)
+
+
+def test_trace_run_nutopel_with_and_without_dependent_launch(tmp_path):
+    """The Nutopel design through the same runner: a model folder on disk (bfloat16 weights; the rank of a decay
+    projection stands in its tensor's shape only), both compute dtypes, mixed steps with sparse wants in a pool that makes pages and the four state slots go
+    round; in float32 the runs with and without programmatic dependent launch agree to the bit."""
+    import plain_nutopel
+    from nutopel_helpers import CFG_A, make_weights, without_ranks
+    from potivik_helpers import rel_rows, write_model
+    W = make_weights(CFG_A, 23, steady=True)
+    folder = write_model(tmp_path / "nutopel_a", without_ranks(CFG_A), W)
+    vocab = CFG_A["vocab"]
+    reqs = {f"q{i}": random_ids(90 + i, n, vocab) for i, n in enumerate([70, 45, 130, 1, 64, 20, 33])}
+    steps = trace_mixed(reqs, capacity_tokens=320, max_live=4, seed=6)
+    for k, s in enumerate(steps):
+        for e in s["entries"]:
+            e["want"] = [] if k % 5 == 4 else [w for w in e["want"] if (w + k) % 3]
+    want = {rid: plain_nutopel.forward(CFG_A, W, ids).numpy() for rid, ids in reqs.items()}
+    results = {}
+    for mode, dtype, tol, pdl in (("serial", "float32", 2e-4, "0"), ("overlapped", "float32", 2e-4, "1"), ("bf16", "bfloat16", 8e-2, "1")):
+        out = tmp_path / f"out_{mode}"
+        _run(folder, dtype, steps, out, max_tokens=320, env={"GIBBS_B200_PDL": pdl})
+        got = results[mode] = _collect(steps, out, vocab)
+        for rid in reqs:
+            rows = sorted(got.get(rid, {}))
+            if rows:
+                e = rel_rows(np.stack([got[rid][p] for p in rows]), want[rid][rows])
+                assert np.median(e) <= tol / 2 and e.max() <= tol, f"{mode}, {rid}: place {rows[int(e.argmax())]} differs by {e.max():.3g}"
+    for rid in results["serial"]:
+        for p in results["serial"][rid]:
+            assert np.array_equal(results["serial"][rid][p], results["overlapped"][rid][p]), (rid, p)
