@@ -51,7 +51,7 @@ __global__ void delta_prep_kernel(float* qk, long long ld_qk, int k_col, const f
   for (int h = threadIdx.x; h < H; h += blockDim.x) beta[(size_t)t * H + h] = hy_sigmoid(b[(size_t)t * ld_b + h]);
 }
 
-constexpr int DS_CHUNKED_FROM = 48; // tokens of a portion from which on chunks pay (one decay a head)
+constexpr int DS_CHUNKED_FROM = 160;// tokens of a portion from which on chunks pay (one decay a head)
 constexpr int DS_TOKENS = 16;       // tokens whose q, k and decay are staged in shared memory at a time
 
 // Block: (request, head, DS_COLS columns of S).  Thread j owns column c0 + j: S[i][c], i < dim, in registers
@@ -330,8 +330,8 @@ GB_OP(gb_op_delta_prep) {
 // a4 decays [tokens, heads * dim] (f32), a5 their row stride, a6 beta [tokens, heads] (f32), a7 recurrent state of
 // slot 0 ([heads][dim][vdim], f32), a8 elements between slots, a9 slot ids, a10 first row per request, a11 rows per
 // request, a12 out [tokens, heads * vdim] (f32), a13 its row stride, a14 requests, a15 heads, a16 kv heads, a17 dim,
-// a18 vdim, a19 longest portion of the step (0: not known), a20 workspace of gb_delta_chunks_floats(heads, dim, vdim) floats a
-// token (16-byte aligned) or 0, a21 tokens; flags bit 0: the kernel with one thread a column, whatever the sizes, bit 1: one
+// a18 vdim, a19 longest portion of the step (0: not known), a20 workspace of gb_delta_scan_workspace(...) floats
+// (16-byte aligned) or 0, a21 tokens; flags bit 0: the kernel with one thread a column, whatever the sizes, bit 1: one
 // decay a head (a4 [tokens, heads]): with a workspace and a portion of DS_CHUNKED_FROM tokens or more the recurrence then takes
 // chunks of tokens at a time (delta_chunks.cu)
 GB_OP(gb_op_delta_scan) {
@@ -391,8 +391,8 @@ GB_OP(gb_op_delta_scan) {
   return 1;
 }
 
-// Floats of workspace per token for the chunked form (0: these sizes have none).
-GB_API long long gb_delta_scan_workspace(int heads, int dim, int vdim) {
+// Floats of workspace the chunked form takes for steps of up to n tokens in up to R portions (0: these sizes have none).
+GB_API long long gb_delta_scan_workspace(int n, int R, int heads, int dim, int vdim) {
   if (dim % 4 || vdim % 4 || dim > DELTA_CHUNK_MAX_DIM) return 0;
-  return gb_delta_chunks_floats(heads, dim, vdim);
+  return gb_delta_chunks_floats(n, R, heads, dim, vdim);
 }

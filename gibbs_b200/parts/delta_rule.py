@@ -37,12 +37,13 @@ SPLIT_COLUMNS = True             # (the tests switch them off to compare the rec
 CHUNKS = True
 
 
-def _chunk_floats(heads: int, dim: int, vdim: int) -> int:
-    """Floats of workspace per token for the recurrence in chunks of tokens; 0: these sizes have no such form."""
+def _chunk_floats(tokens: int, requests: int, heads: int, dim: int, vdim: int) -> int:
+    """Floats of workspace for the recurrence in chunks of tokens, for steps of up to this size; 0: these heads have no such
+    form."""
     from ..ops.library import library
     fn = library(hybrid.LIBRARY).gb_delta_scan_workspace
     fn.restype = ctypes.c_longlong
-    return int(fn(heads, dim, vdim))
+    return int(fn(tokens, requests, heads, dim, vdim))
 
 
 class GatedDeltaRule(BranchPart, Mixer):
@@ -136,8 +137,8 @@ class GatedDeltaRule(BranchPart, Mixer):
                              decay.data_ptr() if self.head_decay else 0], [self.unit_eps, self.q_scale])
         y = rn.buffer("dr_out", H * vdim, torch.float32)
         # one decay a head: long portions in chunks of tokens (csrc/delta_chunks.cu)
-        floats = _chunk_floats(H, dim, vdim) if self.head_decay and CHUNKS and SPLIT_COLUMNS else 0
-        ws = rn.buffer("dr_chunks", floats, torch.float32).data_ptr() if floats else 0
+        floats = _chunk_floats(*rn.largest_step(), H, dim, vdim) if self.head_decay and CHUNKS and SPLIT_COLUMNS else 0
+        ws = rn.buffer("dr_chunks", floats, torch.float32, fixed_rows=1).data_ptr() if floats else 0
         rn.op("delta_scan", [qkv.data_ptr(), qkv.stride(0), G * dim, 2 * G * dim, decay.data_ptr(), decay.stride(0),
                              beta.data_ptr(), keep(rn, rec.state), rec.state.stride(0), slots, rn.q_start, rn.q_len,
                              y.data_ptr(), y.stride(0), rn.R, H, G, dim, vdim, rn.max_portion, ws, rn.N],

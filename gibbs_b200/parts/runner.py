@@ -30,6 +30,10 @@ class Runner:
         or ``fixed_rows`` rows whatever the step."""
         raise NotImplementedError
 
+    def largest_step(self) -> tuple:
+        """(tokens, requests) of the largest step this runner's buffers have to serve."""
+        raise NotImplementedError
+
     def linear(self, x, weight, bias, out, role: str = "") -> None:
         """out = x weight^T (+ bias); the kernel is chosen by the operand types.  ``role`` names
         the product in the timing table."""
@@ -82,6 +86,9 @@ class Eager(Runner):
         rows = fixed_rows if fixed_rows is not None else self.N * per_token
         return torch.empty(rows, int(width), dtype=dtype or self.rt.dtype, device=self.rt.device)
 
+    def largest_step(self):
+        return self.N, self.R
+
     def linear(self, x, weight, bias, out, role=""):
         ops.linear(x[:self.N] if x.shape[0] != self.N else x, weight, bias, out)
 
@@ -119,6 +126,9 @@ class Planned(Runner):
     def buffer(self, name, width, dtype=None, per_token=1, fixed_rows=None):
         rows = fixed_rows if fixed_rows is not None else self.plan.cap * per_token
         return self.plan.buffer(f"{name}[{rows}]", width, dtype, rows=rows)
+
+    def largest_step(self):
+        return self.plan.cap, self.plan.max_requests
 
     def linear(self, x, weight, bias, out, role=""):
         self.plan.linear(x, weight, bias, out, "plain", role=role or "plain")

@@ -57,8 +57,6 @@ def check_rows(got, want, dtype: str, what: str = "", tol=None, noise=()):
     cancel is +1 or -1 behind its norm."""
     e = rel_rows(got, want) if dtype == "float32" else row_errors(got, want)
     tol = np.full(e.shape, TOL[dtype] if tol is None else tol)
-    if dtype == "float32" and len(noise):                      # (where 16-bit rounding moves a row a lot, 32-bit rounding moves it too)
-        tol = np.maximum(tol, 1e-3 * np.max([rel_rows(n, want) for n in noise], axis=0))
     if dtype == "bfloat16" and len(noise):
         tol = np.maximum(tol, 4.0 * np.max([row_errors(n, want) for n in noise], axis=0))
         over = np.sort(e / tol)[::-1]
@@ -285,8 +283,8 @@ def run_delta(q, k, v, g, beta, cuts, chunks: bool, state=None):
     g, beta = g.to(DEV).contiguous(), beta.to(DEV).contiguous()
     S = torch.zeros(1, H, dim, vdim, device=DEV) if state is None else state.to(DEV).clone()
     out = torch.full((T, H * vdim), float("nan"), device=DEV)
-    floats = _chunk_floats(H, dim, vdim)
-    ws = torch.full((T * max(floats, 1),), float("nan"), device=DEV)
+    floats = _chunk_floats(T, 1, H, dim, vdim)
+    ws = torch.full((max(floats, 1),), float("nan"), device=DEV)
     at, c = 0, 0
     while at < T:
         n = min(cuts[min(c, len(cuts) - 1)], T - at)
@@ -297,7 +295,7 @@ def run_delta(q, k, v, g, beta, cuts, chunks: bool, state=None):
                                               o.data_ptr(), H * vdim, 1, H, G, dim, vdim, n, ws.data_ptr() if chunks and floats else 0, n],
                                flags=2)
         torch.cuda.synchronize()
-        assert launches == (2 if chunks and floats and n >= 48 else 1)
+        assert launches == (3 if chunks and floats and n >= 160 else 1)
         at, c = at + n, c + 1
     return out.cpu().reshape(T, H, vdim), S.cpu()
 
@@ -314,7 +312,7 @@ def test_chunks_of_tokens_against_one_token_after_the_other(H, G, dim, vdim, kin
     """Decays near one, decays that forget everything at once (zero among them), keys that are all alike with write strengths
     near one (the triangular system at its stiffest), keys that alternate in sign; cut at and off the chunks' edges."""
     g_ = gen(dim + vdim)
-    T = 261
+    T = 421
     q, k, v = torch.randn(T, G, dim, generator=g_), torch.randn(T, G, dim, generator=g_), torch.randn(T, H, vdim, generator=g_)
     beta = torch.rand(T, H, generator=g_)
     g = torch.exp(-torch.rand(T, H, generator=g_))
@@ -331,7 +329,7 @@ def test_chunks_of_tokens_against_one_token_after_the_other(H, G, dim, vdim, kin
     want = plain_delta(q, k, v, g, beta).reshape(T, -1)
     steps, state = run_delta(q, k, v, g, beta, [T], False)
     scale = float(want.norm(dim=-1).median())
-    for cuts in ([T], [32, 64, 96, 1], [70, 1, 1, 50, 2, 90, 47], [33, 63, 65, 100]):
+    for cuts in ([T], [192, 160, 1], [1, 2, 161, 40, 217], [223]):
         got, S = run_delta(q, k, v, g, beta, cuts, True)
         assert float((got.reshape(T, -1).double() - want).norm(dim=-1).max()) < 2e-5 * scale, cuts
         assert float((S - state).norm()) < 2e-5 * float(state.norm()) + 1e-30
@@ -744,7 +742,13 @@ def test_random_configurations(seed):
             eng = engine_for(model, n_pages=16, max_requests=3, cap=256)
             got = run_trace_on_engine(eng, steps)
             for rid in reqs:
-                check_model(got[rid], truth[rid], dtype, True, f"{what} {rid}", tol=3e-4 if dtype == "float32" else 5e-2)
+                if dtype == "float32":
+                    # (a head of one value whose terms cancel is blown up by its norm, by up to 1 / sqrt(eps): one row in thirty,
+                    # or one, may be such a row)
+                    e = np.sort(rel_rows(got[rid], truth[rid][0]))[::-1]
+                    assert e[max(1, e.size // 30):].max(initial=0.0) <= 3e-4 and e[0] <= 5e-3, f"{what} {rid}: {e[:4]}"
+                else:
+                    check_model(got[rid], truth[rid], dtype, True, f"{what} {rid}", tol=5e-2)
 
 
 def test_pages_of_chunks_a_request_has_left_go_back():
