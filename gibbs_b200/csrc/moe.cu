@@ -9,6 +9,7 @@
 //  gb_op_moe_sort      (token, choice) pairs ordered by expert: offsets[E + 1], the pair behind every
 //                      row, the row of every pair
 //  gb_op_moe_gather    rows[row] = weight * h[token]: the weight multiplies the expert's INPUT
+//  gb_op_moe_dispatch  the grouped choice, the order and the gathered rows together (one kernel for a step of few tokens)
 //  gb_op_moe_experts   per expert, over its rows: act = glu(rows W_gate^T, rows W_up^T) with clamps, or act =
 //                      function(rows W_up^T) for experts without a gate, or out = rows W_down^T (32-bit)
 //  gb_op_moe_combine   y[token] = sum over its choices of out[row] (+ gate * shared[token])
@@ -57,62 +58,69 @@ __global__ void moe_route_kernel(const float* logits, long long ld, int n, int E
   if (shared_gate && lane == 0) shared_gate[t] = hy_sigmoid(z[shared_col]);
 }
 
-// One warp per token.  scores: 0 sigmoid(z), 1 softmax(z) over all `n_out` router outputs, 2 the logits z themselves.
+// A router's rule.  scores: 0 sigmoid(z), 1 softmax(z) over all `n_out` router outputs, 2 the logits z themselves.
 // `normalise`: 0 a chosen output's weight is its score, 1 the score divided by the sum of the chosen scores, 2 the
 // softmax over the chosen scores alone.  The choice is made on
 // score + correction; with `groups` > 1 the outputs form that many equal groups of neighbours, a group's mark is
 // its largest choice score (or, with `mark_two`, the sum of its two largest), and only outputs of the `keep` best groups
 // can be chosen.  The weight of a chosen output is its score without the correction, not renormalised, times
 // `weight_scale`.  Ties go to the lower index.
-__global__ void moe_route_grouped_kernel(const float* logits, long long ld, int n, int n_out, int top, int scores,
-                                         const float* __restrict__ correction, int groups, int keep, int* idx,
-                                         float* weight, int normalise, int mark_two, float weight_scale) {
-  extern __shared__ float route_sm[];                    // per warp: scores [n_out], choice scores [n_out], group marks
-  pdl_trigger();
-  pdl_wait();
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int t = blockIdx.x * (blockDim.x >> 5) + warp;
-  if (t >= n) return;
-  float* s = route_sm + (size_t)warp * (2 * n_out + groups);
-  float* c = s + n_out;
-  float* mark = c + n_out;
-  const float* z = logits + (size_t)t * ld;
-  if (scores == 1) {
+struct RouteParams {
+  const float* logits; long long ld;
+  // instead of logits: the partial tiles [splits][n * n_out] of the product that makes them (+ bias)
+  const float* part; int splits; const float* part_bias; long long part_stride;
+  int n, n_out, top, scores, groups, keep, normalise, mark_two;
+  const float* correction;
+  float weight_scale;
+};
+
+// One warp, one token; s, c [n_out] and mark [groups] are the warp's own shared memory.  Writes top choices and weights.
+__device__ __forceinline__ void route_token(const RouteParams& p, int t, float* s, float* c, float* mark, int lane, int* idx,
+                                            float* weight) {
+  const int n_out = p.n_out, top = p.top;
+  for (int e = lane; e < n_out; e += 32) {
+    float z;
+    if (p.part) {
+      const size_t at = (size_t)t * n_out + e;
+      sum_partials<1>(p.part, p.splits, (size_t)p.part_stride, &at, &z);
+      if (p.part_bias) z += p.part_bias[e];
+    } else {
+      z = p.logits[(size_t)t * p.ld + e];
+    }
+    s[e] = p.scores == 0 ? hy_sigmoid(z) : z;
+  }
+  if (p.scores == 1) {                                    // (every lane its own entries: no barrier in between)
     float mx = -INFINITY;
-    for (int e = lane; e < n_out; e += 32) mx = fmaxf(mx, z[e]);
+    for (int e = lane; e < n_out; e += 32) mx = fmaxf(mx, s[e]);
     mx = warp_max(mx);
     float sum = 0.f;
     for (int e = lane; e < n_out; e += 32) {
-      const float v = expf(z[e] - mx);
+      const float v = expf(s[e] - mx);
       s[e] = v;
       sum += v;
     }
     sum = warp_sum(sum);
     for (int e = lane; e < n_out; e += 32) s[e] = s[e] / sum;
-  } else if (scores == 2) {
-    for (int e = lane; e < n_out; e += 32) s[e] = z[e];
-  } else {
-    for (int e = lane; e < n_out; e += 32) s[e] = hy_sigmoid(z[e]);
   }
-  for (int e = lane; e < n_out; e += 32) c[e] = s[e] + (correction ? correction[e] : 0.f);
+  for (int e = lane; e < n_out; e += 32) c[e] = s[e] + (p.correction ? p.correction[e] : 0.f);
   __syncwarp();
-  const int gs = n_out / groups;
-  if (groups > 1 && keep < groups) {
-    for (int g = lane; g < groups; g += 32) {
+  const int gs = n_out / p.groups;
+  if (p.groups > 1 && p.keep < p.groups) {
+    for (int g = lane; g < p.groups; g += 32) {
       float b = -INFINITY, second = -INFINITY;
       for (int e = g * gs; e < (g + 1) * gs; ++e) {
         second = fmaxf(second, fminf(b, c[e]));
         b = fmaxf(b, c[e]);
       }
-      mark[g] = mark_two && gs > 1 ? b + second : b;
+      mark[g] = p.mark_two && gs > 1 ? b + second : b;
     }
     __syncwarp();
     // the `keep` best groups stay open: the mark of a group that is picked becomes +infinity, which no score
     // reaches, so that the pass below reads one flag per group
-    for (int k = 0; k < keep; ++k) {
+    for (int k = 0; k < p.keep; ++k) {
       float bv = -INFINITY;
       int bg = 0x7fffffff;
-      for (int g = lane; g < groups; g += 32) {
+      for (int g = lane; g < p.groups; g += 32) {
         const float v = mark[g];
         if (v != INFINITY && (bg == 0x7fffffff || v > bv)) { bv = v; bg = g; }
       }
@@ -144,25 +152,86 @@ __global__ void moe_route_grouped_kernel(const float* logits, long long ld, int 
       if (oe != 0x7fffffff && (be == 0x7fffffff || ov > bv || (ov == bv && oe < be))) { bv = ov; be = oe; }
     }
     if (lane == 0) {
-      idx[(size_t)t * top + k] = be;
-      weight[(size_t)t * top + k] = normalise ? s[be] : s[be] * weight_scale;
+      idx[k] = be;
+      weight[k] = p.normalise ? s[be] : s[be] * p.weight_scale;
       c[be] = -INFINITY;                                   // taken
     }
     __syncwarp();
   }
-  if (normalise && lane == 0) {
-    float* w = weight + (size_t)t * top;
+  if (p.normalise && lane == 0) {
     float sum = 0.f;
-    if (normalise == 2) {
-      const float mx = w[0];                                // (the first choice has the largest score)
+    if (p.normalise == 2) {
+      const float mx = weight[0];                           // (the first choice has the largest score)
       for (int k = 0; k < top; ++k) {
-        w[k] = expf(w[k] - mx);
-        sum += w[k];
+        weight[k] = expf(weight[k] - mx);
+        sum += weight[k];
       }
     } else {
-      for (int k = 0; k < top; ++k) sum += w[k];
+      for (int k = 0; k < top; ++k) sum += weight[k];
     }
-    for (int k = 0; k < top; ++k) w[k] = w[k] / sum * weight_scale;
+    for (int k = 0; k < top; ++k) weight[k] = weight[k] / sum * p.weight_scale;
+  }
+}
+
+// one warp per token
+__global__ void moe_route_grouped_kernel(RouteParams p, int* idx, float* weight) {
+  extern __shared__ float route_sm[];                    // per warp: scores [n_out], choice scores [n_out], group marks
+  pdl_trigger();
+  pdl_wait();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int t = blockIdx.x * (blockDim.x >> 5) + warp;
+  if (t >= p.n) return;
+  float* s = route_sm + (size_t)warp * (2 * p.n_out + p.groups);
+  route_token(p, t, s, s + p.n_out, s + 2 * p.n_out, lane, idx + (size_t)t * p.top, weight + (size_t)t * p.top);
+}
+
+// A step of few tokens: the choice, the pairs in the experts' order and the gathered rows in one kernel.  Every block makes the
+// choice and the order for itself, so that no block waits for another; the first one leaves them for the kernels behind, and
+// each copies its share of the rows.
+constexpr int DISPATCH_THREADS = 256, DISPATCH_PAIRS = 256, DISPATCH_TOKENS = 32;
+
+template <typename T>
+__global__ void __launch_bounds__(DISPATCH_THREADS)
+moe_dispatch_kernel(RouteParams p, int* idx, float* weight, int* offsets, int* row_pair, int* pair_row, const T* h, long long ldh,
+                    T* rows, long long ldr, int width, int weight_rows) {
+  extern __shared__ float dispatch_sm[];                 // per warp: scores, choice scores, group marks; then counts [n_out + 1]
+  __shared__ int s_idx[DISPATCH_PAIRS], s_row[DISPATCH_PAIRS];
+  __shared__ float s_w[DISPATCH_PAIRS];
+  pdl_trigger();
+  pdl_wait();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = DISPATCH_THREADS / 32;
+  const int pairs = p.n * p.top;
+  float* s = dispatch_sm + (size_t)warp * (2 * p.n_out + p.groups);
+  for (int t = warp; t < p.n; t += warps) route_token(p, t, s, s + p.n_out, s + 2 * p.n_out, lane, s_idx + t * p.top, s_w + t * p.top);
+  int* start = reinterpret_cast<int*>(dispatch_sm + (size_t)warps * (2 * p.n_out + p.groups));
+  __syncthreads();
+  // first row of every output's range, and behind the last one: pairs of outputs in front of it
+  for (int e = threadIdx.x; e <= p.n_out; e += DISPATCH_THREADS) {
+    int c = 0;
+    for (int q = 0; q < pairs; ++q) c += s_idx[q] < e;
+    start[e] = c;
+  }
+  __syncthreads();
+  for (int q = threadIdx.x; q < pairs; q += DISPATCH_THREADS) {
+    int r = start[s_idx[q]];
+    for (int o = 0; o < q; ++o) r += s_idx[o] == s_idx[q];
+    s_row[q] = r;
+  }
+  __syncthreads();
+  if (blockIdx.x == 0) {
+    for (int e = threadIdx.x; e <= p.n_out; e += DISPATCH_THREADS) offsets[e] = start[e];
+    for (int q = threadIdx.x; q < pairs; q += DISPATCH_THREADS) {
+      idx[q] = s_idx[q];
+      weight[q] = s_w[q];
+      pair_row[q] = s_row[q];
+      row_pair[s_row[q]] = q;
+    }
+  }
+  for (int q = blockIdx.x; q < pairs; q += gridDim.x) {
+    const float w = weight_rows ? s_w[q] : 1.f;
+    const T* src = h + (size_t)(q / p.top) * ldh;
+    T* dst = rows + (size_t)s_row[q] * ldr;
+    for (int d = threadIdx.x; d < width; d += DISPATCH_THREADS) dst[d] = from_f32<T>(w * to_f32(src[d]));
   }
 }
 
@@ -302,7 +371,8 @@ template <typename T>
 __global__ void moe_combine_weighted_any_kernel(const float* out, long long ldo, const int* pair_row, const int* idx,
                                                 const float* weight, const T* h, long long ldh, float* y, long long ldy,
                                                 int width, int top, int E, int accumulate, const float* shared,
-                                                long long lds, ThenNorm then) {
+                                                long long lds, int splits, size_t split_stride,
+                                                const float* __restrict__ shared_bias, ThenNorm then) {
   __shared__ float scratch[32];
   pdl_trigger();
   pdl_wait();
@@ -315,7 +385,14 @@ __global__ void moe_combine_weighted_any_kernel(const float* out, long long ldo,
       const float src = idx[p] < E ? out[(size_t)pair_row[p] * ldo + d] : to_f32(h[t * ldh + d]);
       v = fmaf(weight[p], src, v);
     }
-    if (shared) v += shared[t * lds + d];
+    if (splits > 0) {
+      float sh;
+      const size_t at = t * width + d;
+      sum_partials<1>(shared, splits, split_stride, &at, &sh);
+      v += shared_bias ? sh + shared_bias[d] : sh;
+    } else if (shared) {
+      v += shared[t * lds + d];
+    }
     o[d] = accumulate ? o[d] + v : v;
   }
   if (then.gain != nullptr) hy_then_norm_row(o, width, then, t, scratch);
@@ -334,7 +411,8 @@ template <typename T, int NV>
 __global__ void __launch_bounds__(256)
 moe_combine_weighted_kernel(const float* out, long long ldo, const int* pair_row, const int* idx, const float* weight,
                             const T* h, long long ldh, float* y, long long ldy, int width, int top, int E, int accumulate,
-                            const float* shared, long long lds, ThenNorm then) {
+                            const float* shared, long long lds, int splits, size_t split_stride,
+                            const float* __restrict__ shared_bias, ThenNorm then) {
   __shared__ float scratch[32];
   pdl_trigger();
   pdl_wait();
@@ -347,7 +425,25 @@ moe_combine_weighted_kernel(const float* out, long long ldo, const int* pair_row
     const int d = 4 * (threadIdx.x + i * blockDim.x);
     v[i] = zero;
     own[i] = d < width && accumulate ? load4_f32(o + d) : zero;
-    sh[i] = d < width && shared ? load4_f32(shared + t * lds + d) : zero;
+    sh[i] = d < width && shared && splits == 0 ? load4_f32(shared + t * lds + d) : zero;
+  }
+  for (int u = 0; u < splits; ++u) {                      // (shared: partial tiles [splits][tokens * width])
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int d = 4 * (threadIdx.x + i * blockDim.x);
+      if (d >= width) continue;
+      const float4 x = load4_f32(shared + u * split_stride + t * width + d);
+      sh[i].x += x.x; sh[i].y += x.y; sh[i].z += x.z; sh[i].w += x.w;
+    }
+  }
+  if (splits > 0 && shared_bias) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int d = 4 * (threadIdx.x + i * blockDim.x);
+      if (d >= width) continue;
+      const float4 x = load4_f32(shared_bias + d);
+      sh[i].x += x.x; sh[i].y += x.y; sh[i].z += x.z; sh[i].w += x.w;
+    }
   }
   for (int k = 0; k < top; ++k) {
     const size_t p = t * top + k;
@@ -376,28 +472,80 @@ moe_combine_weighted_kernel(const float* out, long long ldo, const int* pair_row
 
 }  // namespace
 
-// a0 logits (f32), a1 their row stride, a2 tokens, a3 router outputs (experts and identity outputs), a4 top, a5 scores
-// (0 sigmoid, 1 softmax, 2 the logits), a6 correction [outputs] (f32) or 0, a7 groups (1: none), a8 groups kept, a9 chosen
-// outputs [tokens, top] (int32), a10 their weights (f32), a11 how the chosen scores become weights: 0 as they are, 1
-// divided by their sum, 2 their softmax, a12 a group's mark: 0 its largest choice score, 1 the sum of its two largest;
-// f0 factor on the weights (0 means 1)
+namespace {
+
+// The router's operands: a0 logits (f32), a1 their row stride, a2 tokens, a3 router outputs (experts and identity outputs), a4
+// top, a5 scores (0 sigmoid, 1 softmax, 2 the logits), a6 correction [outputs] (f32) or 0, a7 groups (1: none), a8 groups kept,
+// a9 chosen outputs [tokens, top] (int32), a10 their weights (f32), a11 how the chosen scores become weights: 0 as they are, 1
+// divided by their sum, 2 their softmax, a12 a group's mark: 0 its largest choice score, 1 the sum of its two largest; f0 factor
+// on the weights (0 means 1).  A record with GB_OP_TAKES_PARTIALS: the logits are partial tiles of the product in front.
+int route_params(const GbPlanCtx* ctx, const long long* a, const double* f, RouteParams& p) {
+  p.logits = op_ptr<const float>(a[0]); p.ld = a[1];
+  p.part = ctx->part_splits > 0 ? ctx->part : nullptr;
+  p.splits = ctx->part_splits; p.part_bias = ctx->part_bias;
+  p.n = (int)a[2]; p.n_out = (int)a[3]; p.top = (int)a[4]; p.scores = (int)a[5];
+  p.part_stride = (long long)p.n * p.n_out;
+  p.correction = op_ptr<const float>(a[6]);
+  p.groups = (int)a[7]; p.keep = (int)a[8];
+  p.normalise = (int)a[11]; p.mark_two = (int)a[12];
+  p.weight_scale = f[0] != 0.0 ? (float)f[0] : 1.f;
+  if (p.groups < 1) p.groups = 1;
+  if (p.keep < 1 || p.keep > p.groups) p.keep = p.groups;
+  if (p.n_out > MOE_MAX_EXPERTS) GB_FAIL(GB_ERR_ARG, "moe_route_grouped: %d router outputs (at most %d)", p.n_out, MOE_MAX_EXPERTS);
+  if (p.n_out % p.groups) GB_FAIL(GB_ERR_ARG, "moe_route_grouped: %d router outputs in %d groups", p.n_out, p.groups);
+  if (p.top < 1 || p.top > (p.n_out / p.groups) * p.keep)
+    GB_FAIL(GB_ERR_ARG, "moe_route_grouped: top %d of the %d outputs in %d open groups", p.top, (p.n_out / p.groups) * p.keep, p.keep);
+  return GB_OK;
+}
+
+}  // namespace
+
+// (operands: route_params)
 GB_OP(gb_op_moe_route_grouped) {
-  const int n = (int)a[2], n_out = (int)a[3], top = (int)a[4];
-  int groups = (int)a[7], keep = (int)a[8];
-  if (n <= 0) return 0;
-  if (groups < 1) groups = 1;
-  if (keep < 1 || keep > groups) keep = groups;
-  if (n_out > MOE_MAX_EXPERTS) GB_FAIL(GB_ERR_ARG, "moe_route_grouped: %d router outputs (at most %d)", n_out, MOE_MAX_EXPERTS);
-  if (n_out % groups) GB_FAIL(GB_ERR_ARG, "moe_route_grouped: %d router outputs in %d groups", n_out, groups);
-  if (top < 1 || top > (n_out / groups) * keep)
-    GB_FAIL(GB_ERR_ARG, "moe_route_grouped: top %d of the %d outputs in %d open groups", top, (n_out / groups) * keep, keep);
+  RouteParams p;
+  if (a[2] <= 0) return 0;
+  const int rc = route_params(ctx, a, f, p);
+  if (rc < 0) return rc;
   const int warps = 4;
-  const size_t smem = sizeof(float) * warps * (2 * (size_t)n_out + groups);
-  gb_launch(moe_route_grouped_kernel, dim3(gb_div_up(n, warps)), dim3(32 * warps), smem, ctx->stream,
-            op_ptr<const float>(a[0]), a[1], n, n_out, top, (int)a[5], op_ptr<const float>(a[6]), groups, keep,
-            op_ptr<int>(a[9]), op_ptr<float>(a[10]), (int)a[11], (int)a[12], f[0] != 0.0 ? (float)f[0] : 1.f);
+  const size_t smem = sizeof(float) * warps * (2 * (size_t)p.n_out + p.groups);
+  gb_launch(moe_route_grouped_kernel, dim3(gb_div_up(p.n, warps)), dim3(32 * warps), smem, ctx->stream, p, op_ptr<int>(a[9]),
+            op_ptr<float>(a[10]));
   GB_CHECK_LAUNCH("moe_route_grouped");
   return 1;
+}
+
+GB_OP(gb_op_moe_sort);
+GB_OP(gb_op_moe_gather);
+
+// The choice, the experts' order and the gathered rows: moe_route_grouped, moe_sort and moe_gather, in one kernel for a step
+// of few tokens.  a0 to a12 and f0 as of route_params, a13 offsets [outputs + 1], a14 row -> pair, a15 pair -> row, a16 h, a17 its
+// row stride, a18 dtype (of h and rows), a19 rows out, a20 their stride, a21 width; flags bit 0: a row is multiplied by its weight
+GB_OP(gb_op_moe_dispatch) {
+  RouteParams p;
+  if (a[2] <= 0) return 0;
+  const int rc = route_params(ctx, a, f, p);
+  if (rc < 0) return rc;
+  const size_t smem = sizeof(float) * (DISPATCH_THREADS / 32 * (2 * (size_t)p.n_out + p.groups) + p.n_out + 1);
+  if (p.n <= DISPATCH_TOKENS && (long long)p.n * p.top <= DISPATCH_PAIRS && smem <= 40 * 1024) {
+    const int pairs = p.n * p.top;
+    const dim3 grid(pairs < 64 ? pairs : 64);
+#define DISPATCH(T)                                                                                                     \
+    gb_launch(moe_dispatch_kernel<T>, grid, dim3(DISPATCH_THREADS), smem, ctx->stream, p, op_ptr<int>(a[9]), op_ptr<float>(a[10]), \
+              op_ptr<int>(a[13]), op_ptr<int>(a[14]), op_ptr<int>(a[15]), op_ptr<const T>(a[16]), a[17], op_ptr<T>(a[19]), a[20],   \
+              (int)a[21], flags & 1)
+    if (a[18] == GB_BF16) DISPATCH(bf16); else DISPATCH(float);
+#undef DISPATCH
+    GB_CHECK_LAUNCH("moe_dispatch");
+    return 1;
+  }
+  const int r1 = gb_op_moe_route_grouped(ctx, a, f, 0);
+  if (r1 < 0) return r1;
+  const long long so[24] = {a[9], a[2], a[3], a[13], a[14], a[15], a[4]};
+  const int r2 = gb_op_moe_sort(ctx, so, f, 0);
+  if (r2 < 0) return r2;
+  const long long ga[24] = {a[16], a[17], a[18], a[14], (flags & 1) ? a[10] : 0, a[19], a[20], a[2], a[21], a[4]};
+  const int r3 = gb_op_moe_gather(ctx, ga, f, 0);
+  return r3 < 0 ? r3 : r1 + r2 + r3;
 }
 
 // a0 logits (f32), a1 their row stride, a2 tokens, a3 experts, a4 top, a5 column of the shared expert's gate logit,
@@ -491,17 +639,22 @@ GB_OP(gb_op_moe_combine) {
 // a5 the feed-forward's input h, a6 its row stride, a7 its dtype, a8 y (f32), a9 its row stride, a10 tokens, a11 width,
 // a12 top, a13 real experts (a choice from here on returns h), a14 an output added for every token (f32) or 0, a15 its row
 // stride, a16 gain of a norm taken of the new rows or 0: none, a17 its output [tokens, width], a18 that dtype, a19 its kind
-// (0 layer norm, 1 RMS norm), a20 its eps (the bits of a 32-bit float); flags bit 0: add into y
+// (0 layer norm, 1 RMS norm), a20 its eps (the bits of a 32-bit float); flags bit 0: add into y.  A record with
+// GB_OP_TAKES_PARTIALS: a14's output may be partial tiles of the product in front
 GB_OP(gb_op_moe_combine_weighted) {
   const int n = (int)a[10], width = (int)a[11];
   if (n <= 0) return 0;
   const ThenNorm then = hy_then_of(a[16], a[17], a[18], a[19], a[20]);
-  const bool vec = width % 4 == 0 && width <= 4096 && a[1] % 4 == 0 && a[6] % 4 == 0 && a[9] % 4 == 0 && a[15] % 4 == 0 &&
+  const int splits = a[14] ? ctx->part_splits : 0;
+  const float* shared = splits > 0 ? ctx->part : op_ptr<const float>(a[14]);
+  const float* shared_bias = splits > 0 ? ctx->part_bias : nullptr;
+  const size_t split_stride = (size_t)n * width;
+  const bool vec = (((uintptr_t)shared | (uintptr_t)shared_bias) & 15) == 0 && width % 4 == 0 && width <= 4096 && a[1] % 4 == 0 && a[6] % 4 == 0 && a[9] % 4 == 0 && a[15] % 4 == 0 &&
                    ((a[0] | a[8] | a[14]) & 15) == 0 && (a[5] & (a[7] == GB_BF16 ? 7 : 15)) == 0 && hy_then_vec(then);
 #define COMBINE(T, KERNEL, THREADS)                                                                                     \
   gb_launch(KERNEL, dim3(n), dim3(THREADS), 0, ctx->stream, op_ptr<const float>(a[0]), a[1], op_ptr<const int>(a[2]),    \
             op_ptr<const int>(a[3]), op_ptr<const float>(a[4]), op_ptr<const T>(a[5]), a[6], op_ptr<float>(a[8]), a[9],  \
-            width, (int)a[12], (int)a[13], flags & 1, op_ptr<const float>(a[14]), a[15], then)
+            width, (int)a[12], (int)a[13], flags & 1, shared, a[15], splits, split_stride, shared_bias, then)
   const int threads = hy_row_threads(width);
 #define COMBINE_OF(T)                                                                                                   \
   do {                                                                                                                  \

@@ -498,7 +498,7 @@ template <int NV>
 __global__ void __launch_bounds__(256)
 normed_sum_kernel(float* x, long long ldx, const float* y1, long long ld1, const float* __restrict__ g1, const float* y2,
                   long long ld2, const float* __restrict__ g2, int dim, float eps, float f1, float f2, int accumulate,
-                  ThenNorm then) {
+                  int splits, size_t split_stride, const float* __restrict__ part_bias, ThenNorm then) {
   __shared__ float scratch[32];
   pdl_trigger();
   const size_t row = blockIdx.x;
@@ -521,9 +521,31 @@ normed_sum_kernel(float* x, long long ldx, const float* y1, long long ld1, const
   for (int i = 0; i < NV; ++i) {
     const int d = 4 * (threadIdx.x + i * blockDim.x);
     const bool in = d < dim;
-    ya[i] = in ? *reinterpret_cast<const float4*>(a + d) : zero;
-    yb[i] = in && b ? *reinterpret_cast<const float4*>(b + d) : zero;
+    ya[i] = in && (b || splits == 0) ? *reinterpret_cast<const float4*>(a + d) : zero;
+    yb[i] = in && b && splits == 0 ? *reinterpret_cast<const float4*>(b + d) : zero;
     v[i] = in && accumulate ? *reinterpret_cast<const float4*>(o + d) : zero;
+  }
+  // the last of the outputs as partial tiles [splits][rows * dim]: added in their order
+  for (int u = 0; u < splits; ++u) {
+    const float* part = (b ? y2 : y1) + u * split_stride + row * dim;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int d = 4 * (threadIdx.x + i * blockDim.x);
+      if (d >= dim) continue;
+      const float4 x = *reinterpret_cast<const float4*>(part + d);
+      float4& y = b ? yb[i] : ya[i];
+      y.x += x.x; y.y += x.y; y.z += x.z; y.w += x.w;
+    }
+  }
+  if (splits > 0 && part_bias) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int d = 4 * (threadIdx.x + i * blockDim.x);
+      if (d >= dim) continue;
+      const float4 x = *reinterpret_cast<const float4*>(part_bias + d);
+      float4& y = b ? yb[i] : ya[i];
+      y.x += x.x; y.y += x.y; y.z += x.z; y.w += x.w;
+    }
   }
   float s1 = 0.f, s2 = 0.f;
 #pragma unroll
@@ -549,7 +571,8 @@ normed_sum_kernel(float* x, long long ldx, const float* y1, long long ld1, const
 // The same for rows of any length and alignment, read again for every pass.
 __global__ void normed_sum_any_kernel(float* x, long long ldx, const float* y1, long long ld1, const float* __restrict__ g1,
                                       const float* y2, long long ld2, const float* __restrict__ g2, int dim, float eps,
-                                      float f1, float f2, int accumulate, ThenNorm then) {
+                                      float f1, float f2, int accumulate, int splits, size_t split_stride,
+                                      const float* __restrict__ part_bias, ThenNorm then) {
   __shared__ float scratch[32];
   pdl_trigger();
   pdl_wait();
@@ -557,16 +580,26 @@ __global__ void normed_sum_any_kernel(float* x, long long ldx, const float* y1, 
   float* o = x + row * ldx;
   const float* a = y1 + row * ld1;
   const float* b = y2 ? y2 + row * ld2 : nullptr;
+  // entry d of the first (second) output; the last of them may be partial tiles [splits][rows * dim]
+  auto partial = [&](const float* y, int d) {
+    float v;
+    const size_t at = row * dim + d;
+    sum_partials<1>(y, splits, split_stride, &at, &v);
+    return part_bias ? v + part_bias[d] : v;
+  };
+  auto first = [&](int d) { return b || splits == 0 ? a[d] : partial(y1, d); };
+  auto second = [&](int d) { return splits == 0 ? b[d] : partial(y2, d); };
   float s1 = 0.f, s2 = 0.f;
   for (int d = threadIdx.x; d < dim; d += blockDim.x) {
-    s1 += a[d] * a[d];
-    if (b) s2 += b[d] * b[d];
+    const float v = first(d), w = b ? second(d) : 0.f;
+    s1 += v * v;
+    s2 += w * w;
   }
   const float r1 = f1 / sqrtf(block_sum(s1, scratch) / (float)dim + eps);
   const float r2 = b ? f2 / sqrtf(block_sum(s2, scratch) / (float)dim + eps) : 0.f;
   for (int d = threadIdx.x; d < dim; d += blockDim.x) {
-    float s = a[d] * r1 * g1[d];
-    if (b) s = fmaf(b[d] * r2, g2[d], s);
+    float s = first(d) * r1 * g1[d];
+    if (b) s = fmaf(second(d) * r2, g2[d], s);
     o[d] = accumulate ? o[d] + s : s;
   }
   if (then.gain != nullptr) hy_then_norm_row(o, dim, then, row, scratch);
@@ -807,17 +840,22 @@ GB_OP(gb_op_head_norm) {
 // a0 x (f32), a1 its row stride, a2 y1 (f32), a3 its row stride, a4 its gain [dim], a5 y2 (f32) or 0, a6 its row stride,
 // a7 its gain, a8 rows, a9 dim, a10 gain of a norm taken of the new rows or 0: none, a11 its output [rows, dim], a12 that
 // dtype, a13 its kind (0 layer norm, 1 RMS norm), a14 its eps (the bits of a 32-bit float); f0 eps of y1's and y2's norm,
-// f1 factor on the first, f2 on the second; flags bit 0: add into x (else it is overwritten)
+// f1 factor on the first, f2 on the second; flags bit 0: add into x (else it is overwritten).  A record with
+// GB_OP_TAKES_PARTIALS: the last of the outputs may be partial tiles of the product in front
 GB_OP(gb_op_normed_sum) {
   const int n = (int)a[8], dim = (int)a[9];
   if (n <= 0) return 0;
   const ThenNorm then = hy_then_of(a[10], a[11], a[12], a[13], a[14]);
+  const int splits = ctx->part_splits;
+  const float* part_bias = splits > 0 ? ctx->part_bias : nullptr;
+  const float* y1 = splits > 0 && !a[5] ? ctx->part : op_ptr<const float>(a[2]);
+  const float* y2 = splits > 0 && a[5] ? ctx->part : op_ptr<const float>(a[5]);
   const bool vec = dim % 4 == 0 && dim <= 4096 && a[1] % 4 == 0 && a[3] % 4 == 0 && a[6] % 4 == 0 &&
-                   ((a[0] | a[2] | a[4] | a[5] | a[7]) & 15) == 0 && hy_then_vec(then);
+                   ((a[0] | (uintptr_t)y1 | a[4] | (uintptr_t)y2 | a[7] | (uintptr_t)part_bias) & 15) == 0 && hy_then_vec(then);
 #define NORMED_SUM(KERNEL, THREADS)                                                                                     \
-  gb_launch(KERNEL, dim3(n), dim3(THREADS), 0, ctx->stream, op_ptr<float>(a[0]), a[1], op_ptr<const float>(a[2]), a[3],  \
-            op_ptr<const float>(a[4]), op_ptr<const float>(a[5]), a[6], op_ptr<const float>(a[7]), dim, (float)f[0],      \
-            (float)f[1], (float)f[2], flags & 1, then)
+  gb_launch(KERNEL, dim3(n), dim3(THREADS), 0, ctx->stream, op_ptr<float>(a[0]), a[1], y1, a[3],  \
+            op_ptr<const float>(a[4]), y2, a[6], op_ptr<const float>(a[7]), dim, (float)f[0], (float)f[1], (float)f[2],   \
+            flags & 1, splits, (size_t)n * dim, part_bias, then)
   const int threads = hy_row_threads(dim);
   if (!vec) NORMED_SUM(normed_sum_any_kernel, norm_threads(dim));
   else if (dim <= 4 * threads) NORMED_SUM(normed_sum_kernel<1>, threads);

@@ -25,7 +25,7 @@ OPERATIONS = ("row_norm", "norm_add", "clamped_glu", "gelu_mul_rows", "gated_gro
               "moe_experts", "moe_experts_tc", "moe_combine", "moe_route_grouped", "moe_combine_weighted",
               "embed_scaled", "qk_prep", "sink_attention", "sink_attention_tc", "act_rows", "head_norm", "delta_prep",
               "delta_scan", "scaled_sum", "sigmoid_attention", "sigmoid_attention_tc", "linear_scan", "forget_write_gates",
-              "exp_gates", "low_rank_decays", "normed_sum", "selective_scan", "stream_read", "stream_mix")
+              "exp_gates", "low_rank_decays", "normed_sum", "moe_dispatch", "selective_scan", "stream_read", "stream_mix")
 
 NORM_LAYER, NORM_RMS = 0, 1
 TAKES_PENDING = 1 << 30          # a record's flag: the operation adds the sums a product left pending itself

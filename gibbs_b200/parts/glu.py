@@ -195,27 +195,30 @@ class RoutedGLU(BranchPart, FeedForward):
         if accumulate and not self.weight_on_output:
             raise ValueError("a routed unit with weights on the experts' inputs writes its output")
         logits = rn.buffer("moe_logits", n_out + (1 if shared else 0), torch.float32)
-        rn.linear(h, self.w_router, self.router_bias, logits, role="router")
         idx = rn.buffer("moe_choice", top, torch.int32)
         wts = rn.buffer("moe_weight", top, torch.float32)
         sg = rn.buffer("moe_shared_gate", 1, torch.float32)
-        if self.plain_rule:
-            rn.op("moe_route", [logits.data_ptr(), logits.stride(0), rn.N, E, top, E, idx.data_ptr(), wts.data_ptr(),
-                                sg.data_ptr() if shared else 0])
-        else:
-            if shared:
-                raise ValueError("a shared expert's gate comes with the plain router rule")
-            rn.op("moe_route_grouped", [logits.data_ptr(), logits.stride(0), rn.N, n_out, top, self.scores,
-                                        keep(rn, self.correction), self.groups, self.groups_keep, idx.data_ptr(),
-                                        wts.data_ptr(), self.normalise, self.mark_two], [self.weight_scale])
         # (identity outputs are sorted behind the experts: their rows lie beyond offsets[E] and no product reads them)
         offsets = rn.buffer("moe_offsets", n_out + 1, torch.int32, fixed_rows=1)
         row_pair = rn.buffer("moe_row_pair", top, torch.int32)
         pair_row = rn.buffer("moe_pair_row", top, torch.int32)
-        rn.op("moe_sort", [idx.data_ptr(), rn.N, n_out, offsets.data_ptr(), row_pair.data_ptr(), pair_row.data_ptr(), top])
         rows = rn.buffer("moe_rows", d, per_token=top)
-        rn.op("moe_gather", [h.data_ptr(), h.stride(0), ops.dtype_code(h.dtype), row_pair.data_ptr(),
-                             0 if self.weight_on_output else wts.data_ptr(), rows.data_ptr(), rows.stride(0), rn.N, d, top])
+        if self.plain_rule:
+            rn.linear(h, self.w_router, self.router_bias, logits, role="router")
+            rn.op("moe_route", [logits.data_ptr(), logits.stride(0), rn.N, E, top, E, idx.data_ptr(), wts.data_ptr(),
+                                sg.data_ptr() if shared else 0])
+            rn.op("moe_sort", [idx.data_ptr(), rn.N, n_out, offsets.data_ptr(), row_pair.data_ptr(), pair_row.data_ptr(), top])
+            rn.op("moe_gather", [h.data_ptr(), h.stride(0), ops.dtype_code(h.dtype), row_pair.data_ptr(),
+                                 0 if self.weight_on_output else wts.data_ptr(), rows.data_ptr(), rows.stride(0), rn.N, d, top])
+        else:
+            if shared:
+                raise ValueError("a shared expert's gate comes with the plain router rule")
+            rn.partial_linear(h, self.w_router, self.router_bias, logits, role="router")
+            rn.op("moe_dispatch", [logits.data_ptr(), logits.stride(0), rn.N, n_out, top, self.scores, keep(rn, self.correction),
+                                   self.groups, self.groups_keep, idx.data_ptr(), wts.data_ptr(), self.normalise, self.mark_two,
+                                   offsets.data_ptr(), row_pair.data_ptr(), pair_row.data_ptr(), h.data_ptr(), h.stride(0),
+                                   ops.dtype_code(h.dtype), rows.data_ptr(), rows.stride(0), d], [self.weight_scale],
+                  flags=(0 if self.weight_on_output else 1) | hybrid.TAKES_PARTIALS)
         act = rn.buffer("moe_act", f, per_token=top)
         wdt = ops.dtype_code(self.w_down.dtype)
         eout = rn.buffer("moe_expert_out", d, torch.float32, per_token=top)
@@ -246,13 +249,16 @@ class RoutedGLU(BranchPart, FeedForward):
             sh = None
             if self.shared is not None:
                 sh = rn.buffer("moe_shared_out", d, torch.float32)
+                # (the kernel behind it adds the partial tiles its last product may leave)
+                leaves, rn.partial_branches = rn.partial_branches, True
                 self.shared.run(rn, h, sh)
+                rn.partial_branches = leaves
             behind, normed_rows = then_operands(rn, then)
             rn.op("moe_combine_weighted", [eout.data_ptr(), eout.stride(0), pair_row.data_ptr(), idx.data_ptr(),
                                            wts.data_ptr(), h.data_ptr(), h.stride(0), ops.dtype_code(h.dtype),
                                            out.data_ptr(), out.stride(0), rn.N, d, top, E,
                                            0 if sh is None else sh.data_ptr(), 0 if sh is None else sh.stride(0), *behind],
-                  flags=1 if accumulate else 0)
+                  flags=(1 if accumulate else 0) | (0 if sh is None else hybrid.TAKES_PARTIALS))
             return normed_rows
         sh = None
         if shared:

@@ -114,13 +114,15 @@ class ParallelMixers(BranchPart, Mixer):
         ys = []
         for i, side in enumerate(self.sides):
             y = rn.buffer(f"par_out{i}", self.hidden, torch.float32)
-            rn.linear(o[:, starts[i]:starts[i] + side.heads_width], self.out_weights[i], None, y, role="par_out")
+            # (the last product may leave its sums in parts: the kernel behind it adds them)
+            linear = rn.partial_linear if i == len(self.sides) - 1 else rn.linear
+            linear(o[:, starts[i]:starts[i] + side.heads_width], self.out_weights[i], None, y, role="par_out")
             ys.append([y.data_ptr(), y.stride(0), keep(rn, self.gains[i])])
         ys += [[0, 0, 0]] * (2 - len(ys))
         behind, normed_rows = then_operands(rn, then)
         rn.op("normed_sum", [out.data_ptr(), out.stride(0), *ys[0], *ys[1], rn.N, self.hidden, *behind],
               [self.out_norm_eps, self.factors[0], self.factors[1] if len(self.sides) > 1 else 0.0],
-              flags=1 if accumulate else 0)
+              flags=(1 if accumulate else 0) | hybrid.TAKES_PARTIALS)
         return normed_rows
 
 

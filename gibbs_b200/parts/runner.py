@@ -54,6 +54,11 @@ class Runner:
         ``ops.EPILOGUES``: the product's epilogue applies it to the 32-bit sums."""
         raise NotImplementedError
 
+    def partial_linear(self, x, weight, bias, out, role: str = "") -> None:
+        """out = x weight^T (+ bias) in 32-bit for the operation recorded next, which takes partial tiles
+        (``hybrid.TAKES_PARTIALS``): a plan may leave the sums of a split K in parts."""
+        self.linear(x, weight, bias, out, role=role)
+
     # set by an arrangement whose next kernel reads a sublayer's output and can add up partial tiles itself
     partial_branches = False
 
@@ -144,11 +149,14 @@ class Planned(Runner):
     def act_linear(self, x, weight, bias, out, act, role=""):
         self.plan.linear(x, weight, bias, out, "plain", role=role or "act", act=ops.EPILOGUES[act])
 
+    def partial_linear(self, x, weight, bias, out, role=""):
+        # (the sum of the partial tiles in their order is what the product's own reduction writes)
+        self.plan.linear(x, weight, bias, out, "plain", role=role or "plain", partials="always")
+
     def branch_linear(self, x, weight, bias, out, accumulate=False, role=""):
         if accumulate or not self.partial_branches:
             return super().branch_linear(x, weight, bias, out, accumulate, role)
-        # (the sum of the partial tiles in their order is what the product's own reduction writes)
-        self.plan.linear(x, weight, bias, out, "plain", role=role or "plain", partials="always")
+        self.partial_linear(x, weight, bias, out, role)
 
     def op(self, name, a, f=(), label="", flags=0):
         self.plan.emit(hybrid.plan_id(name), list(a), list(f), flags=flags, label=label or name)
