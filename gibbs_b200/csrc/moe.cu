@@ -74,19 +74,66 @@ struct RouteParams {
   float weight_scale;
 };
 
+// A 32-bit number whose order as an unsigned integer is the order of floats (no NaNs).
+__device__ __forceinline__ unsigned ordered(float v) {
+  const unsigned b = __float_as_uint(v);
+  return b & 0x80000000u ? ~b : b | 0x80000000u;
+}
+
+// At most 32 router outputs, sigmoid scores or logits, weights as they are: a lane an output, maxima by one reduction over the
+// warp and ties by the lowest lane.  The same choices and weights as below.
+__device__ __forceinline__ void route_token_32(const RouteParams& p, float z, int lane, int* idx, float* weight) {
+  const bool in = lane < p.n_out;
+  const float s = p.scores == 0 ? hy_sigmoid(z) : z;
+  const float c = s + (in && p.correction ? p.correction[lane] : 0.f);
+  bool open = in;
+  if (p.groups > 1 && p.keep < p.groups) {
+    const int gs = p.n_out / p.groups;
+    const int g = lane < p.groups ? lane : 0;             // lane g marks group g
+    float b = -INFINITY, second = -INFINITY;
+    for (int e = 0; e < gs; ++e) {
+      const float v = __shfl_sync(0xffffffffu, c, g * gs + e);
+      second = fmaxf(second, fminf(b, v));
+      b = fmaxf(b, v);
+    }
+    const unsigned mark = lane < p.groups ? max(ordered(p.mark_two && gs > 1 ? b + second : b), 1u) : 0u;
+    unsigned kept = 0;
+    for (int k = 0; k < p.keep; ++k) {
+      const unsigned mine = (kept >> lane) & 1u ? 0u : mark;
+      const unsigned top = __reduce_max_sync(0xffffffffu, mine);
+      kept |= 1u << (__ffs(__ballot_sync(0xffffffffu, mine == top)) - 1);
+    }
+    open = in && ((kept >> (lane / gs)) & 1u);
+  }
+  unsigned key = open ? max(ordered(c), 2u) : in ? 1u : 0u;
+  for (int k = 0; k < p.top; ++k) {
+    const unsigned top = __reduce_max_sync(0xffffffffu, key);
+    const int e = __ffs(__ballot_sync(0xffffffffu, key == top)) - 1;
+    if (lane == e) {
+      idx[k] = e;
+      weight[k] = s * p.weight_scale;
+      key = 1u;                                            // taken
+    }
+  }
+}
+
 // One warp, one token; s, c [n_out] and mark [groups] are the warp's own shared memory.  Writes top choices and weights.
 __device__ __forceinline__ void route_token(const RouteParams& p, int t, float* s, float* c, float* mark, int lane, int* idx,
                                             float* weight) {
   const int n_out = p.n_out, top = p.top;
-  for (int e = lane; e < n_out; e += 32) {
+  auto logit = [&](int e) {
+    if (!p.part) return p.logits[(size_t)t * p.ld + e];
     float z;
-    if (p.part) {
-      const size_t at = (size_t)t * n_out + e;
-      sum_partials<1>(p.part, p.splits, (size_t)p.part_stride, &at, &z);
-      if (p.part_bias) z += p.part_bias[e];
-    } else {
-      z = p.logits[(size_t)t * p.ld + e];
-    }
+    const size_t at = (size_t)t * n_out + e;
+    sum_partials<1>(p.part, p.splits, (size_t)p.part_stride, &at, &z);
+    return p.part_bias ? z + p.part_bias[e] : z;
+  };
+  if (n_out <= 32 && p.scores != 1 && !p.normalise) {
+    route_token_32(p, lane < n_out ? logit(lane) : 0.f, lane, idx, weight);
+    return;
+  }
+  for (int e = lane; e < n_out; e += 32) {
+    const float z = logit(e);
     s[e] = p.scores == 0 ? hy_sigmoid(z) : z;
   }
   if (p.scores == 1) {                                    // (every lane its own entries: no barrier in between)
@@ -185,6 +232,11 @@ __global__ void moe_route_grouped_kernel(RouteParams p, int* idx, float* weight)
   route_token(p, t, s, s + p.n_out, s + 2 * p.n_out, lane, idx + (size_t)t * p.top, weight + (size_t)t * p.top);
 }
 
+// A row copied in pieces of 16 bytes by the whole block.
+__device__ __forceinline__ void copy_row16(const void* src, void* dst, int pieces) {
+  for (int i = threadIdx.x; i < pieces; i += blockDim.x) static_cast<uint4*>(dst)[i] = static_cast<const uint4*>(src)[i];
+}
+
 // A step of few tokens: the choice, the pairs in the experts' order and the gathered rows in one kernel.  Every block makes the
 // choice and the order for itself, so that no block waits for another; the first one leaves them for the kernels behind, and
 // each copies its share of the rows.
@@ -193,7 +245,7 @@ constexpr int DISPATCH_THREADS = 256, DISPATCH_PAIRS = 256, DISPATCH_TOKENS = 32
 template <typename T>
 __global__ void __launch_bounds__(DISPATCH_THREADS)
 moe_dispatch_kernel(RouteParams p, int* idx, float* weight, int* offsets, int* row_pair, int* pair_row, const T* h, long long ldh,
-                    T* rows, long long ldr, int width, int weight_rows) {
+                    T* rows, long long ldr, int width, int weight_rows, int vec) {
   extern __shared__ float dispatch_sm[];                 // per warp: scores, choice scores, group marks; then counts [n_out + 1]
   __shared__ int s_idx[DISPATCH_PAIRS], s_row[DISPATCH_PAIRS];
   __shared__ float s_w[DISPATCH_PAIRS];
@@ -208,12 +260,14 @@ moe_dispatch_kernel(RouteParams p, int* idx, float* weight, int* offsets, int* r
   // first row of every output's range, and behind the last one: pairs of outputs in front of it
   for (int e = threadIdx.x; e <= p.n_out; e += DISPATCH_THREADS) {
     int c = 0;
+#pragma unroll 8
     for (int q = 0; q < pairs; ++q) c += s_idx[q] < e;
     start[e] = c;
   }
   __syncthreads();
   for (int q = threadIdx.x; q < pairs; q += DISPATCH_THREADS) {
     int r = start[s_idx[q]];
+#pragma unroll 8
     for (int o = 0; o < q; ++o) r += s_idx[o] == s_idx[q];
     s_row[q] = r;
   }
@@ -231,6 +285,10 @@ moe_dispatch_kernel(RouteParams p, int* idx, float* weight, int* offsets, int* r
     const float w = weight_rows ? s_w[q] : 1.f;
     const T* src = h + (size_t)(q / p.top) * ldh;
     T* dst = rows + (size_t)s_row[q] * ldr;
+    if (vec && !weight_rows) {
+      copy_row16(src, dst, width * (int)sizeof(T) / 16);
+      continue;
+    }
     for (int d = threadIdx.x; d < width; d += DISPATCH_THREADS) dst[d] = from_f32<T>(w * to_f32(src[d]));
   }
 }
@@ -260,6 +318,18 @@ __global__ void moe_sort_kernel(const int* idx, int pairs, int E, int* offsets, 
     row_pair[row] = p;
     pair_row[p] = row;
   }
+}
+
+// several rows a block: `lanes` neighbouring threads (whole warps) a row
+__global__ void moe_gather16_kernel(const char* h, long long ldh_bytes, const int* row_pair, char* rows, long long ldr_bytes, int pairs,
+                                    int pieces, int top, int lanes) {
+  pdl_trigger();
+  const int row = blockIdx.x * (blockDim.x / lanes) + threadIdx.x / lanes;
+  pdl_wait();
+  if (row >= pairs) return;
+  const uint4* src = reinterpret_cast<const uint4*>(h + (size_t)(row_pair[row] / top) * ldh_bytes);
+  uint4* dst = reinterpret_cast<uint4*>(rows + (size_t)row * ldr_bytes);
+  for (int i = threadIdx.x % lanes; i < pieces; i += lanes) dst[i] = src[i];
 }
 
 template <typename T>
@@ -445,18 +515,30 @@ moe_combine_weighted_kernel(const float* out, long long ldo, const int* pair_row
       sh[i].x += x.x; sh[i].y += x.y; sh[i].z += x.z; sh[i].w += x.w;
     }
   }
-  for (int k = 0; k < top; ++k) {
-    const size_t p = t * top + k;
-    const float w = weight[p];
-    const bool real = idx[p] < E;
-    const float* src = out + (size_t)pair_row[p] * ldo;
+  // four choices at a time, so that their rows are on their way together
+  for (int k0 = 0; k0 < top; k0 += 4) {
+    float w[4];
+    int row[4];
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      const size_t p = t * top + min(k0 + u, top - 1);
+      w[u] = k0 + u < top ? weight[p] : 0.f;
+      row[u] = idx[p] < E ? pair_row[p] : -1;
+    }
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int d = 4 * (threadIdx.x + i * blockDim.x);
       if (d >= width) continue;
-      const float4 x = real ? load4_f32(src + d) : load4_f32(h + t * ldh + d);
-      v[i].x = fmaf(w, x.x, v[i].x); v[i].y = fmaf(w, x.y, v[i].y);
-      v[i].z = fmaf(w, x.z, v[i].z); v[i].w = fmaf(w, x.w, v[i].w);
+      float4 x[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u)
+        if (k0 + u < top) x[u] = row[u] >= 0 ? load4_f32(out + (size_t)row[u] * ldo + d) : load4_f32(h + t * ldh + d);
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        if (k0 + u >= top) continue;
+        v[i].x = fmaf(w[u], x[u].x, v[i].x); v[i].y = fmaf(w[u], x[u].y, v[i].y);
+        v[i].z = fmaf(w[u], x[u].z, v[i].z); v[i].w = fmaf(w[u], x[u].w, v[i].w);
+      }
     }
   }
 #pragma unroll
@@ -532,7 +614,9 @@ GB_OP(gb_op_moe_dispatch) {
 #define DISPATCH(T)                                                                                                     \
     gb_launch(moe_dispatch_kernel<T>, grid, dim3(DISPATCH_THREADS), smem, ctx->stream, p, op_ptr<int>(a[9]), op_ptr<float>(a[10]), \
               op_ptr<int>(a[13]), op_ptr<int>(a[14]), op_ptr<int>(a[15]), op_ptr<const T>(a[16]), a[17], op_ptr<T>(a[19]), a[20],   \
-              (int)a[21], flags & 1)
+              (int)a[21], flags & 1, vec)
+    const long long size = a[18] == GB_BF16 ? 2 : 4;
+    const int vec = ((a[16] | a[19] | a[17] * size | a[20] * size | a[21] * size) & 15) == 0;
     if (a[18] == GB_BF16) DISPATCH(bf16); else DISPATCH(float);
 #undef DISPATCH
     GB_CHECK_LAUNCH("moe_dispatch");
@@ -578,6 +662,14 @@ GB_OP(gb_op_moe_gather) {
   const int pairs = (int)(a[7] * a[9]), width = (int)a[8];
   if (pairs <= 0) return 0;
   const dim3 grid(pairs), block(width <= 256 ? 64 : 256);
+  const long long size = a[2] == GB_BF16 ? 2 : 4;
+  if (!a[4] && ((a[0] | a[5] | a[1] * size | a[6] * size | width * size) & 15) == 0) {
+    const int pieces = (int)(width * size / 16), lanes = pieces >= 128 ? 128 : pieces >= 64 ? 64 : 32;
+    gb_launch(moe_gather16_kernel, dim3(gb_div_up(pairs, 256 / lanes)), dim3(256), 0, ctx->stream, op_ptr<const char>(a[0]), a[1] * size,
+              op_ptr<const int>(a[3]), op_ptr<char>(a[5]), a[6] * size, pairs, pieces, (int)a[9], lanes);
+    GB_CHECK_LAUNCH("moe_gather");
+    return 1;
+  }
   if (a[2] == GB_BF16)
     gb_launch(moe_gather_kernel<bf16>, grid, block, 0, ctx->stream, op_ptr<const bf16>(a[0]), a[1], op_ptr<const int>(a[3]),
               op_ptr<const float>(a[4]), op_ptr<bf16>(a[5]), a[6], pairs, width, (int)a[9]);

@@ -27,7 +27,9 @@ namespace {
 
 using namespace sm100;
 
-constexpr int BM = 128, BK = 64, UMMA_K = 16, STAGES = 4;
+constexpr int BM = 128, BK = 64, UMMA_K = 16;
+// (stages: as many as leave room for two blocks an SM)
+template <int BN> constexpr int stages_of() { return BN <= 64 ? 4 : 3; }
 constexpr int W_TILE_BYTES = BM * BK * 2;
 constexpr int STATUS_TIMEOUT = 24;
 
@@ -48,6 +50,7 @@ template <int BN>
 __global__ void __launch_bounds__(192)
 moe_experts_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant__ CUtensorMap tmap_x,
                       const GroupedParams p) {
+  constexpr int STAGES = stages_of<BN>();
   constexpr int X_TILE_BYTES = BN * BK * 2, STAGE_BYTES = W_TILE_BYTES + X_TILE_BYTES;
   constexpr int TMEM_COLS = BN < 32 ? 32 : BN;
   pdl_trigger();
@@ -262,7 +265,7 @@ std::unordered_map<WKey, CUtensorMap, WKeyHash> g_wmaps;   // weights do not mov
 template <int BN>
 int launch(const CUtensorMap& tw, const CUtensorMap& tx, const GroupedParams& p, int weight_tiles, int row_tiles,
            cudaStream_t stream) {
-  constexpr int SMEM = STAGES * (W_TILE_BYTES + BN * BK * 2) + 1024;
+  constexpr int SMEM = stages_of<BN>() * (W_TILE_BYTES + BN * BK * 2) + 1024;
   static bool raised = false;
   if (!raised) {
     GB_CUDA(cudaFuncSetAttribute(moe_experts_tc_kernel<BN>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM));
@@ -306,7 +309,8 @@ GB_OP(gb_op_moe_experts_tc) {
     }
   }
   // few rows an expert (decoding): narrow token tiles
-  const int BN = pairs <= 16 * E ? 16 : 64;
+  // (and wide ones where an expert has many: a tile's weights are read from L2 once for twice the tokens)
+  const int BN = pairs <= 16 * E ? 16 : pairs < 192 * E ? 64 : 128;
   if (!make_tmap(&tx, op_ptr<const void>(a[0]), a[2], K, a[1], BN))
     GB_FAIL(GB_ERR_CUDA, "moe_experts_tc: cuTensorMapEncodeTiled failed (rows)");
   GroupedParams p;
@@ -319,8 +323,9 @@ GB_OP(gb_op_moe_experts_tc) {
   p.status = ctx->status;
   const int weight_tiles = gb_div_up(rows_per_expert, BM);
   const int row_tiles = gb_div_up(pairs, BN) + E;          // at most this many over all experts
-  return BN == 16 ? launch<16>(tw, tx, p, weight_tiles, row_tiles, ctx->stream)
-                  : launch<64>(tw, tx, p, weight_tiles, row_tiles, ctx->stream);
+  return BN == 16   ? launch<16>(tw, tx, p, weight_tiles, row_tiles, ctx->stream)
+         : BN == 64 ? launch<64>(tw, tx, p, weight_tiles, row_tiles, ctx->stream)
+                    : launch<128>(tw, tx, p, weight_tiles, row_tiles, ctx->stream);
 }
 
 // Forget the tensor maps of weights (a model was unloaded).
