@@ -385,18 +385,23 @@ __global__ void __launch_bounds__(READ_THREADS) delta_chunk_read_kernel(DeltaChu
 template <int DK>
 int launch(const DeltaChunkParams& p, int n, cudaStream_t stream) {
   constexpr int prep_smem = 4 * (2 * DC * (DK + 4) + 2 * DC * (DC + 4) + 3 * DC);
+  // A launch that begins while the kernel in front still runs is placed where there is room, several blocks on the SMs that
+  // emptied first.  The scan lives on one SM's shared memory a block: with no more blocks than SMs it asks for so much of it that
+  // two do not fit.
+  constexpr int scan_alone = ScanLayout<DK>::BYTES > 120 * 1024 ? ScanLayout<DK>::BYTES : 120 * 1024;
   static bool raised = false;                            // once, before any stream capture replays the launch
   if (!raised) {
     GB_CUDA(cudaFuncSetAttribute(delta_chunk_prep_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, prep_smem));
-    GB_CUDA(cudaFuncSetAttribute(delta_chunk_scan_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, ScanLayout<DK>::BYTES));
+    GB_CUDA(cudaFuncSetAttribute(delta_chunk_scan_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, scan_alone));
     GB_CUDA(cudaFuncSetAttribute(delta_chunk_read_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, ReadLayout<DK>::BYTES));
     raised = true;
   }
   const int chunks = gb_delta_chunks_count(n, p.R);
   gb_launch(delta_chunk_prep_kernel<DK>, dim3(chunks, p.H), dim3(PREP_THREADS), prep_smem, stream, p);
   GB_CHECK_LAUNCH("delta_scan (chunks by themselves)");
-  gb_launch(delta_chunk_scan_kernel<DK>, dim3(p.R, p.H, gb_div_up(p.vdim, SCAN_COLS)), dim3(ScanLayout<DK>::THREADS),
-            ScanLayout<DK>::BYTES, stream, p);
+  const dim3 scan_grid(p.R, p.H, gb_div_up(p.vdim, SCAN_COLS));
+  const int scan_smem = (long long)scan_grid.x * scan_grid.y * scan_grid.z <= 148 ? scan_alone : ScanLayout<DK>::BYTES;
+  gb_launch(delta_chunk_scan_kernel<DK>, scan_grid, dim3(ScanLayout<DK>::THREADS), scan_smem, stream, p);
   GB_CHECK_LAUNCH("delta_scan (chunks in order)");
   gb_launch(delta_chunk_read_kernel<DK>, dim3(chunks, p.H, gb_div_up(p.vdim, READ_COLS)), dim3(READ_THREADS), ReadLayout<DK>::BYTES,
             stream, p);
