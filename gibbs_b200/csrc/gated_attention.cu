@@ -84,9 +84,10 @@ enum { PREP_NORM_WHOLE = 1, PREP_Q_BF16 = 2, PREP_PAGES_BF16 = 4, PREP_NORM_HEAD
 // One normed and rotated element of a projection: entry d of a head of `dim` entries that starts at `base`.
 // `gain` is indexed like the projection (norm over the whole projection) or by d (`gain_per_head`: one gain
 // vector shared by all heads).  The first `rot_dims` entries turn by pos * inv_freq[i], in adjacent pairs
-// (2i, 2i+1) or, with `halves`, in pairs (i, i + rot_dims/2); `turns` holds their cosines and sines.
+// (2i, 2i+1) or, with `halves`, in pairs (i, i + rot_dims/2); cosines and sines are multiplied by mscale.
 __device__ __forceinline__ float prep_element(const float* x, const float* __restrict__ gain, bool gain_per_head,
-                                              float rstd, int base, int d, int rot_dims, bool halves, const float* turns) {
+                                              float rstd, int base, int d, int rot_dims, bool halves,
+                                              const float* __restrict__ inv_freq, int pos, float mscale) {
   const int gb = gain_per_head ? 0 : base;
   const float own = x[base + d] * rstd * (gain ? gain[gb + d] : 1.f);
   if (d >= rot_dims) return own;
@@ -95,7 +96,8 @@ __device__ __forceinline__ float prep_element(const float* x, const float* __res
   const int partner = halves ? (second ? d - half : d + half) : (d ^ 1);
   const int fi = halves ? (second ? d - half : d) : (d >> 1);
   const float other = x[base + partner] * rstd * (gain ? gain[gb + partner] : 1.f);
-  const float c = turns[2 * fi], s = turns[2 * fi + 1];
+  const float ang = (float)pos * inv_freq[fi];
+  const float c = cosf(ang) * mscale, s = sinf(ang) * mscale;
   // the pair (u, v) becomes (u c - v s, v c + u s)
   return second ? own * c + other * s : own * c - other * s;
 }
@@ -104,30 +106,24 @@ __device__ __forceinline__ float prep_element(const float* x, const float* __res
 // attention), and so is a key head: a key row in the pages holds them all.  A warp takes one head of `dim`
 // entries at a time: its norm (when heads are normed one by one), then its elements.
 template <typename TC, typename TQ>
-__global__ void qk_prep_kernel(const float* fused, long long ld, int k_col, int v_col, const float* __restrict__ q_gain,
+__global__ void __launch_bounds__(512, 3) qk_prep_kernel(const float* fused, long long ld, int k_col, int v_col, const float* __restrict__ q_gain,
                                const float* __restrict__ k_gain, const float* __restrict__ inv_freq, int rot_dims,
                                const int* tok_req, const int* tok_pos, const int* block_table, int bt_stride,
                                int page_size, TC* k_pages, TC* v_pages, int n_pages, int H, int G, int dim, int vdim,
                                int maps, int mode, float eps, float temp_coef, float temp_every, TQ* q_out, long long ldq,
                                int* status) {
   __shared__ float scratch[32];
-  extern __shared__ float turns[];                       // [rot_dims / 2] pairs of cosine and sine: the same for every head
   pdl_trigger();
   const int t = blockIdx.x;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
   const int pos = tok_pos[t];
-  for (int i = threadIdx.x; i < rot_dims >> 1; i += blockDim.x) {
-    const float ang = (float)pos * inv_freq[i], mscale = inv_freq[rot_dims >> 1];
-    turns[2 * i] = cosf(ang) * mscale;
-    turns[2 * i + 1] = sinf(ang) * mscale;
-  }
-  __syncthreads();
   const bool writes = k_pages != nullptr;
   const bool whole = mode & PREP_NORM_WHOLE, per_head = mode & PREP_NORM_HEAD, halves = mode & PREP_ROT_HALVES;
   // PREP_NORM_AFTER: every head is turned first and then divided by the root mean square of the TURNED head (no gain)
   const bool after = mode & PREP_NORM_AFTER;
   // a query grows with its position: 1 + coef * ln(floor((pos + 1) / every) + 1)
   const float temp = temp_every > 0.f ? fmaf(temp_coef, logf(floorf((float)(pos + 1) / temp_every) + 1.f), 1.f) : 1.f;
+  const float mscale = rot_dims > 0 ? inv_freq[rot_dims >> 1] : 1.f;
   int page = -1;
   if (writes) page = block_table[(size_t)tok_req[t] * bt_stride + pos / page_size];
   pdl_wait();
@@ -156,14 +152,14 @@ __global__ void qk_prep_kernel(const float* fused, long long ld, int k_col, int 
     if (after) {
       float ss = 0.f;
       for (int d = lane; d < dim; d += 32) {
-        const float v = prep_element(row, nullptr, true, 1.f, h * dim, d, rot_dims, halves, turns);
+        const float v = prep_element(row, nullptr, true, 1.f, h * dim, d, rot_dims, halves, inv_freq, pos, mscale);
         ss += v * v;
       }
       post = temp / sqrtf(warp_sum(ss) / (float)dim + eps);
     }
     for (int d = lane; d < dim; d += 32)
       q_out[(size_t)t * ldq + h * dim + d] = from_f32<TQ>(post * prep_element(row, normed ? q_gain : nullptr, per_head, rstd,
-                                                                              h * dim, d, rot_dims, halves, turns));
+                                                                              h * dim, d, rot_dims, halves, inv_freq, pos, mscale));
   }
   if (!writes) return;
   if (page < 0 || page >= n_pages) {
@@ -184,14 +180,14 @@ __global__ void qk_prep_kernel(const float* fused, long long ld, int k_col, int 
     if (after) {
       float ss = 0.f;
       for (int d = lane; d < dim; d += 32) {
-        const float v = prep_element(row + k_col, nullptr, true, 1.f, h * dim, d, rot_dims, halves, turns);
+        const float v = prep_element(row + k_col, nullptr, true, 1.f, h * dim, d, rot_dims, halves, inv_freq, pos, mscale);
         ss += v * v;
       }
       post = 1.0f / sqrtf(warp_sum(ss) / (float)dim + eps);
     }
     for (int d = lane; d < dim; d += 32)
       dst[d] = from_f32<TC>(post * prep_element(row + k_col, normed ? k_gain : nullptr, per_head, rstd, h * dim, d, rot_dims,
-                                                halves, turns));
+                                                halves, inv_freq, pos, mscale));
   }
   for (int i = threadIdx.x; i < G * vdim; i += blockDim.x) {
     const int g = i / vdim, d = i - g * vdim;
@@ -508,7 +504,7 @@ GB_OP(gb_op_qk_prep) {
   const long long ldq = (long long)H * maps * dim;
   const int mode = flags & (PREP_NORM_WHOLE | PREP_NORM_HEAD | PREP_ROT_HALVES | PREP_NORM_AFTER);
 #define PREP(TC, TQ)                                                                                                     \
-  gb_launch(qk_prep_kernel<TC, TQ>, dim3(n), dim3(threads), sizeof(float) * (size_t)a[7], ctx->stream, op_ptr<const float>(a[0]), a[1], (int)a[2],    \
+  gb_launch(qk_prep_kernel<TC, TQ>, dim3(n), dim3(threads), 0, ctx->stream, op_ptr<const float>(a[0]), a[1], (int)a[2],    \
             (int)a[3], op_ptr<const float>(a[4]), op_ptr<const float>(a[5]), op_ptr<const float>(a[6]), (int)a[7],        \
             op_ptr<const int>(a[8]), op_ptr<const int>(a[9]), op_ptr<const int>(a[10]), (int)a[11], (int)a[12],           \
             op_ptr<TC>(a[13]), op_ptr<TC>(a[14]), (int)a[15], H, G, dim, vdim, maps, mode, (float)f[0], (float)f[1], \
