@@ -198,7 +198,7 @@ int run_op(Walk& w, const PlanOp& o, bool force = false) {
       // symbol), a8 n, a9 k, a10 kernel (0 tensor cores, 1 FFMA), a11 mode (0 bf16, 1 f32, 2 add into f32, 3 SwiGLU),
       // a12 x dtype, a13 W dtype, a14 out dtype; mode 3 with f0 != 0: the gated unit's constants f0 alpha, f1 limit
       // (0: none), f2 what is added to u (all zero: SwiGLU), a15 the bits of a 32-bit float: the cubic term inside the
-      // gate's sigmoid (0: none); mode 0: a16 a function of the finished sums (0: none, 1: the square of relu)
+      // gate's sigmoid (0: none); mode 0: a16 a function of the finished sums (0: none, 1: the square of relu, 2: the exact gelu)
       const bool glu = a[11] == 3 && o.f[0] != 0.0;
       const int M = (int)val(w, a[7]);
       if (M <= 0) return 0;

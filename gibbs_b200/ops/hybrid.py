@@ -1,5 +1,5 @@
 """Bindings of the "hybrid" kernel library (csrc/norms.cu, latent_attention.cu,
-gated_attention.cu, gated_attention_tc.cu, sigmoid_attention_tc.cu, ssm.cu, selective_scan.cu, delta_rule.cu,
+gated_attention.cu, gated_attention_tc.cu, sigmoid_attention_tc.cu, ssm.cu, selective_scan.cu, delta_rule.cu, delta_chunks.cu,
 linear_scan.cu, streams.cu, moe.cu): layer norms, clamped gated units, latent attention, gated attention with a sink,
 attention without a softmax, state-space, delta-rule and linear recurrences, residual streams and routed experts.
 
